@@ -14,12 +14,22 @@ _lib = None
 
 _c_int, _c_float, _c_void_p, _c_char_p = ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_char_p
 
+
+class LayerSpec(ctypes.Structure):
+    """cpmcu_layer_spec of include/cpmcu_b200.h: one layer of a layered model."""
+    _fields_ = [("heads", _c_int), ("kv_heads", _c_int), ("dim", _c_int), ("vdim", _c_int), ("scale", _c_float),
+                ("window", _c_int), ("bias_exp", _c_float), ("qk_norm", _c_int), ("kv_from", _c_int), ("experts", _c_int),
+                ("identity", _c_int), ("top", _c_int), ("groups", _c_int), ("keep_groups", _c_int),
+                ("router_scale", _c_float), ("expert_ff", _c_int), ("shared_ff", _c_int)]
+
+
 _SIGNATURES = {
     "cpmcu_last_error": (_c_char_p, []),
     "cpmcu_init_base_model": (_c_int, [_c_float] + [_c_int] * 7 + [_c_float, _c_int, _c_int] + [_c_float] * 3),
     "cpmcu_init_minicpm4_model": (_c_int, [_c_float] + [_c_int] * 7 + [_c_float, _c_int, _c_int] + [_c_float] * 3 + [_c_int] * 5),
     "cpmcu_init_w4a16_gptq_marlin_base_model": (_c_int, [_c_float] + [_c_int] * 7 + [_c_float, _c_int, _c_int, _c_int] + [_c_float] * 3),
     "cpmcu_init_w4a16_gptq_marlin_minicpm4_model": (_c_int, [_c_float] + [_c_int] * 7 + [_c_float, _c_int, _c_int, _c_int] + [_c_float] * 3 + [_c_int] * 5),
+    "cpmcu_init_layered_model": (_c_int, [_c_float, _c_int, _c_int, _c_float, _c_float] + [_c_int] * 3 + [_c_void_p]),
     "cpmcu_init_eagle_model": (_c_int, [_c_int] * 5),
     "cpmcu_init_minicpm4_eagle_model": (_c_int, [_c_int] * 9 + [_c_float, _c_int, _c_int]),
     "cpmcu_init_w4a16_gm_spec_w4a16_gm_model": (_c_int, []),
@@ -28,6 +38,7 @@ _SIGNATURES = {
     "cpmcu_init_storage": (_c_int, []),
     "cpmcu_load_model": (_c_int, [_c_char_p, _c_void_p]),
     "cpmcu_prefill": (_c_int, [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p]),
+    "cpmcu_prefill_rows": (_c_int, [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p]),
     "cpmcu_decode": (_c_int, [_c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int]),
     "cpmcu_draft": (_c_int, [_c_void_p] * 5),
     "cpmcu_verify_and_fix": (_c_int, [_c_int] + [_c_void_p] * 6),
@@ -44,7 +55,16 @@ _SIGNATURES = {
     "cpmcu_total_launches": (ctypes.c_long, []),
     "cpmcu_get_tree": (_c_int, [_c_void_p] * 6),
     "cpmcu_capture_blockmasks": (_c_int, [_c_void_p]),
+    "cpmcu_capture_layers": (_c_int, [_c_void_p]),
+    "cpmcu_profile": (_c_int, [_c_int, _c_void_p, _c_void_p]),
     "cpmcu_release": (None, []),
+    "cpmcu_layer_attention": (_c_int, [_c_void_p] * 4 + [_c_int] * 5 + [_c_void_p]),
+    "cpmcu_layer_qkv_norm_append": (_c_int, [_c_void_p] * 4 + [_c_float] + [_c_int] * 4 + [_c_void_p] * 3),
+    "cpmcu_layer_out_norm": (_c_int, [_c_void_p] * 3 + [_c_float, _c_void_p] + [_c_int] * 3 + [_c_float, _c_int]),
+    "cpmcu_moe_route": (_c_int, [_c_void_p] * 4 + [_c_int] * 2 + [_c_void_p] * 2),
+    "cpmcu_layer_mixture": (_c_int, [_c_void_p] * 7 + [_c_float, _c_void_p] + [_c_int] * 3 + [_c_float]),
+    "cpmcu_bench_experts": (_c_int, [_c_void_p] + [_c_int] * 4 + [_c_void_p]),
+    "cpmcu_bench_layer_attention": (_c_int, [_c_void_p] + [_c_int] * 4 + [_c_void_p]),
     "cpmcu_linear_bf16": (_c_int, [_c_void_p] * 4 + [_c_int] * 4),
     "cpmcu_linear_w4a16": (_c_int, [_c_void_p] * 4 + [_c_int] * 4),
     "cpmcu_bench_linear": (_c_int, [_c_int] * 6 + [_c_void_p]),
@@ -150,6 +170,13 @@ def init_w4a16_gptq_marlin_minicpm4_model(memory_limit, vocab_size, num_hidden_l
          sparse_switch, int(apply_compress_lse))
 
 
+def init_layered_model(memory_limit, vocab_size, width, norm_eps, residual_mult, torch_dtype, chunk_length, layers):
+    """layers: a list of LayerSpec."""
+    arr = (LayerSpec * len(layers))(*layers)
+    call("cpmcu_init_layered_model", memory_limit, vocab_size, width, norm_eps, residual_mult, torch_dtype, chunk_length,
+         len(layers), ctypes.cast(arr, _c_void_p))
+
+
 def init_eagle_model(num_layers, num_iter, topk_per_iter, tree_size, torch_dtype):
     call("cpmcu_init_eagle_model", num_layers, num_iter, topk_per_iter, tree_size, torch_dtype)
 
@@ -184,6 +211,13 @@ def load_model(name, param):
 
 def prefill(input_length, history_length, input, position_ids, output):
     call("cpmcu_prefill", input_length, history_length, input, position_ids, output)
+
+
+def prefill_rows(input_length, history_length, input, position_ids, want, output):
+    """want: list of token places in this chunk whose logits are written, in order, to `output`."""
+    arr = (ctypes.c_int32 * max(1, len(want)))(*want)
+    call("cpmcu_prefill_rows", input_length, history_length, input, position_ids, ctypes.cast(arr, _c_void_p), len(want),
+         output or None)
 
 
 def decode(input_length, padded_length, input, position_ids, cache_length, mask_2d, output, cuda_graph):
@@ -231,6 +265,14 @@ def profile_step():
     call("cpmcu_profile_step", ctypes.cast(ms, _c_void_p), ctypes.cast(cnt, _c_void_p),
          ctypes.cast(ctypes.pointer(total), _c_void_p))
     return {"linear": (ms[0], cnt[0]), "attention": (ms[1], cnt[1]), "selection": (ms[2], cnt[2])}, total.value
+
+
+def profile(on):
+    """profile(True) starts per-launch timing; profile(False) stops and returns {class: (ms, launches)}."""
+    ms, cnt = (ctypes.c_float * 6)(), (ctypes.c_int * 6)()
+    call("cpmcu_profile", int(on), ctypes.cast(ms, _c_void_p), ctypes.cast(cnt, _c_void_p))
+    names = ("linear", "attention", "selection", "experts", "routing", "rows")
+    return {n: (ms[i], cnt[i]) for i, n in enumerate(names)}
 
 
 def last_step_ms():

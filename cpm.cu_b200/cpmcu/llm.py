@@ -3,10 +3,14 @@ library.  Same constructor keywords, `init_storage`, `_load`, `load_from_hf`,
 `prefill`, `decode` and `generate` contracts; all device work happens in
 libcpmcu_b200.so through `cpmcu.C`.
 
-Two additions that the reference does not have, both optional:
+Additions that the reference does not have, all optional:
   * `config=` / `tokenizer=` let a caller pass a ready configuration object
     instead of a Hugging Face directory (used with synthetic weights);
-  * `load_state_dict()` feeds tensors that are already in memory.
+  * `load_state_dict_tensors()` feeds tensors that are already in memory;
+  * `extend()` appends a portion of a sequence and returns the logits of chosen
+    tokens of it.
+Other model designs subclass it (`tipetar.py`) and override the three hooks
+`_read_config`, `_create_native` and `_load`.
 """
 import glob
 import json
@@ -20,7 +24,7 @@ import torch.nn.functional as F
 
 from . import C
 
-dtype_map = {torch.float16: 0, torch.bfloat16: 1}
+dtype_map = {torch.float16: 0, torch.bfloat16: 1, torch.float32: 2}
 
 
 def dtype_to_int(dtype):
@@ -45,13 +49,7 @@ class LLM(torch.nn.Module):
                  random_seed=None, minicpm4_yarn=False, config=None, tokenizer=None):
         super().__init__()
         self.path = path
-        if config is None:
-            from transformers import AutoConfig, AutoTokenizer
-            self.tokenizer = AutoTokenizer.from_pretrained(path, trust_remote_code=True)
-            self.config = AutoConfig.from_pretrained(path, trust_remote_code=True)
-        else:
-            self.tokenizer = tokenizer
-            self.config = config if not isinstance(config, dict) else types.SimpleNamespace(**config)
+        self._read_config(path, config, tokenizer)
         self.dtype = dtype if dtype is not None else getattr(self.config, "torch_dtype", torch.bfloat16)
         self.dtype_int = dtype_to_int(self.dtype)
         self.cuda_graph = cuda_graph
@@ -72,16 +70,28 @@ class LLM(torch.nn.Module):
             self.generator = torch.Generator(device="cuda")
             self.generator.manual_seed(random_seed)
 
+        self._create_native(memory_limit, apply_sparse,
+                            (sink_window_size, block_window_size, sparse_topk_k, sparse_switch, apply_compress_lse))
+        self.logits = torch.empty((64, self.config.vocab_size), dtype=self.dtype, device="cuda")
+        self.max_total_length = 0
+
+    def _read_config(self, path, config, tokenizer):
+        if config is None:
+            from transformers import AutoConfig, AutoTokenizer
+            self.tokenizer = AutoTokenizer.from_pretrained(path, trust_remote_code=True)
+            self.config = AutoConfig.from_pretrained(path, trust_remote_code=True)
+        else:
+            self.tokenizer = tokenizer
+            self.config = config if not isinstance(config, dict) else types.SimpleNamespace(**config)
+
+    def _create_native(self, memory_limit, apply_sparse, sparse_args):
         cfg = self.config
         if not hasattr(cfg, "head_dim") or cfg.head_dim is None:
             cfg.head_dim = cfg.hidden_size // cfg.num_attention_heads
         scale_embed = getattr(cfg, "scale_emb", 1.0)
         scale_lmhead = (cfg.dim_model_base / cfg.hidden_size) if hasattr(cfg, "dim_model_base") else 1.0
         scale_residual = cfg.scale_depth / math.sqrt(cfg.num_hidden_layers) if hasattr(cfg, "scale_depth") else 1.0
-        self._init_native(memory_limit, scale_embed, scale_lmhead, scale_residual, apply_sparse,
-                          (sink_window_size, block_window_size, sparse_topk_k, sparse_switch, apply_compress_lse))
-        self.logits = torch.empty((64, cfg.vocab_size), dtype=self.dtype, device="cuda")
-        self.max_total_length = 0
+        self._init_native(memory_limit, scale_embed, scale_lmhead, scale_residual, apply_sparse, sparse_args)
 
     def _init_native(self, memory_limit, scale_embed, scale_lmhead, scale_residual, apply_sparse, sparse_args):
         """Create the native model (bf16 target).  Quantised subclasses override this."""
@@ -209,6 +219,40 @@ class LLM(torch.nn.Module):
         cache_length -= n
         return self.logits[:n].clone()
 
+    def _decode_one(self, token, position):
+        """Logits [1, vocab] after `token`, which becomes row `position` of the cache."""
+        if not hasattr(self, "input_ids"):
+            self.input_ids = torch.tensor([0], dtype=torch.int32, device="cuda")
+            self.position_ids = torch.tensor([0], dtype=torch.int32, device="cuda")
+            self.cache_length = torch.tensor([0], dtype=torch.int32, device="cuda")
+        self.input_ids[0] = token
+        self.position_ids[0] = position
+        self.cache_length[0] = position
+        return self.decode(self.input_ids, self.position_ids, self.cache_length)
+
+    def extend(self, tokens, history, want):
+        """Append `tokens` (a list of ids) behind the `history` tokens the cache holds; history 0 starts a new sequence.
+        Returns the logits [len(want), vocab] of the places `want` among these tokens.  A single token behind others is
+        a decoding step, everything else a prefill in chunks."""
+        n = len(tokens)
+        if history + n > self.max_total_length:
+            raise ValueError(f"{history} cached + {n} new tokens exceed the {self.max_total_length} tokens the KV cache holds "
+                             f"under the current memory limit")
+        if n == 1 and history > 0:
+            return self._decode_one(tokens[0], history)[[0] * len(want)]
+        ids = torch.tensor(tokens, dtype=torch.int32, device="cuda")
+        pos = torch.arange(history, history + n, dtype=torch.int32, device="cuda")
+        out = torch.empty((len(want), self.config.vocab_size), dtype=self.dtype, device="cuda")
+        for i in range(0, n, self.chunk_length):
+            m = min(n - i, self.chunk_length)
+            rows = sorted({w - i for w in want if i <= w < i + m})
+            part = torch.empty((len(rows), self.config.vocab_size), dtype=self.dtype, device="cuda")
+            C.prefill_rows(m, history + i, ids[i:].data_ptr(), pos[i:].data_ptr(), rows, part.data_ptr())
+            for k, w in enumerate(want):
+                if i <= w < i + m:
+                    out[k] = part[rows.index(w - i)]
+        return out
+
     def _pick(self, logits):
         if self.temperature > 0.0:
             probs = F.softmax(logits.float() / self.temperature, dim=-1)
@@ -241,18 +285,11 @@ class LLM(torch.nn.Module):
         torch.cuda.synchronize()
         prefill_time = time.time() - t0
         token = self._pick(logits[0]).item()
-        if not hasattr(self, "input_ids"):
-            self.input_ids = torch.tensor([0], dtype=torch.int32, device="cuda")
-            self.position_ids = torch.tensor([0], dtype=torch.int32, device="cuda")
-            self.cache_length = torch.tensor([0], dtype=torch.int32, device="cuda")
 
         def steps():
             nonlocal token
             for i in range(generation_length - 1):
-                self.input_ids[0] = token
-                self.position_ids[0] = prefix_length + i
-                self.cache_length[0] = prefix_length + i
-                logits = self.decode(self.input_ids, self.position_ids, self.cache_length)
+                logits = self._decode_one(token, prefix_length + i)
                 token = self._pick(logits[0]).item()
                 yield token
 

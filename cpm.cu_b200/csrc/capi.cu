@@ -1,6 +1,7 @@
 // extern "C" surface of libcpmcu_b200.so (declared in include/cpmcu_b200.h).
 // Holds the single global model the reference keeps in src/entry.cu:98 and
 // turns C++ exceptions into return codes + a thread-local message.
+#include <algorithm>
 #include <cstdio>
 #include <memory>
 #include <vector>
@@ -159,6 +160,42 @@ int cpmcu_init_w4a16_gptq_marlin_minicpm4_model(float memory_limit, int vocab_si
                        scale_residual, group_size, &sp);
 }
 
+}  // extern "C"
+
+namespace {
+LayerSpec to_spec(const cpmcu_layer_spec& c) {
+    LayerSpec s;
+    s.heads = c.heads; s.kv_heads = c.kv_heads; s.dim = c.dim; s.vdim = c.vdim;
+    s.scale = c.scale; s.window = c.window; s.bias_exp = c.bias_exp; s.qk_norm = c.qk_norm; s.kv_from = c.kv_from;
+    s.experts = c.experts; s.identity = c.identity; s.top = c.top; s.groups = c.groups; s.keep_groups = c.keep_groups;
+    s.router_scale = c.router_scale; s.expert_ff = c.expert_ff; s.shared_ff = c.shared_ff;
+    return s;
+}
+}  // namespace
+
+extern "C" {
+
+int cpmcu_init_layered_model(float memory_limit, int vocab_size, int width, float norm_eps, float residual_mult,
+                             int torch_dtype, int chunk_length, int num_layers, const cpmcu_layer_spec* layers) {
+    return guarded([&] {
+        CPM_REQUIRE(torch_dtype == 1 || torch_dtype == 2, "layered models run in torch_dtype 1 (bfloat16) or 2 (float32)");
+        CPM_REQUIRE(num_layers >= 1 && layers != nullptr, "layered model: no layers");
+        ModelConfig mc;
+        mc.memory_limit = memory_limit;
+        mc.vocab = vocab_size;
+        mc.layers = num_layers;
+        mc.hidden = width;
+        mc.eps = norm_eps;
+        mc.chunk_length = chunk_length;
+        mc.scale_residual = residual_mult;
+        mc.fp32 = torch_dtype == 2;
+        for (int i = 0; i < num_layers; ++i) mc.specs.push_back(to_spec(layers[i]));
+        g_engine.reset();
+        g_engine = std::make_unique<Engine>(mc);
+        return 0;
+    });
+}
+
 int cpmcu_init_eagle_model(int num_layers, int num_iter, int topk_per_iter, int tree_size, int torch_dtype) {
     return guarded([&] {
         require_bf16(torch_dtype);
@@ -218,7 +255,44 @@ int cpmcu_load_model(const char* name, const void* param) {
 int cpmcu_prefill(int input_length, int history_length, const int32_t* input, const int32_t* position_ids,
                   void* output) {
     return guarded([&] {
-        engine().prefill(input_length, history_length, input, position_ids, static_cast<bf16*>(output));
+        engine().prefill(input_length, history_length, input, position_ids, output);
+        return 0;
+    });
+}
+
+int cpmcu_prefill_rows(int input_length, int history_length, const int32_t* input, const int32_t* position_ids,
+                       const int32_t* want, int n_want, void* output) {
+    return guarded([&] {
+        engine().prefill_rows(input_length, history_length, input, position_ids, want, n_want, output);
+        return 0;
+    });
+}
+
+int cpmcu_capture_layers(float* device_buf) {
+    return guarded([&] {
+        engine().capture_layers(device_buf);
+        return 0;
+    });
+}
+
+int cpmcu_profile(int on, float* ms, int* launches) {
+    return guarded([&] {
+        Runtime& rt = runtime();
+        CUDA_CHECK(cudaStreamSynchronize(rt.stream));
+        for (int k = 0; k < KC_COUNT; ++k) {
+            double sum = 0.0;
+            for (auto& pr : rt.prof[k]) {
+                float x = 0.f;
+                if (pr.second != nullptr) cudaEventElapsedTime(&x, pr.first, pr.second);
+                sum += x;
+                cudaEventDestroy(pr.first);
+                cudaEventDestroy(pr.second);
+            }
+            if (!on && ms) ms[k] = static_cast<float>(sum);
+            if (!on && launches) launches[k] = static_cast<int>(rt.prof[k].size());
+            rt.prof[k].clear();
+        }
+        rt.profile = on != 0;
         return 0;
     });
 }
@@ -227,7 +301,7 @@ int cpmcu_decode(int input_length, int padded_length, const int32_t* input, cons
                  const int32_t* cache_length, const uint64_t* mask_2d, void* output, int cuda_graph) {
     return guarded([&] {
         engine().decode(input_length, padded_length, input, position_ids, cache_length, mask_2d,
-                        static_cast<bf16*>(output), cuda_graph != 0);
+                        output, cuda_graph != 0);
         return 0;
     });
 }
@@ -647,6 +721,282 @@ int cpmcu_silu_gate(const void* gate_up, void* out, int rows, int inter) {
     return guarded([&] {
         launch_silu_gate(static_cast<const bf16*>(gate_up), static_cast<bf16*>(out), rows, inter, runtime().stream);
         sync_and_check("silu_gate");
+        return 0;
+    });
+}
+
+// ---- mechanisms of layered models
+int cpmcu_layer_attention(const cpmcu_layer_spec* spec, const void* q, const void* k_cache, const void* v_cache, int budget,
+                          int tq, int kv_total, int splits, int fp32, void* out) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        cudaStream_t s = runtime().stream;
+        const int dk = pad64(sp.dim), dv = pad64(sp.vdim), out_ld = sp.heads * sp.vdim;
+        CPM_REQUIRE(tq >= 1 && kv_total >= tq && kv_total <= budget, "layer_attention: lengths out of range");
+        DeviceBuf len(4);
+        CUDA_CHECK(cudaMemcpyAsync(len.p, &kv_total, 4, cudaMemcpyHostToDevice, s));
+        if (splits >= 1) {
+            CPM_REQUIRE(!fp32 && biased_attn_fits(sp.heads, sp.kv_heads, dk, dv), "layer_attention: shape needs the plain kernel");
+            const size_t rows = static_cast<size_t>(tq) * sp.heads;
+            DeviceBuf ws_o(rows * splits * dv * 4), ws_ml(rows * splits * 2 * 4);
+            AttnPlan p = make_biased_attn_plan(static_cast<const bf16*>(q), sp.heads * dk, static_cast<const bf16*>(k_cache),
+                                               static_cast<const bf16*>(v_cache), budget, tq, sp.heads, sp.kv_heads, dk, dv, sp.vdim,
+                                               splits, sp.scale, sp.window, sp.bias_exp, static_cast<bf16*>(out), out_ld,
+                                               static_cast<float*>(ws_o.p), static_cast<float*>(ws_ml.p));
+            p.kv_len = static_cast<const int32_t*>(len.p);
+            launch_tree_attention(p, s);
+            sync_and_check("layer_attention");
+            return 0;
+        }
+        PlainAttnArgs a;
+        a.q = q; a.k_cache = k_cache; a.v_cache = v_cache; a.out = out;
+        a.tq = tq; a.hq = sp.heads; a.hkv = sp.kv_heads; a.dk = dk; a.dv = dv; a.out_cols = sp.vdim; a.out_ld = out_ld;
+        a.kv_len = static_cast<const int32_t*>(len.p); a.kv_len_add = 0;
+        a.scale = sp.scale; a.window = sp.window; a.bias_exp = sp.bias_exp;
+        if (fp32) launch_plain_attention<float>(a, s);
+        else launch_plain_attention<bf16>(a, s);
+        sync_and_check("layer_attention");
+        return 0;
+    });
+}
+
+int cpmcu_layer_qkv_norm_append(const cpmcu_layer_spec* spec, const void* qkv, const void* wq, const void* wk, float eps,
+                                int rows, int kv_row, int cache_rows, int fp32, void* q_out, void* k_cache, void* v_cache) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        cudaStream_t s = runtime().stream;
+        DeviceBuf len(4);
+        CUDA_CHECK(cudaMemcpyAsync(len.p, &kv_row, 4, cudaMemcpyHostToDevice, s));
+        QkvNormArgs a;
+        a.qkv = qkv;
+        a.ld = sp.heads * sp.dim + (k_cache ? sp.kv_heads * (sp.dim + sp.vdim) : 0);
+        a.heads = sp.heads; a.kv_heads = sp.kv_heads;
+        a.dim = sp.dim; a.dim_p = pad64(sp.dim); a.vdim = sp.vdim; a.vdim_p = pad64(sp.vdim);
+        a.wq = static_cast<const bf16*>(wq); a.wk = static_cast<const bf16*>(wk); a.eps = eps;
+        a.q_out = q_out; a.k_cache = k_cache; a.v_cache = v_cache;
+        a.kv_len = static_cast<const int32_t*>(len.p); a.kv_off = 0; a.cache_rows = cache_rows; a.error = runtime().d_error;
+        if (fp32) launch_qkv_norm_append<float>(a, rows, s);
+        else launch_qkv_norm_append<bf16>(a, rows, s);
+        sync_and_check("layer_qkv_norm_append");
+        return 0;
+    });
+}
+
+int cpmcu_layer_out_norm(float* x32, void* xh, const void* delta, float mult, const void* w, int rows, int width, int ld,
+                         float eps, int fp32) {
+    return guarded([&] {
+        cudaStream_t s = runtime().stream;
+        const bf16* wb = static_cast<const bf16*>(w);
+        if (fp32) launch_out_norm<float>(x32, static_cast<float*>(xh), static_cast<const float*>(delta), MoeMix(), mult, wb, rows, width, ld, eps, s);
+        else launch_out_norm<bf16>(x32, static_cast<bf16*>(xh), static_cast<const bf16*>(delta), MoeMix(), mult, wb, rows, width, ld, eps, s);
+        sync_and_check("layer_out_norm");
+        return 0;
+    });
+}
+
+}  // extern "C"
+
+namespace {
+// Router results, row groups and counters of a stand-alone call.
+struct MoeScratch {
+    DeviceBuf z, expert, weight, rank, id_weight, counts, offset, entries, n_entries, tickets;
+    MoeBuffers b;
+    MoeScratch(const LayerSpec& sp, int rows, cudaStream_t s)
+        : z(static_cast<size_t>(rows) * (sp.experts + sp.identity) * 4), expert(static_cast<size_t>(rows) * sp.top * 4),
+          weight(static_cast<size_t>(rows) * sp.top * 4), rank(static_cast<size_t>(rows) * sp.top * 4), id_weight(static_cast<size_t>(rows) * 4),
+          counts((sp.experts + sp.identity) * 4), offset((sp.experts + sp.identity) * 4), entries(kMoeMaxEntries * 16), n_entries(4),
+          tickets(moe_ticket_ints(rows) * 4) {
+        CUDA_CHECK(cudaMemsetAsync(counts.p, 0, (sp.experts + sp.identity) * 4, s));
+        CUDA_CHECK(cudaMemsetAsync(tickets.p, 0, moe_ticket_ints(rows) * 4, s));
+        b.z = static_cast<float*>(z.p);
+        b.expert = static_cast<int32_t*>(expert.p);
+        b.weight = static_cast<float*>(weight.p);
+        b.rank = static_cast<int32_t*>(rank.p);
+        b.id_weight = static_cast<float*>(id_weight.p);
+        b.counts = static_cast<int32_t*>(counts.p);
+        b.offset = static_cast<int32_t*>(offset.p);
+        b.entries = static_cast<int4*>(entries.p);
+        b.n_entries = static_cast<int32_t*>(n_entries.p);
+        b.tickets = static_cast<int32_t*>(tickets.p);
+    }
+};
+
+void check_mixture(const LayerSpec& sp, int rows, int ld) {
+    const int n = sp.experts + sp.identity;
+    CPM_REQUIRE(rows >= 1 && ld >= 64 && ld % 64 == 0 && ld <= 16384, "mixture: rows must be padded to a multiple of 64 columns");
+    CPM_REQUIRE(sp.experts >= 1 && sp.identity >= 0 && n <= kMoeMaxOutputs && sp.groups >= 1 && n % sp.groups == 0 && sp.keep_groups >= 1 &&
+                    sp.keep_groups <= sp.groups && sp.top >= 1 && sp.top <= kMoeMaxTop && sp.top <= n / sp.groups * sp.keep_groups,
+                "mixture: bad expert counts or groups");
+}
+}  // namespace
+
+extern "C" {
+
+int cpmcu_moe_route(const cpmcu_layer_spec* spec, const float* x32, const void* router, const float* correction, int rows,
+                    int ld, int32_t* expert, float* weight) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        check_mixture(sp, rows, ld);
+        cudaStream_t s = runtime().stream;
+        MoeScratch m(sp, rows, s);
+        launch_moe_route(sp, x32, static_cast<const bf16*>(router), correction, m.b, rows, ld, moe_pick_tile(sp, rows), false, s);
+        CUDA_CHECK(cudaMemcpyAsync(expert, m.b.expert, static_cast<size_t>(rows) * sp.top * 4, cudaMemcpyDeviceToDevice, s));
+        CUDA_CHECK(cudaMemcpyAsync(weight, m.b.weight, static_cast<size_t>(rows) * sp.top * 4, cudaMemcpyDeviceToDevice, s));
+        sync_and_check("moe_route");
+        return 0;
+    });
+}
+
+int cpmcu_layer_mixture(const cpmcu_layer_spec* spec, float* x32, void* xh, const void* router, const float* correction,
+                        const void* gate_up, const void* down, float mult, const void* w, int rows, int width, int ld, float eps) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        check_mixture(sp, rows, ld);
+        cudaStream_t s = runtime().stream;
+        MoeScratch m(sp, rows, s);
+        // the caller's row-major matrices into the kernels' layout
+        const size_t gu_bytes = moe_gate_up_elems(sp, ld) * 2, dn_bytes = moe_down_elems(sp, width) * 2;
+        DeviceBuf gu(gu_bytes), dn(dn_bytes);
+        CUDA_CHECK(cudaMemsetAsync(gu.p, 0, gu_bytes, s));
+        CUDA_CHECK(cudaMemsetAsync(dn.p, 0, dn_bytes, s));
+        const bf16 *g = static_cast<const bf16*>(gate_up), *d = static_cast<const bf16*>(down);
+        for (int e = 0; e < sp.experts + (sp.shared_ff > 0 ? 1 : 0); ++e) {
+            const int ff = e < sp.experts ? sp.expert_ff : sp.shared_ff;
+            bf16* ge = static_cast<bf16*>(gu.p) + moe_gate_up_offset(sp, ld, e);
+            retile_weight_rows(g, ff, width, ge, ld, 1, 0, 0, s);
+            retile_weight_rows(g + static_cast<size_t>(ff) * width, ff, width, ge, ld, 2, 0, 0, s);
+            retile_weight_rows(d, width, ff, static_cast<bf16*>(dn.p) + moe_down_offset(sp, width, e), pad64(ff), 0, 0, 0, s);
+            g += static_cast<size_t>(2) * ff * width;
+            d += static_cast<size_t>(width) * ff;
+        }
+        const int slots = rows * (sp.top + (sp.shared_ff > 0 ? 1 : 0)), ld_act = std::max(pad64(sp.expert_ff), pad64(sp.shared_ff));
+        DeviceBuf mx(static_cast<size_t>(rows) * sp.top * ld * 2), act(static_cast<size_t>(slots) * ld_act * 2), y(static_cast<size_t>(slots) * ld * 2);
+        CUDA_CHECK(cudaMemsetAsync(y.p, 0, static_cast<size_t>(slots) * ld * 2, s));
+        const bool single = rows == 1;
+        const int tile = moe_pick_tile(sp, rows);
+        const bf16* x = static_cast<const bf16*>(xh);
+        MoeGemmPlan p1 = make_moe_gate_up_plan(sp, static_cast<const bf16*>(gu.p), single ? x : static_cast<const bf16*>(mx.p),
+                                               single ? 1 : rows * sp.top, x, ld, static_cast<bf16*>(act.p), ld_act, rows, tile, m.b);
+        MoeGemmPlan p2 = make_moe_down_plan(sp, static_cast<const bf16*>(dn.p), static_cast<const bf16*>(act.p), slots, ld_act, width,
+                                            static_cast<bf16*>(y.p), ld, rows, tile, m.b);
+        launch_moe_route(sp, x32, static_cast<const bf16*>(router), correction, m.b, rows, ld, tile, single, s);
+        if (!single) launch_moe_gather<bf16>(sp, x, static_cast<bf16*>(mx.p), m.b, rows, ld, s);
+        launch_moe_gemm(p1, s);
+        launch_moe_gemm(p2, s);
+        MoeMix mix;
+        mix.y = y.p; mix.expert = m.b.expert; mix.weight = m.b.weight; mix.rank = m.b.rank; mix.offset = m.b.offset; mix.id_weight = m.b.id_weight;
+        mix.top = sp.top; mix.experts = sp.experts;
+        mix.shared_row0 = sp.shared_ff > 0 ? rows * sp.top : -1;
+        launch_out_norm<bf16>(x32, static_cast<bf16*>(xh), nullptr, mix, mult, static_cast<const bf16*>(w), rows, width, ld, eps, s);
+        sync_and_check("layer_mixture");
+        return 0;
+    });
+}
+
+int cpmcu_bench_experts(const cpmcu_layer_spec* spec, int width, int rows, int copies, int iters, float* us) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        const int ld = pad64(width);
+        check_mixture(sp, rows, ld);
+        CPM_REQUIRE(copies >= 1 && copies <= 64 && iters >= 1, "bench_experts: bad repetition counts");
+        cudaStream_t s = runtime().stream;
+        MoeScratch m(sp, rows, s);
+        const int tile = moe_pick_tile(sp, rows);
+        // every expert gets the same number of rows (the first ones one more)
+        std::vector<int4> ent;
+        const int slots_e = rows * std::min(sp.top, sp.experts);
+        int at = 0;
+        for (int e = 0; e < sp.experts && at < slots_e; ++e) {
+            const int cnt = slots_e / sp.experts + (e < slots_e % sp.experts ? 1 : 0);
+            const int ne = ceil_div(cnt, tile);
+            for (int k = 0; k < ne; ++k) {
+                const int b = static_cast<int>(static_cast<long long>(cnt) * k / ne), c = static_cast<int>(static_cast<long long>(cnt) * (k + 1) / ne);
+                ent.push_back(make_int4(e, rows == 1 ? 0 : at + b, at + b, c - b));
+            }
+            at += cnt;
+        }
+        CPM_REQUIRE(ent.size() <= static_cast<size_t>(kMoeMaxEntries), "bench_experts: too many row groups");
+        const int n_ent = static_cast<int>(ent.size());
+        CUDA_CHECK(cudaMemcpyAsync(m.b.entries, ent.data(), ent.size() * 16, cudaMemcpyHostToDevice, s));
+        CUDA_CHECK(cudaMemcpyAsync(m.b.n_entries, &n_ent, 4, cudaMemcpyHostToDevice, s));
+        const size_t gu_elems = moe_gate_up_elems(sp, ld), dn_elems = moe_down_elems(sp, width);
+        const int slots = rows * (sp.top + (sp.shared_ff > 0 ? 1 : 0)), ld_act = std::max(pad64(sp.expert_ff), pad64(sp.shared_ff));
+        DeviceBuf gu(gu_elems * 2 * copies), dn(dn_elems * 2 * copies), x(static_cast<size_t>(rows) * ld * 2);
+        DeviceBuf mx(static_cast<size_t>(rows) * sp.top * ld * 2), act(static_cast<size_t>(slots) * ld_act * 2), y(static_cast<size_t>(slots) * ld * 2);
+        CUDA_CHECK(cudaMemsetAsync(gu.p, 0x3c, gu_elems * 2 * copies, s));
+        CUDA_CHECK(cudaMemsetAsync(dn.p, 0x3c, dn_elems * 2 * copies, s));
+        CUDA_CHECK(cudaMemsetAsync(x.p, 0x3c, static_cast<size_t>(rows) * ld * 2, s));
+        CUDA_CHECK(cudaMemsetAsync(mx.p, 0x3c, static_cast<size_t>(rows) * sp.top * ld * 2, s));
+        CUDA_CHECK(cudaMemsetAsync(act.p, 0x3c, static_cast<size_t>(slots) * ld_act * 2, s));
+        for (int which = 0; which < 2; ++which) {
+            std::vector<MoeGemmPlan> plans;
+            for (int c = 0; c < copies; ++c) {
+                if (which == 0) {
+                    plans.push_back(make_moe_gate_up_plan(sp, static_cast<const bf16*>(gu.p) + gu_elems * c,
+                                                          static_cast<const bf16*>(rows == 1 ? x.p : mx.p), rows == 1 ? 1 : rows * sp.top,
+                                                          static_cast<const bf16*>(x.p), ld, static_cast<bf16*>(act.p), ld_act, rows, tile, m.b));
+                } else {
+                    plans.push_back(make_moe_down_plan(sp, static_cast<const bf16*>(dn.p) + dn_elems * c, static_cast<const bf16*>(act.p), slots,
+                                                       ld_act, width, static_cast<bf16*>(y.p), ld, rows, tile, m.b));
+                }
+            }
+            for (int c = 0; c < 3; ++c) launch_moe_gemm(plans[c % copies], s);
+            cudaEvent_t e0, e1;
+            CUDA_CHECK(cudaEventCreate(&e0));
+            CUDA_CHECK(cudaEventCreate(&e1));
+            CUDA_CHECK(cudaEventRecord(e0, s));
+            for (int i = 0; i < iters; ++i) launch_moe_gemm(plans[i % copies], s);
+            CUDA_CHECK(cudaEventRecord(e1, s));
+            CUDA_CHECK(cudaStreamSynchronize(s));
+            float ms = 0.f;
+            CUDA_CHECK(cudaEventElapsedTime(&ms, e0, e1));
+            cudaEventDestroy(e0);
+            cudaEventDestroy(e1);
+            us[which] = ms * 1000.f / iters;
+        }
+        sync_and_check("bench_experts");
+        return 0;
+    });
+}
+
+int cpmcu_bench_layer_attention(const cpmcu_layer_spec* spec, int rows, int kv_total, int splits, int iters, float* us) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        cudaStream_t s = runtime().stream;
+        const int budget = (kv_total + 255) / 128 * 128, layers = 8;
+        const int dk = pad64(sp.dim), dv = pad64(sp.vdim);
+        const size_t kb = static_cast<size_t>(budget) * sp.kv_heads * dk * 2, vb = static_cast<size_t>(budget) * sp.kv_heads * dv * 2;
+        DeviceBuf q(static_cast<size_t>(rows) * sp.heads * dk * 2), k(kb * layers), v(vb * layers), out(static_cast<size_t>(rows) * sp.heads * sp.vdim * 2), len(4);
+        const size_t n = static_cast<size_t>(rows) * sp.heads;
+        DeviceBuf ws_o(n * splits * dv * 4), ws_ml(n * splits * 2 * 4);
+        CUDA_CHECK(cudaMemsetAsync(q.p, 0x3c, n * dk * 2, s));
+        CUDA_CHECK(cudaMemsetAsync(k.p, 0x3c, kb * layers, s));
+        CUDA_CHECK(cudaMemsetAsync(v.p, 0x3c, vb * layers, s));
+        CUDA_CHECK(cudaMemcpyAsync(len.p, &kv_total, 4, cudaMemcpyHostToDevice, s));
+        std::vector<AttnPlan> plans;
+        for (int l = 0; l < layers; ++l) {
+            plans.push_back(make_biased_attn_plan(static_cast<const bf16*>(q.p), sp.heads * dk,
+                                                  reinterpret_cast<const bf16*>(static_cast<uint8_t*>(k.p) + kb * l),
+                                                  reinterpret_cast<const bf16*>(static_cast<uint8_t*>(v.p) + vb * l), budget, rows, sp.heads,
+                                                  sp.kv_heads, dk, dv, sp.vdim, splits, sp.scale, sp.window, sp.bias_exp,
+                                                  static_cast<bf16*>(out.p), sp.heads * sp.vdim, static_cast<float*>(ws_o.p),
+                                                  static_cast<float*>(ws_ml.p)));
+            plans.back().kv_len = static_cast<const int32_t*>(len.p);
+        }
+        for (int l = 0; l < 3; ++l) launch_tree_attention(plans[l], s);
+        cudaEvent_t e0, e1;
+        CUDA_CHECK(cudaEventCreate(&e0));
+        CUDA_CHECK(cudaEventCreate(&e1));
+        CUDA_CHECK(cudaEventRecord(e0, s));
+        for (int i = 0; i < iters; ++i) launch_tree_attention(plans[i % layers], s);
+        CUDA_CHECK(cudaEventRecord(e1, s));
+        CUDA_CHECK(cudaStreamSynchronize(s));
+        float ms = 0.f;
+        CUDA_CHECK(cudaEventElapsedTime(&ms, e0, e1));
+        cudaEventDestroy(e0);
+        cudaEventDestroy(e1);
+        *us = ms * 1000.f / iters;
+        sync_and_check("bench_layer_attention");
         return 0;
     });
 }

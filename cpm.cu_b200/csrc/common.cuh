@@ -54,9 +54,18 @@ enum KernelError : int {
     ERR_ATTN_TIMEOUT = 2,
     ERR_BAD_TREE = 4,
     ERR_KV_OVERFLOW = 8,  // a K/V row beyond the cache budget was about to be written (the store is skipped)
+    ERR_BAD_TOKEN = 16,   // a token id outside the vocabulary (token 0 was used in its place)
 };
 
-enum KernelClass : int { KC_LINEAR = 0, KC_ATTENTION = 1, KC_OTHER = 2, KC_COUNT = 3 };
+enum KernelClass : int {
+    KC_LINEAR = 0,
+    KC_ATTENTION = 1,
+    KC_OTHER = 2,
+    KC_MOE = 3,   // grouped expert products
+    KC_ROUTE = 4, // router, row layout and gather of a mixture of experts
+    KC_ROW = 5,   // row-wise kernels of layered models
+    KC_COUNT = 6
+};
 
 struct Runtime {
     cudaStream_t stream = nullptr;
@@ -280,7 +289,11 @@ struct AttnPlan {
     CUtensorMap tm_q;  // [tq, hq, d] viewed as 3-D (d, heads, tokens)
     CUtensorMap tm_k;  // [budget, hkv*d]
     CUtensorMap tm_v;
-    int tq = 0, hq = 0, hkv = 0, d = 128;
+    int tq = 0, hq = 0, hkv = 0, d = 128, dv = 128;
+    int out_cols = 128;               // value columns stored per head
+    bool biased = false;              // made by make_biased_attn_plan
+    int exact_window = 0;             // biased plans: > 0 = per-token sliding window (tokens)
+    float bias_exp = 0.f;             // biased plans: > 0 = distance bias with slopes 2^(-bias_exp * (h + 1) / hq)
     int splits = 1;
     const int32_t* kv_len = nullptr;  // device scalar
     int kv_len_add = 0;               // keys visible = *kv_len + kv_len_add
@@ -301,4 +314,12 @@ size_t attn_workspace_bytes(int tq, int hq, int d, int splits);
 AttnPlan make_attn_plan(const bf16* q, int q_ld_tokens, const bf16* k_cache, const bf16* v_cache, int budget,
                         int tq, int hq, int hkv, int d, int splits, bf16* out, int out_ld, float* ws_o,
                         float* ws_ml);
+// The same kernel with key / value rows of dk / dv (64 or 128) columns per head, of which out_cols value columns are real,
+// any GQA ratio up to 128, an exact per-token window and a distance bias:
+//   score = scale * (q . k) - 2^(-bias_exp * (h + 1) / hq) * (i - j),   0 <= i - j < exact_window
+// (exact_window 0 = no window, bias_exp 0 = no bias).  q: token t, head h at q + t * q_ld + h * dk.
+bool biased_attn_fits(int hq, int hkv, int dk, int dv);
+AttnPlan make_biased_attn_plan(const bf16* q, int q_ld_tokens, const bf16* k_cache, const bf16* v_cache, int budget, int tq,
+                               int hq, int hkv, int dk, int dv, int out_cols, int splits, float scale, int exact_window,
+                               float bias_exp, bf16* out, int out_ld, float* ws_o, float* ws_ml);
 void launch_tree_attention(const AttnPlan& plan, cudaStream_t s);

@@ -475,6 +475,15 @@ __global__ void retile_rows_kernel(const bf16* __restrict__ src, int first_row, 
     *reinterpret_cast<uint4*>(dst + tile_major_offset(retile_dst_row(first_row + r, mode, row_offset), k_offset + c8 * 8, K)) = v;
 }
 
+// the same one element at a time, for row lengths that are not multiples of 8
+__global__ void retile_rows_scalar_kernel(const bf16* __restrict__ src, int first_row, int rows, int src_cols,
+                                          bf16* __restrict__ dst, int K, int mode, int row_offset, int k_offset) {
+    const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+    if (idx >= static_cast<size_t>(rows) * src_cols) return;
+    const int r = static_cast<int>(idx / src_cols), c = static_cast<int>(idx - static_cast<size_t>(r) * src_cols);
+    dst[tile_major_offset(retile_dst_row(first_row + r, mode, row_offset), k_offset + c, K)] = src[idx];
+}
+
 __global__ void gather_retiled_kernel(const bf16* __restrict__ src, const int32_t* __restrict__ idx, bf16* __restrict__ dst,
                                       int K) {
     const int d = blockIdx.x, s = idx[d];
@@ -490,13 +499,21 @@ size_t linear_weight_elems(int N, int K) { return static_cast<size_t>(ceil_div(N
 void retile_weight_rows(const void* src, int rows, int src_cols, bf16* dst, int K, int mode, int row_offset, int k_offset,
                         cudaStream_t s) {
     if (rows <= 0) return;
-    CPM_REQUIRE(src_cols % 8 == 0 && K % 64 == 0 && k_offset % 8 == 0 && k_offset + src_cols <= K, "retile: bad column range");
+    CPM_REQUIRE(K % 64 == 0 && k_offset % 8 == 0 && k_offset + src_cols <= K, "retile: bad column range");
     CPM_REQUIRE(mode >= 0 && mode <= 2 && (mode == 0 || row_offset == 0), "retile: bad row mapping");
     cudaPointerAttributes attr = {};
     const bool on_device = cudaPointerGetAttributes(&attr, src) == cudaSuccess &&
                            (attr.type == cudaMemoryTypeDevice || attr.type == cudaMemoryTypeManaged);
     cudaGetLastError();  // an unregistered host pointer is not an error here
+    const bool vec = src_cols % 8 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
     auto run = [&](const bf16* rows_on_device, int first_row, int n) {
+        if (!vec) {
+            const size_t elems = static_cast<size_t>(n) * src_cols;
+            retile_rows_scalar_kernel<<<static_cast<unsigned>((elems + 255) / 256), 256, 0, s>>>(
+                rows_on_device, first_row, n, src_cols, dst, K, mode, row_offset, k_offset);
+            CUDA_CHECK(cudaGetLastError());
+            return;
+        }
         const size_t threads = static_cast<size_t>(n) * (src_cols / 8);
         retile_rows_kernel<<<static_cast<unsigned>((threads + 255) / 256), 256, 0, s>>>(rows_on_device, first_row, n, src_cols, dst,
                                                                                       K, mode, row_offset, k_offset);

@@ -40,8 +40,6 @@ __global__ void publish_kernel(const int32_t* result, const int32_t* tokens, con
     if (threadIdx.x < 16) out[1 + threadIdx.x] = (threadIdx.x < n) ? tokens[threadIdx.x] : -1;
 }
 
-// The engine's split-K counters (two per output tile) live in one buffer of kTicketInts ints.
-constexpr int kTicketInts = 1 << 16;
 LinearPlan checked(const LinearPlan& p) {
     CPM_REQUIRE(2LL * ceil_div(p.N, 128) * ceil_div(p.M, p.mt) <= kTicketInts,
                 "linear: more output tiles than the engine's split-K counters cover");
@@ -66,6 +64,13 @@ void* Engine::Pool::take(size_t bytes) {
 }
 
 Engine::Engine(const ModelConfig& mc) : mc_(mc) {
+    if (layered()) {
+        check_specs();
+        lw_.resize(mc.specs.size());
+        runtime();
+        return;
+    }
+    CPM_REQUIRE(!mc.fp32, "only layered models run in fp32");
     CPM_REQUIRE(mc.head_dim == 128, "only head_dim 128 is supported");
     CPM_REQUIRE(mc.hidden % 64 == 0 && mc.inter % 64 == 0, "hidden and intermediate sizes must be multiples of 64");
     CPM_REQUIRE(mc.hq % mc.hkv == 0, "num_attention_heads must be a multiple of num_key_value_heads");
@@ -83,6 +88,7 @@ Engine::Engine(const ModelConfig& mc) : mc_(mc) {
 
 Engine::~Engine() {
     if (step_graph_) cudaGraphExecDestroy(step_graph_);
+    if (decode_graph_) cudaGraphExecDestroy(decode_graph_);
     if (ev0_) cudaEventDestroy(ev0_);
     if (ev1_) cudaEventDestroy(ev1_);
     if (ev_mid_) cudaEventDestroy(ev_mid_);
@@ -92,6 +98,7 @@ Engine::~Engine() {
 
 void Engine::attach_eagle(const EagleConfig& ec) {
     CPM_REQUIRE(!storage_ready_, "attach the drafter before init_storage");
+    CPM_REQUIRE(!layered(), "layered models have no EAGLE drafter");
     CPM_REQUIRE(ec.num_layers == 1, "only a 1-layer EAGLE drafter is supported");
     CPM_REQUIRE(ec.tree_size >= 2 && ec.tree_size <= 64, "tree_size must be in [2,64]");
     CPM_REQUIRE(ec.topk >= 1 && ec.topk <= 32 && ec.topk <= ec.tree_size - 1, "topk_per_iter out of range");
@@ -128,6 +135,10 @@ int Engine::attn_splits_for(int rows) const {
 }
 
 void Engine::lay_out(Pool& p) {
+    if (layered()) {
+        lay_out_layered(p);
+        return;
+    }
     const int H = mc_.hidden, I = mc_.inter, V = mc_.vocab, d = mc_.head_dim;
     const int kvd = mc_.hkv * d;
     const size_t R = max_rows_;
@@ -265,6 +276,7 @@ int Engine::init_storage() {
     lay_out(count);
     const size_t fixed = count.used + (1 << 20);
     size_t per_token = static_cast<size_t>(mc_.layers + (has_eagle_ ? 1 : 0)) * 2 * mc_.hkv * mc_.head_dim * 2;
+    if (layered()) per_token = layered_bytes_per_token();
     if (mc_.sparse.enabled) {
         // c1 + c2 rows per layer (1/16 + 1/64 of a key row), one score per 16 tokens and one mask bit per 64
         // tokens for each of the hkv * max_rows_ (kv head, query) pairs
@@ -294,8 +306,10 @@ int Engine::init_storage() {
     CUDA_CHECK(cudaMemsetAsync(pool_.base, 0, pool_.cap, rt.stream));
     std::vector<bf16*> ptrs;
     for (auto& c : kv_) { ptrs.push_back(c.k); ptrs.push_back(c.v); }
-    CUDA_CHECK(cudaMemcpyAsync(d_cache_ptrs_, ptrs.data(), ptrs.size() * sizeof(bf16*), cudaMemcpyHostToDevice,
-                               rt.stream));
+    if (!ptrs.empty()) {
+        CUDA_CHECK(cudaMemcpyAsync(d_cache_ptrs_, ptrs.data(), ptrs.size() * sizeof(bf16*), cudaMemcpyHostToDevice,
+                                   rt.stream));
+    }
     CUDA_CHECK(cudaStreamSynchronize(rt.stream));
     CUDA_CHECK(cudaMallocHost(&h_result_, 32 * sizeof(int32_t)));
     memset(h_result_, 0, 32 * sizeof(int32_t));
@@ -333,6 +347,10 @@ int Engine::init_storage() {
 // ------------------------------------------------------------------ loading
 void Engine::load(const std::string& name, const void* src) {
     CPM_REQUIRE(storage_ready_, "load_model before init_storage");
+    if (layered()) {
+        load_layered(name, src);
+        return;
+    }
     Runtime& rt = runtime();
     const int H = mc_.hidden, I = mc_.inter, d = mc_.head_dim;
     auto copy = [&](void* dst, size_t bytes) {
@@ -579,15 +597,29 @@ void Engine::target_forward(ForwardPlans& fp, const RowCtx& c, const int32_t* id
         pending = delta_;
     }
     launch_add_rms_norm(x_, pending, mc_.scale_residual, final_norm_, norm_out_, rows, H, mc_.eps, s);
+    if (logits_out == nullptr) return;
     if (all_logits) lm_head_rows(norm_out_, rows, rows, logits_out, logits_ld, s);
     else lm_head_rows(norm_out_ + static_cast<size_t>(rows - 1) * H, 1, 1, logits_out, logits_ld, s);
 }
 
 // ------------------------------------------------------------------ prefill / decode (reference API)
-void Engine::prefill(int n, int history, const int32_t* ids, const int32_t* pos, bf16* logits_out) {
+void Engine::prefill(int n, int history, const int32_t* ids, const int32_t* pos, void* logits_out) {
+    const int32_t last = n - 1;
+    prefill_rows(n, history, ids, pos, &last, 1, logits_out);
+}
+
+void Engine::prefill_rows(int n, int history, const int32_t* ids, const int32_t* pos, const int32_t* want, int n_want,
+                          void* logits_out) {
     CPM_REQUIRE(storage_ready_, "prefill before init_storage");
     CPM_REQUIRE(n >= 1 && n <= max_rows_, "prefill chunk larger than chunk_length");
     CPM_REQUIRE(history >= 0 && history + n <= budget_, "prefill exceeds the KV budget");
+    CPM_REQUIRE(n_want >= 0 && n_want <= n, "prefill: more logits asked for than tokens");
+    for (int i = 0; i < n_want; ++i) CPM_REQUIRE(want[i] >= 0 && want[i] < n, "prefill: logits asked for a token outside the chunk");
+    if (layered()) {
+        layered_prefill(n, history, ids, want, n_want, logits_out);
+        return;
+    }
+    const int last_only = (n_want == 1 && want[0] == n - 1);
     Runtime& rt = runtime();
     cudaStream_t s = rt.stream;
     const int H = mc_.hidden;
@@ -612,12 +644,16 @@ void Engine::prefill(int n, int history, const int32_t* ids, const int32_t* pos,
         for (int k = 0; k < KC_COUNT; ++k) rt.prof[k].clear();
         rt.profile = true;
     }
-    target_forward(fp, c, ids, false, logits_out, mc_.vocab, s);
+    target_forward(fp, c, ids, false, last_only ? static_cast<bf16*>(logits_out) : nullptr, mc_.vocab, s);
+    for (int i = 0; i < n_want && !last_only; ++i) {
+        lm_head_rows(norm_out_ + static_cast<size_t>(want[i]) * H, 1, 1, static_cast<bf16*>(logits_out) + static_cast<size_t>(i) * mc_.vocab,
+                     mc_.vocab, s);
+    }
     if (prof_prefill) {
         // CUDA events around every launch of the pass: time per kernel class, and the GEMMs of the last layer
         rt.profile = false;
         CUDA_CHECK(cudaStreamSynchronize(s));
-        const char* names[KC_COUNT] = {"linear", "attention", "other"};
+        const char* names[KC_COUNT] = {"linear", "attention", "other", "experts", "route", "rows"};
         for (int k = 0; k < KC_COUNT; ++k) {
             double sum = 0.0;
             std::vector<float> each;
@@ -653,13 +689,18 @@ void Engine::prefill(int n, int history, const int32_t* ids, const int32_t* pos,
 }
 
 void Engine::decode(int n, int padded_len, const int32_t* ids, const int32_t* pos, const int32_t* cache_length,
-                    const uint64_t* mask, bf16* logits_out, bool cuda_graph) {
-    (void)cuda_graph;
+                    const uint64_t* mask, void* logits_out, bool cuda_graph) {
     CPM_REQUIRE(storage_ready_, "decode before init_storage");
     CPM_REQUIRE(n >= 1 && n <= 64, "decode supports 1..64 tokens");
     // padded_len is the caller's ceil((cache length + n) / 128) * 128 and the budget is a multiple of 128
     CPM_REQUIRE(padded_len <= 0 || padded_len <= budget_, "decode: cache length + tokens exceeds the KV budget");
     require_room(n, "decode");
+    if (layered()) {
+        CPM_REQUIRE(mask == nullptr, "decode: layered models take no tree mask");
+        layered_decode(n, ids, cache_length, logits_out, cuda_graph);
+        return;
+    }
+    (void)cuda_graph;
     cudaStream_t s = runtime().stream;
     RowCtx c;
     c.rows = n;
@@ -669,7 +710,7 @@ void Engine::decode(int n, int padded_len, const int32_t* ids, const int32_t* po
     c.attn_kv_add = 0;
     c.mask = mask;
     c.mask_k = mask ? n : 0;
-    target_forward(target_plans(n), c, ids, true, logits_out, mc_.vocab, s);
+    target_forward(target_plans(n), c, ids, true, static_cast<bf16*>(logits_out), mc_.vocab, s);
     CUDA_CHECK(cudaStreamSynchronize(s));
     check_errors("decode");
 }
@@ -896,7 +937,7 @@ void Engine::check_errors(const char* where) {
         }
         throw std::runtime_error(std::string("cpmcu_b200: kernel error flags ") + std::to_string(e) + " raised in " +
                                  where + " (1 = GEMM pipeline timeout, 2 = attention pipeline timeout, 4 = malformed draft tree, "
-                                 "8 = K/V row beyond the cache budget)");
+                                 "8 = K/V row beyond the cache budget, 16 = token id outside the vocabulary)");
     }
 }
 
@@ -1076,8 +1117,10 @@ void Engine::profile_step(float* ms, int* counts, float* total_ms) {
             cudaEventDestroy(pr.first);
             cudaEventDestroy(pr.second);
         }
-        ms[c] = static_cast<float>(sum);
-        counts[c] = static_cast<int>(rt.prof[c].size());
+        if (c < 3) {   // the classes a speculative step launches
+            ms[c] = static_cast<float>(sum);
+            counts[c] = static_cast<int>(rt.prof[c].size());
+        }
         rt.prof[c].clear();
     }
     if (h_result_[31] != 0) check_errors("profile_step");

@@ -8,11 +8,13 @@
 #pragma once
 #include <map>
 #include <memory>
+#include <set>
 #include <string>
 #include <vector>
 
 #include "common.cuh"
 #include "draft_tree.cuh"
+#include "layered.cuh"
 #include "sparse_select.cuh"
 
 struct ModelConfig {
@@ -24,6 +26,10 @@ struct ModelConfig {
     bool w4a16 = false;  // target linears arrive as GPTQ-Marlin int4 + scales (embeddings / LM head stay bf16)
     int group_size = 128;
     SparseConfig sparse;  // InfLLM-v2 block selection in the target layers (init_minicpm4_model)
+    // Layered models: every layer described by its own LayerSpec (empty for Llama-format targets), norms on the
+    // sublayers' outputs, a 32-bit residual stream scaled by scale_residual
+    std::vector<LayerSpec> specs;
+    bool fp32 = false;    // activations, caches and logits in fp32 (layered models only)
 };
 
 struct EagleConfig {
@@ -54,6 +60,26 @@ struct KVLayer {
     bf16* v = nullptr;
 };
 
+// One layer of a layered model.  bf16 models keep the matrices tile-major (linear_weight_elems), fp32 models row-major.
+struct LayeredWeights {
+    bf16 *qkv = nullptr, *o = nullptr;          // rows q | k | v (q alone with kv_from); o: K = pad64(heads * vdim)
+    bf16 *q_norm = nullptr, *k_norm = nullptr, *norm1 = nullptr, *norm2 = nullptr;
+    bf16* router = nullptr;                     // [outputs][ld]
+    float* correction = nullptr;                // [outputs]
+    bf16 *gate_up = nullptr, *down = nullptr;   // expert after expert, the shared expert last
+    void *k = nullptr, *v = nullptr;            // cache rows [budget][kv_heads][pad64(dim) | pad64(vdim)]; kv_from: that layer's
+};
+struct LayeredPlans {
+    struct Layer {
+        LinearPlan qkv, o;
+        AttnPlan attn;
+        bool tensor_attn = false;   // head widths the tensor-core attention kernel takes
+        MoeGemmPlan gate_up, down;
+    };
+    int rows = 0, tile = 0;
+    std::vector<Layer> layers;
+};
+
 // How a batch of rows walks through a decoder layer.
 struct RowCtx {
     int rows = 0;
@@ -79,6 +105,9 @@ struct ForwardPlans {
     std::vector<LayerPlans> layers;
 };
 
+// The engine's split-K counters (two per output tile) live in one buffer of kTicketInts ints.
+constexpr int kTicketInts = 1 << 16;
+
 class Engine {
 public:
     explicit Engine(const ModelConfig& mc);
@@ -88,9 +117,11 @@ public:
     void load(const std::string& name, const void* src);
 
     // reference-compatible entry points (device pointers owned by the caller)
-    void prefill(int n, int history, const int32_t* ids, const int32_t* pos, bf16* logits_out);
+    void prefill(int n, int history, const int32_t* ids, const int32_t* pos, void* logits_out);
+    // the same with the logits of rows want[0..n_want) (host) of this chunk, [n_want, vocab]
+    void prefill_rows(int n, int history, const int32_t* ids, const int32_t* pos, const int32_t* want, int n_want, void* logits_out);
     void decode(int n, int padded_len, const int32_t* ids, const int32_t* pos, const int32_t* cache_length,
-                const uint64_t* mask, bf16* logits_out, bool cuda_graph);
+                const uint64_t* mask, void* logits_out, bool cuda_graph);
     void draft(int32_t* tree_ids, int32_t* tree_pos, const int32_t* cache_length, uint64_t* tree_mask,
                int32_t* tree_parent);
     int verify_and_fix(int T, int32_t* pred, const int32_t* gt, const int32_t* pos, const int32_t* cache_length,
@@ -112,6 +143,10 @@ public:
     double last_verify_ms() const { return last_verify_ms_; }
     long launches_per_step() const { return launches_per_step_; }
 
+    bool layered() const { return !mc_.specs.empty(); }
+    // test hook: the residual stream after every layer of each forward pass, [layers][rows][width] fp32 at `buf` (device
+    // memory owned by the caller; null stops it)
+    void capture_layers(float* buf) { layer_capture_ = buf; }
     const ModelConfig& config() const { return mc_; }
     bool has_eagle() const { return has_eagle_; }
     int budget() const { return budget_; }
@@ -135,6 +170,26 @@ private:
     void lay_out(Pool& pool);
     template <typename T>
     T* take(Pool& pool, size_t count) { return reinterpret_cast<T*>(pool.take(count * sizeof(T))); }
+
+    // ---- layered models (engine_layered.cu)
+    void check_specs() const;
+    void lay_out_layered(Pool& pool);
+    size_t layered_bytes_per_token() const;
+    void load_layered(const std::string& name, const void* src);
+    LayeredPlans& layered_plans(int rows);
+    // appends `rows` tokens at cache rows *kv_len + kv_off ...; the stream is left in x32_
+    template <typename T>
+    void layered_forward(int rows, const int32_t* ids, const int32_t* kv_len, int kv_off, cudaStream_t s);
+    template <typename T>
+    void layered_mixture(int layer, LayeredPlans& lp, cudaStream_t s);
+    // logits of n stream rows (rows_idx: device list, null = rows 0..n)
+    template <typename T>
+    void layered_logits(const int32_t* rows_idx, int n, void* out, cudaStream_t s);
+    void layered_prefill(int n, int history, const int32_t* ids, const int32_t* want, int n_want, void* logits_out);
+    void layered_decode(int n, const int32_t* ids, const int32_t* cache_length, void* logits_out, bool cuda_graph);
+    int layered_attn_splits(const LayerSpec& sp, int rows) const;
+    size_t elem_bytes() const { return mc_.fp32 ? 4 : 2; }
+    int ld() const { return pad64(mc_.hidden); }
 
     // ---- building blocks
     void build_layer_plans(LayerPlans& lp, const LayerWeights& w, const KVLayer& kv, int rows, int attn_splits);
@@ -214,6 +269,20 @@ private:
     void* argmax_ws_ = nullptr;
     bf16** d_cache_ptrs_ = nullptr;
     uint64_t* bm_capture_ = nullptr;
+    // ---- layered models
+    std::vector<LayeredWeights> lw_;
+    std::set<std::string> not_loaded_;                // tensors the configuration needs and load() has not seen
+    std::map<int, std::unique_ptr<LayeredPlans>> lplans_;
+    float* x32_ = nullptr;                            // [R][ld] residual stream
+    void *lx_ = nullptr, *lqkv_ = nullptr, *lq_ = nullptr, *lattn_ = nullptr, *ldelta_ = nullptr, *lnorm_ = nullptr;
+    void *moe_x_ = nullptr, *moe_gu_ = nullptr, *moe_act_ = nullptr, *moe_y_ = nullptr;
+    size_t moe_rows_ = 0;                             // rows of moe_x_ / moe_act_ / moe_y_
+    MoeBuffers moe_;
+    int32_t* want_ = nullptr;                         // [R] rows whose logits are asked for
+    float* layer_capture_ = nullptr;
+    cudaGraphExec_t decode_graph_ = nullptr;          // one-token decode for the pointers below
+    const void* decode_key_[3] = {nullptr, nullptr, nullptr};
+    long decode_launches_ = 0;
     SparseBuffers sp_;  // InfLLM-v2 compressed caches, scores and block masks (sparse target only)
     // device state words
     int32_t* st_ = nullptr;

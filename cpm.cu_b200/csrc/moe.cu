@@ -1,0 +1,636 @@
+// Mixture of experts for layered models (layered.cuh): fp32 router with grouped choice and identity experts, the layout
+// of the chosen rows, and the grouped expert products on the tensor cores.
+//
+//   route    fp32 logits (one warp per few outputs, rows staged in shared memory); the CTA counted last of a block of rows
+//            picks its rows' experts; the CTA counted last of the launch cuts every expert's rows into groups
+//   gather   each chosen row's input is copied to its place, expert after expert
+//   gate/up  grouped tcgen05 product, SwiGLU in the epilogue
+//   down     grouped tcgen05 product
+// The weighted sum over a token's experts, the identity part and the output norm are one kernel (out_norm_kernel).
+#include <algorithm>
+
+#include "gemm_common.cuh"
+#include "layered.cuh"
+#include "ptx.cuh"
+
+namespace {
+
+// ---------------------------------------------------------------- router
+constexpr int RT_WARPS = 8;
+constexpr int RT_KC = 1024;   // columns of x staged at a time
+
+struct RouteArgs {
+    const float* x;
+    const bf16* w;
+    const float* correction;
+    int rows, ld;
+    int outputs, experts, top, groups, keep;
+    float scale;
+    int tile, direct;
+    MoeBuffers b;
+};
+
+__device__ __forceinline__ void warp_argmax(float& v, int& i) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+        if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
+    }
+}
+
+// Largest of n values in shared memory, lowest index first among equals.
+__device__ __forceinline__ int argmax_of(const float* a, int n, int lane) {
+    float v = -INFINITY;
+    int i = 0x7fffffff;
+    for (int e = lane; e < n; e += 32) {
+        if (a[e] > v || i == 0x7fffffff) { v = a[e]; i = e; }
+    }
+    warp_argmax(v, i);
+    return i;
+}
+
+// The experts of one row, one warp.  sc: 2 * outputs + 2 * groups floats of scratch.
+__device__ void choose_experts(const RouteArgs& a, int row, float* sc, int lane) {
+    const int n = a.outputs;
+    float* score = sc;
+    float* choice = sc + n;
+    float* group = sc + 2 * n;
+    float* kept = group + a.groups;
+    const float* z = a.b.z + static_cast<size_t>(row) * n;
+    float m = -INFINITY;
+    for (int e = lane; e < n; e += 32) {
+        score[e] = __ldcg(z + e);
+        m = fmaxf(m, score[e]);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    float sum = 0.f;
+    for (int e = lane; e < n; e += 32) {
+        score[e] = expf(score[e] - m);
+        sum += score[e];
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    for (int e = lane; e < n; e += 32) {
+        score[e] = score[e] / sum;
+        choice[e] = a.correction != nullptr ? score[e] + a.correction[e] : score[e];
+    }
+    __syncwarp();
+    if (a.keep < a.groups) {
+        const int per = n / a.groups;
+        for (int g = lane; g < a.groups; g += 32) {
+            float v = choice[g * per];
+            for (int e = 1; e < per; ++e) v = fmaxf(v, choice[g * per + e]);
+            group[g] = v;
+            kept[g] = 0.f;
+        }
+        __syncwarp();
+        for (int k = 0; k < a.keep; ++k) {
+            const int g = argmax_of(group, a.groups, lane);
+            __syncwarp();
+            if (lane == 0) { kept[g] = 1.f; group[g] = -INFINITY; }
+            __syncwarp();
+        }
+        for (int e = lane; e < n; e += 32) {
+            if (kept[e / per] == 0.f) choice[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    int mine = -1;       // lane k holds choice k
+    float s_mine = 0.f;
+    for (int k = 0; k < a.top; ++k) {
+        const int e = argmax_of(choice, n, lane);
+        if (lane == k) { mine = e; s_mine = score[e]; }
+        __syncwarp();
+        if (lane == 0) choice[e] = -INFINITY;
+        __syncwarp();
+    }
+    float total = s_mine;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) total += __shfl_xor_sync(0xffffffffu, total, o);
+    const float weight = s_mine / (total + 1e-20f) * a.scale;
+    float idw = (mine >= a.experts) ? weight : 0.f;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) idw += __shfl_xor_sync(0xffffffffu, idw, o);
+    if (lane < a.top) {
+        const size_t i = static_cast<size_t>(row) * a.top + lane;
+        a.b.expert[i] = mine;
+        a.b.weight[i] = weight;
+        a.b.rank[i] = (mine < a.experts) ? atomicAdd(&a.b.counts[mine], 1) : 0;
+    }
+    if (lane == 0) a.b.id_weight[row] = idw;
+    __syncwarp();
+}
+
+// Rows of every expert one after the other, cut into groups of at most `tile` rows (as even as possible); one warp.
+__device__ void lay_out_rows(const RouteArgs& a, int lane) {
+    int row0 = 0, entry0 = 0;
+    for (int e0 = 0; e0 < a.experts; e0 += 32) {
+        const int e = e0 + lane;
+        const int cnt = (e < a.experts) ? __ldcg(&a.b.counts[e]) : 0;
+        const int ne = (cnt + a.tile - 1) / a.tile;
+        int rows_to = cnt, entries_to = ne;   // inclusive prefix sums
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int r = __shfl_up_sync(0xffffffffu, rows_to, o), n = __shfl_up_sync(0xffffffffu, entries_to, o);
+            if (lane >= o) { rows_to += r; entries_to += n; }
+        }
+        if (e < a.experts) {
+            const int first = row0 + rows_to - cnt;
+            a.b.offset[e] = first;
+            a.b.counts[e] = 0;
+            for (int k = 0; k < ne; ++k) {
+                const int b = static_cast<int>(static_cast<long long>(cnt) * k / ne), c = static_cast<int>(static_cast<long long>(cnt) * (k + 1) / ne);
+                const int at = entry0 + entries_to - ne + k;
+                if (at < kMoeMaxEntries) a.b.entries[at] = make_int4(e, a.direct ? 0 : first + b, first + b, c - b);
+            }
+        }
+        row0 += __shfl_sync(0xffffffffu, rows_to, 31);
+        entry0 += __shfl_sync(0xffffffffu, entries_to, 31);
+    }
+    if (lane == 0) *a.b.n_entries = min(entry0, kMoeMaxEntries);
+}
+
+// grid: (row blocks of RB, blocks of RT_WARPS * EPW outputs)
+template <int RB, int EPW>
+__global__ void __launch_bounds__(RT_WARPS * 32)
+moe_route_kernel(const RouteArgs a) {
+    grid_dep_trigger();
+    extern __shared__ float sm[];
+    __shared__ int s_last;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r0 = blockIdx.x * RB, nr = min(RB, a.rows - r0);
+    const int e0 = (blockIdx.y * RT_WARPS + warp) * EPW;
+    grid_dep_wait();
+    float acc[EPW][RB];
+#pragma unroll
+    for (int i = 0; i < EPW; ++i) {
+#pragma unroll
+        for (int r = 0; r < RB; ++r) acc[i][r] = 0.f;
+    }
+    for (int k0 = 0; k0 < a.ld; k0 += RT_KC) {
+        const int kn = min(RT_KC, a.ld - k0);   // a multiple of 64
+        __syncthreads();
+        for (int i = threadIdx.x * 4; i < RB * kn; i += RT_WARPS * 32 * 4) {
+            const int r = i / kn, c = i - r * kn;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (r < nr) v = *reinterpret_cast<const float4*>(a.x + static_cast<size_t>(r0 + r) * a.ld + k0 + c);
+            *reinterpret_cast<float4*>(sm + r * RT_KC + c) = v;
+        }
+        __syncthreads();
+        for (int c = lane * 4; c < kn; c += 128) {
+            float w[EPW][4];
+#pragma unroll
+            for (int i = 0; i < EPW; ++i) {
+                bf16 b[4] = {};
+                if (e0 + i < a.outputs) *reinterpret_cast<uint2*>(b) = *reinterpret_cast<const uint2*>(a.w + static_cast<size_t>(e0 + i) * a.ld + k0 + c);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) w[i][e] = __bfloat162float(b[e]);
+            }
+#pragma unroll
+            for (int r = 0; r < RB; ++r) {
+                const float4 x = *reinterpret_cast<const float4*>(sm + r * RT_KC + c);
+#pragma unroll
+                for (int i = 0; i < EPW; ++i) {
+                    acc[i][r] = fmaf(x.x, w[i][0], acc[i][r]);
+                    acc[i][r] = fmaf(x.y, w[i][1], acc[i][r]);
+                    acc[i][r] = fmaf(x.z, w[i][2], acc[i][r]);
+                    acc[i][r] = fmaf(x.w, w[i][3], acc[i][r]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < EPW; ++i) {
+#pragma unroll
+        for (int r = 0; r < RB; ++r) {
+            float v = acc[i][r];
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+            if (lane == 0 && r < nr && e0 + i < a.outputs) a.b.z[static_cast<size_t>(r0 + r) * a.outputs + e0 + i] = v;
+        }
+    }
+    // the CTA counted last of this block of rows chooses its experts
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int last = 1;
+        if (gridDim.y > 1) {
+            last = atomicAdd(&a.b.tickets[1 + blockIdx.x], 1) == static_cast<int>(gridDim.y) - 1;
+            if (last) a.b.tickets[1 + blockIdx.x] = 0;
+        }
+        s_last = last;
+    }
+    __syncthreads();
+    if (s_last == 0) return;
+    __threadfence();
+    const int per_warp = 2 * a.outputs + 2 * a.groups;
+    for (int r = warp; r < nr; r += RT_WARPS) choose_experts(a, r0 + r, sm + warp * per_warp, lane);
+    // the CTA counted last of the launch lays out the rows
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        const int last = atomicAdd(&a.b.tickets[0], 1) == static_cast<int>(gridDim.x) - 1;
+        if (last) a.b.tickets[0] = 0;
+        s_last = last;
+    }
+    __syncthreads();
+    if (s_last == 0) return;
+    __threadfence();
+    if (warp == 0) lay_out_rows(a, lane);
+}
+
+// One CTA per token row: its input goes to every chosen expert's slot.
+template <typename T>
+__global__ void moe_gather_kernel(const T* __restrict__ src, T* __restrict__ dst, const MoeBuffers b, int top, int experts, int ld) {
+    grid_dependency_sync();
+    __shared__ int slot[kMoeMaxTop];
+    if (threadIdx.x < top) {
+        const size_t i = static_cast<size_t>(blockIdx.x) * top + threadIdx.x;
+        const int e = b.expert[i];
+        slot[threadIdx.x] = e < experts ? b.offset[e] + b.rank[i] : -1;
+    }
+    __syncthreads();
+    const int n16 = ld * static_cast<int>(sizeof(T)) / 16;
+    const uint4* s = reinterpret_cast<const uint4*>(src + static_cast<size_t>(blockIdx.x) * ld);
+    for (int c = threadIdx.x; c < n16; c += blockDim.x) {
+        const uint4 v = s[c];
+        for (int k = 0; k < top; ++k) {
+            if (slot[k] >= 0) reinterpret_cast<uint4*>(dst + static_cast<size_t>(slot[k]) * ld)[c] = v;
+        }
+    }
+}
+
+// ---------------------------------------------------------------- grouped products
+constexpr int BLOCK_K = 64;
+constexpr int UMMA_K = 16;
+constexpr int W_TILE_BYTES = gemm::BLOCK_N * BLOCK_K * 2;
+constexpr int NUM_THREADS = 192;   // warp 0 TMA, warp 1 MMA + TMEM, warps 2-5 epilogue
+
+template <int MT>
+struct Cfg {
+    static constexpr int STAGE_BYTES = W_TILE_BYTES + MT * BLOCK_K * 2;
+    static constexpr int STAGES = (MT <= 16) ? 10 : (MT <= 32) ? 9 : (MT <= 64) ? 8 : (MT <= 128) ? 6 : 4;
+    static constexpr int TMEM_COLS = (2 * MT < 32) ? 32 : 2 * MT;
+    static constexpr int CTRL_BYTES = 256;
+    static constexpr int ENTRY_BYTES = 16 * kMoeMaxEntries;
+    static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + CTRL_BYTES + gemm::SWIGLU_XCH_BYTES + ENTRY_BYTES + 1024;
+    static_assert(SMEM_BYTES <= 232448, "shared memory budget");
+};
+
+struct GemmArgs {
+    int n_tiles, kblocks, N;
+    int n_tiles_s, kblocks_s, N_s;
+    int groups_s;          // row groups of the shared expert (all tokens)
+    int rows;              // tokens
+    int tile;
+    long long w_row_s;
+    int xs_row0, ys_row0;
+    bf16* y;
+    int ldy;
+    const int4* entries;
+    const int32_t* n_entries;
+    int* error;
+};
+
+// Output tile t: the shared expert's tiles come first, then the experts' row groups; the feature tile runs fastest, so
+// CTAs of a wave share a group's rows and its expert's matrix passes through L2 once for all of the expert's groups.
+struct TileJob {
+    bool shared;
+    int n_tile, kblocks, N;
+    int w_row;             // first row of the weight tile in the weight map (without the k-block)
+    int x_row, y_row, rows;
+};
+
+template <bool SWIGLU>
+__device__ __forceinline__ TileJob tile_job(const GemmArgs& a, const int4* entries, int t) {
+    TileJob j;
+    const int ts = a.groups_s * a.n_tiles_s;
+    if (t < ts) {
+        const int g = t / a.n_tiles_s;
+        j.shared = true;
+        j.n_tile = t - g * a.n_tiles_s;
+        j.kblocks = a.kblocks_s;
+        j.N = a.N_s;
+        j.w_row = static_cast<int>(a.w_row_s) + j.n_tile * a.kblocks_s * gemm::BLOCK_N;
+        j.x_row = a.xs_row0 + g * a.tile;
+        j.y_row = a.ys_row0 + g * a.tile;
+        j.rows = min(a.tile, a.rows - g * a.tile);
+    } else {
+        const int g = (t - ts) / a.n_tiles;
+        const int4 e = entries[g];
+        j.shared = false;
+        j.n_tile = (t - ts) - g * a.n_tiles;
+        j.kblocks = a.kblocks;
+        j.N = a.N;
+        j.w_row = (e.x * a.n_tiles + j.n_tile) * a.kblocks * gemm::BLOCK_N;
+        j.x_row = SWIGLU ? e.y : e.z;   // the down product reads the rows gate/up wrote
+        j.y_row = e.z;
+        j.rows = e.w;
+    }
+    return j;
+}
+
+template <int MT, bool SWIGLU>
+__global__ void __launch_bounds__(NUM_THREADS, 1)
+moe_gemm_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x,
+                     const __grid_constant__ CUtensorMap tm_xs, const GemmArgs a) {
+    using C = Cfg<MT>;
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    uint8_t* tiles = smem;
+    uint64_t* full = reinterpret_cast<uint64_t*>(smem + C::STAGES * C::STAGE_BYTES);
+    uint64_t* empty = full + C::STAGES;
+    uint64_t* acc_full = empty + C::STAGES;
+    uint64_t* acc_empty = acc_full + 2;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+    float* xch = reinterpret_cast<float*>(smem + C::STAGES * C::STAGE_BYTES + C::CTRL_BYTES);
+    int4* entries = reinterpret_cast<int4*>(smem + C::STAGES * C::STAGE_BYTES + C::CTRL_BYTES + gemm::SWIGLU_XCH_BYTES);
+
+    const int warp = threadIdx.x >> 5;
+    const int lane = threadIdx.x & 31;
+    grid_dep_trigger();
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < C::STAGES; ++s) {
+            ptx::mbar_init(&full[s], 1);
+            ptx::mbar_init(&empty[s], 1);
+        }
+        for (int s = 0; s < 2; ++s) {
+            ptx::mbar_init(&acc_full[s], 1);
+            ptx::mbar_init(&acc_empty[s], 128);
+        }
+        *abort_flag = 0;
+        ptx::mbar_fence_init();
+        ptx::prefetch_tensormap(&tm_w);
+        ptx::prefetch_tensormap(&tm_x);
+        ptx::prefetch_tensormap(&tm_xs);
+    }
+    if (warp == 1) {
+        ptx::tmem_alloc(tmem_slot, C::TMEM_COLS);
+        ptx::tmem_relinquish();
+    }
+    grid_dep_wait();   // the row groups come from the router
+    const int n_entries = min(*a.n_entries, kMoeMaxEntries);
+    for (int i = threadIdx.x; i < n_entries; i += NUM_THREADS) entries[i] = a.entries[i];
+    ptx::tc_fence_before();
+    __syncthreads();
+    ptx::tc_fence_after();
+    const uint32_t tmem_base = *tmem_slot;
+    const int total = a.groups_s * a.n_tiles_s + n_entries * a.n_tiles;
+
+    if (warp == 0) {
+        // ------------------------------------------------ TMA producer
+        if (lane == 0) {
+            int stage = 0;
+            uint32_t phase = 0;
+            bool ok = true;
+            for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
+                const TileJob j = tile_job<SWIGLU>(a, entries, t);
+                for (int kb = 0; kb < j.kblocks; ++kb) {
+                    if (!ptx::mbar_wait(&empty[stage], phase ^ 1, abort_flag)) { ok = false; break; }
+                    uint8_t* dst = tiles + stage * C::STAGE_BYTES;
+                    ptx::mbar_arrive_expect_tx(&full[stage], C::STAGE_BYTES);
+                    ptx::tma_load_2d(dst, &tm_w, &full[stage], 0, j.w_row + kb * gemm::BLOCK_N);
+                    ptx::tma_load_2d(dst + W_TILE_BYTES, j.shared ? &tm_xs : &tm_x, &full[stage], kb * BLOCK_K, j.x_row);
+                    if (++stage == C::STAGES) { stage = 0; phase ^= 1; }
+                }
+            }
+            if (!ok) {
+                // give copies already in flight time to land before the CTA retires
+                const long long t0 = clock64();
+                while (clock64() - t0 < 2000000LL) {}
+            }
+        }
+    } else if (warp == 1) {
+        // ------------------------------------------------ MMA issuer
+        if (lane == 0) {
+            int stage = 0;
+            uint32_t phase = 0;
+            int acc = 0;
+            uint32_t acc_phase = 0;
+            bool ok = true;
+            for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
+                const TileJob j = tile_job<SWIGLU>(a, entries, t);
+                // a group that is not full costs only its rows (rounded up to 16)
+                const int n_mma = min(MT, (j.rows + 15) & ~15);
+                const uint32_t idesc = ptx::umma_idesc_bf16(gemm::BLOCK_N, n_mma, 0, 0);
+                if (!ptx::mbar_wait(&acc_empty[acc], acc_phase ^ 1, abort_flag)) break;
+                ptx::tc_fence_after();
+                const uint32_t d_tmem = tmem_base + acc * MT;
+                for (int kb = 0; kb < j.kblocks; ++kb) {
+                    if (!ptx::mbar_wait(&full[stage], phase, abort_flag)) { ok = false; break; }
+                    ptx::tc_fence_after();
+                    const uint32_t wa = ptx::smem_u32(tiles + stage * C::STAGE_BYTES);
+                    const uint32_t xa = wa + W_TILE_BYTES;
+#pragma unroll
+                    for (int k = 0; k < BLOCK_K / UMMA_K; ++k) {
+                        const uint64_t da = ptx::umma_desc_sw128(wa + k * UMMA_K * 2, 16, 1024);
+                        const uint64_t db = ptx::umma_desc_sw128(xa + k * UMMA_K * 2, 16, 1024);
+                        ptx::umma_ss(d_tmem, da, db, idesc, (kb > 0 || k > 0) ? 1u : 0u);
+                    }
+                    ptx::umma_commit(&empty[stage]);
+                    if (++stage == C::STAGES) { stage = 0; phase ^= 1; }
+                }
+                if (!ok) break;
+                ptx::umma_commit(&acc_full[acc]);
+                acc ^= 1;
+                if (acc == 0) acc_phase ^= 1;
+            }
+        }
+    } else {
+        // ------------------------------------------------ epilogue (128 threads; lane = feature, column = row of the group)
+        const int q = warp & 3;
+        const int row = q * 32 + lane;
+        int acc = 0, xi = 0;
+        uint32_t acc_phase = 0;
+        for (int t = blockIdx.x; t < total; t += gridDim.x) {
+            const TileJob j = tile_job<SWIGLU>(a, entries, t);
+            const int n = SWIGLU ? j.n_tile * 64 + (row & 63) : j.n_tile * gemm::BLOCK_N + row;
+            if (!ptx::mbar_wait_warp(&acc_full[acc], acc_phase, abort_flag)) break;
+            ptx::tc_fence_after();
+            const uint32_t t_addr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + acc * MT;
+#pragma unroll 1
+            for (int c0 = 0; c0 < MT; c0 += 16) {
+                if (c0 >= j.rows) break;   // uniform across the CTA
+                uint32_t r[16];
+                ptx::tmem_ld16(t_addr + c0, r);
+                ptx::tmem_wait_ld();
+                bf16* y = a.y + static_cast<size_t>(j.y_row + c0) * a.ldy + n;
+                if constexpr (SWIGLU) {
+                    // lanes 0-63 hold the gate projection, lanes 64-127 the up projection of the same 64 features; the gate
+                    // values pass through one of two shared-memory buffers to the warps of the up half, which store
+                    float* xb = xch + (xi & 1) * (2 * 16 * 32);
+                    ++xi;
+                    if (q < 2) {
+#pragma unroll
+                        for (int c = 0; c < 16; ++c) xb[(q * 16 + c) * 32 + lane] = __bfloat162float(__float2bfloat16(__uint_as_float(r[c])));
+                    }
+                    // a buffer is written again two batches later, past the next batch's barrier
+                    ptx::named_bar_sync(1, 128);
+                    if (q >= 2 && n < j.N) {
+#pragma unroll
+                        for (int c = 0; c < 16; ++c) {
+                            if (c0 + c < j.rows) {
+                                const float uv = __bfloat162float(__float2bfloat16(__uint_as_float(r[c])));
+                                y[static_cast<size_t>(c) * a.ldy] = __float2bfloat16(silu_mul(xb[((q - 2) * 16 + c) * 32 + lane], uv));
+                            }
+                        }
+                    }
+                } else if (n < j.N) {
+#pragma unroll
+                    for (int c = 0; c < 16; ++c) {
+                        if (c0 + c < j.rows) y[static_cast<size_t>(c) * a.ldy] = __float2bfloat16(__uint_as_float(r[c]));
+                    }
+                }
+            }
+            ptx::tc_fence_before();
+            ptx::mbar_arrive(&acc_empty[acc]);
+            if (++acc == 2) { acc = 0; acc_phase ^= 1; }
+        }
+    }
+
+    ptx::tc_fence_before();
+    __syncthreads();
+    if (warp == 1) {
+        ptx::tc_fence_after();
+        ptx::tmem_dealloc(tmem_base, C::TMEM_COLS);
+    }
+    if (threadIdx.x == 0 && *abort_flag) atomicOr(a.error, ERR_GEMM_TIMEOUT);
+}
+
+template <int MT, bool SWIGLU>
+void launch_gemm(const MoeGemmPlan& p, const GemmArgs& a, int grid, cudaStream_t s) {
+    static bool configured = false;
+    if (!configured) {
+        CUDA_CHECK(cudaFuncSetAttribute(moe_gemm_umma_kernel<MT, SWIGLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<MT>::SMEM_BYTES));
+        configured = true;
+    }
+    launch_kernel(moe_gemm_umma_kernel<MT, SWIGLU>, dim3(grid), dim3(NUM_THREADS), Cfg<MT>::SMEM_BYTES, s, p.tm_w, p.tm_x, p.tm_xs, a);
+}
+
+CUtensorMap weight_map(const bf16* w, size_t elems) { return make_tmap_2d(w, BLOCK_K, elems / BLOCK_K, BLOCK_K * 2, BLOCK_K, gemm::BLOCK_N); }
+
+}  // namespace
+
+size_t moe_ticket_ints(int max_rows) { return 1 + static_cast<size_t>(max_rows); }
+
+int moe_pick_tile(const LayerSpec& sp, int rows) {
+    // tokens of one expert: the average with some room for uneven choices, never more than all
+    const long long avg = (static_cast<long long>(rows) * sp.top * 5 / 4 + sp.experts + sp.identity - 1) / (sp.experts + sp.identity);
+    int tile = 16;
+    while (tile < 256 && tile < std::min<long long>(avg, rows)) tile *= 2;
+    while (tile < 256 && moe_max_entries(sp, rows, tile) > kMoeMaxEntries) tile *= 2;
+    return tile;
+}
+
+int moe_max_entries(const LayerSpec& sp, int rows, int tile) {
+    const long long slots = static_cast<long long>(rows) * std::min(sp.top, sp.experts);
+    return static_cast<int>(std::min<long long>(slots, slots / tile + sp.experts));
+}
+
+void launch_moe_route(const LayerSpec& sp, const float* x32, const bf16* w, const float* correction, const MoeBuffers& b, int rows,
+                      int ld, int tile, bool direct, cudaStream_t s) {
+    ProfileScope prof(KC_ROUTE, s);
+    RouteArgs a;
+    a.x = x32; a.w = w; a.correction = correction;
+    a.rows = rows; a.ld = ld;
+    a.outputs = sp.experts + sp.identity; a.experts = sp.experts; a.top = sp.top;
+    a.groups = sp.groups; a.keep = sp.keep_groups;
+    a.scale = sp.router_scale;
+    a.tile = tile; a.direct = direct ? 1 : 0;
+    a.b = b;
+    CPM_REQUIRE(moe_max_entries(sp, rows, tile) <= kMoeMaxEntries, "mixture of experts: too many row groups");
+    const size_t choose = static_cast<size_t>(RT_WARPS) * (2 * a.outputs + 2 * a.groups) * sizeof(float);
+    auto run = [&](auto kernel, int rb, int epw, bool& configured) {
+        const size_t smem = std::max<size_t>(choose, static_cast<size_t>(rb) * RT_KC * sizeof(float));
+        if (!configured) {
+            CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, RT_WARPS * 4 * kMoeMaxOutputs * 4));
+            configured = true;
+        }
+        launch_kernel(kernel, dim3(ceil_div(rows, rb), ceil_div(a.outputs, RT_WARPS * epw)), dim3(RT_WARPS * 32), smem, s, a);
+    };
+    static bool c1 = false, c8 = false;
+    if (rows <= 16) run(moe_route_kernel<1, 1>, 1, 1, c1);
+    else run(moe_route_kernel<8, 4>, 8, 4, c8);
+}
+
+template <typename T>
+void launch_moe_gather(const LayerSpec& sp, const T* src, T* dst, const MoeBuffers& b, int rows, int ld, cudaStream_t s) {
+    ProfileScope prof(KC_ROUTE, s);
+    launch_kernel(moe_gather_kernel<T>, dim3(rows), dim3(256), 0, s, src, dst, b, sp.top, sp.experts, ld);
+}
+template void launch_moe_gather<bf16>(const LayerSpec&, const bf16*, bf16*, const MoeBuffers&, int, int, cudaStream_t);
+template void launch_moe_gather<float>(const LayerSpec&, const float*, float*, const MoeBuffers&, int, int, cudaStream_t);
+
+size_t moe_gate_up_offset(const LayerSpec& sp, int K, int expert) { return static_cast<size_t>(expert) * 2 * pad64(sp.expert_ff) * K; }
+size_t moe_gate_up_elems(const LayerSpec& sp, int K) { return moe_gate_up_offset(sp, K, sp.experts) + static_cast<size_t>(2) * pad64(sp.shared_ff) * K; }
+size_t moe_down_offset(const LayerSpec& sp, int width, int expert) { return static_cast<size_t>(expert) * linear_weight_elems(width, pad64(sp.expert_ff)); }
+size_t moe_down_elems(const LayerSpec& sp, int width) { return moe_down_offset(sp, width, sp.experts) + linear_weight_elems(width, pad64(sp.shared_ff)); }
+
+MoeGemmPlan make_moe_gate_up_plan(const LayerSpec& sp, const bf16* w, const bf16* x, int x_rows, const bf16* xs, int K, bf16* act,
+                                  int ld_act, int rows, int tile, const MoeBuffers& b) {
+    CPM_REQUIRE(K % BLOCK_K == 0 && ld_act % BLOCK_K == 0, "mixture of experts: padded widths must be multiples of 64");
+    MoeGemmPlan p;
+    const int ff = pad64(sp.expert_ff), ffs = pad64(sp.shared_ff);
+    p.tm_w = weight_map(w, moe_gate_up_elems(sp, K));
+    p.tm_x = make_tmap_2d(x, K, x_rows, static_cast<uint64_t>(K) * 2, BLOCK_K, tile);
+    p.tm_xs = make_tmap_2d(xs, K, rows, static_cast<uint64_t>(K) * 2, BLOCK_K, tile);
+    p.tile = tile; p.rows = rows; p.max_entries = moe_max_entries(sp, rows, tile);
+    p.swiglu = 1;
+    p.n_tiles = ff / 64; p.kblocks = K / BLOCK_K; p.N = ff;
+    p.n_tiles_s = ffs / 64; p.kblocks_s = p.kblocks; p.N_s = ffs;
+    p.w_row_s = static_cast<long long>(moe_gate_up_offset(sp, K, sp.experts) / BLOCK_K);
+    p.xs_row0 = 0; p.ys_row0 = rows * sp.top;
+    p.y = act; p.ldy = ld_act;
+    p.entries = b.entries; p.n_entries = b.n_entries;
+    return p;
+}
+
+MoeGemmPlan make_moe_down_plan(const LayerSpec& sp, const bf16* w, const bf16* act, int act_rows, int ld_act, int width, bf16* y,
+                               int ld_y, int rows, int tile, const MoeBuffers& b) {
+    CPM_REQUIRE(ld_act % BLOCK_K == 0, "mixture of experts: padded widths must be multiples of 64");
+    MoeGemmPlan p;
+    const int ff = pad64(sp.expert_ff), ffs = pad64(sp.shared_ff);
+    p.tm_w = weight_map(w, moe_down_elems(sp, width));
+    p.tm_x = make_tmap_2d(act, ld_act, act_rows, static_cast<uint64_t>(ld_act) * 2, BLOCK_K, tile);
+    p.tm_xs = p.tm_x;
+    p.tile = tile; p.rows = rows; p.max_entries = moe_max_entries(sp, rows, tile);
+    p.n_tiles = ceil_div(width, gemm::BLOCK_N); p.kblocks = ff / BLOCK_K; p.N = width;
+    p.n_tiles_s = ffs > 0 ? p.n_tiles : 0; p.kblocks_s = ffs / BLOCK_K; p.N_s = width;
+    p.w_row_s = static_cast<long long>(moe_down_offset(sp, width, sp.experts) / BLOCK_K);
+    p.xs_row0 = p.ys_row0 = rows * sp.top;
+    p.y = y; p.ldy = ld_y;
+    p.entries = b.entries; p.n_entries = b.n_entries;
+    return p;
+}
+
+void launch_moe_gemm(const MoeGemmPlan& p, cudaStream_t s) {
+    ProfileScope prof(KC_MOE, s);
+    GemmArgs a;
+    a.n_tiles = p.n_tiles; a.kblocks = p.kblocks; a.N = p.N;
+    a.n_tiles_s = p.n_tiles_s; a.kblocks_s = p.kblocks_s; a.N_s = p.N_s;
+    a.groups_s = p.n_tiles_s > 0 ? ceil_div(p.rows, p.tile) : 0;
+    if (a.n_tiles_s == 0) a.n_tiles_s = 1;   // a divisor only
+    a.rows = p.rows; a.tile = p.tile;
+    a.w_row_s = p.w_row_s; a.xs_row0 = p.xs_row0; a.ys_row0 = p.ys_row0;
+    a.y = p.y; a.ldy = p.ldy;
+    a.entries = p.entries; a.n_entries = p.n_entries;
+    a.error = runtime().d_error;
+    const long long most = static_cast<long long>(a.groups_s) * a.n_tiles_s + static_cast<long long>(p.max_entries) * p.n_tiles;
+    const int grid = static_cast<int>(std::max<long long>(1, std::min<long long>(most, runtime().num_sms)));
+    switch (p.tile * 2 + p.swiglu) {
+        case 16 * 2: launch_gemm<16, false>(p, a, grid, s); break;
+        case 16 * 2 + 1: launch_gemm<16, true>(p, a, grid, s); break;
+        case 32 * 2: launch_gemm<32, false>(p, a, grid, s); break;
+        case 32 * 2 + 1: launch_gemm<32, true>(p, a, grid, s); break;
+        case 64 * 2: launch_gemm<64, false>(p, a, grid, s); break;
+        case 64 * 2 + 1: launch_gemm<64, true>(p, a, grid, s); break;
+        case 128 * 2: launch_gemm<128, false>(p, a, grid, s); break;
+        case 128 * 2 + 1: launch_gemm<128, true>(p, a, grid, s); break;
+        case 256 * 2: launch_gemm<256, false>(p, a, grid, s); break;
+        case 256 * 2 + 1: launch_gemm<256, true>(p, a, grid, s); break;
+        default: throw std::invalid_argument("cpmcu_b200: bad row group size");
+    }
+}

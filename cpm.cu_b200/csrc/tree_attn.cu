@@ -26,8 +26,14 @@
 // gridDim.y key splits each write an unnormalised partial (O, max, sum); a
 // small second kernel merges them.  With one split the kernel normalises and
 // stores bf16 directly.
+//
+// Layers of layered models (LayerSpec) run the BIASED instantiations: key and value widths of 64 or 128 columns, a
+// sliding window that is exact per token (exact_window: token at position i sees j with 0 <= i - j < exact_window) and a
+// distance bias, score = scale * (q . k) - slope_h * (i - j), slope_h = 2^(-bias_exp * (h + 1) / hq).
 #include <algorithm>
 #include <cstdio>
+#include <cstring>
+#include <type_traits>
 #include <vector>
 
 #include "common.cuh"
@@ -35,19 +41,22 @@
 
 namespace {
 
-constexpr int D = 128;          // head dim
 constexpr int ROWS = 128;       // query rows per tile (UMMA M)
 constexpr int KEYS = 128;       // keys per tile
-constexpr int HALF_BYTES = ROWS * 128;        // one 64-column half: 128 rows x 128 B
-constexpr int TILE_BYTES = 2 * HALF_BYTES;    // 32 KB
-constexpr int SMEM_Q = 0;
-constexpr int SMEM_K = SMEM_Q + TILE_BYTES;          // 2 stages
-constexpr int SMEM_V = SMEM_K + 2 * TILE_BYTES;      // 2 stages
-constexpr int SMEM_P = SMEM_V + 2 * TILE_BYTES;      // 2 stages
-constexpr int SMEM_CTRL = SMEM_P + 2 * TILE_BYTES;
-constexpr int SMEM_UNION = SMEM_CTRL + 128;  // 256 B: bitmask over up to 2048 key tiles (block-sparse mode)
-constexpr int SMEM_XCH = SMEM_CTRL + 512;   // 2 x 128 floats
-constexpr int SMEM_TOTAL = SMEM_XCH + 1024 + 1024;
+constexpr int HALF_BYTES = ROWS * 128;        // 64 columns of a tile: 128 rows x 128 B
+// DK, DV: columns of a query / key row and of a value row of one head in memory, 64 or 128
+template <int DK, int DV>
+struct AttnCfg {
+    static constexpr int K_TILE = KEYS * DK * 2, V_TILE = KEYS * DV * 2, P_TILE = ROWS * KEYS * 2;
+    static constexpr int SMEM_Q = 0;
+    static constexpr int SMEM_K = SMEM_Q + ROWS * DK * 2;        // 2 stages
+    static constexpr int SMEM_V = SMEM_K + 2 * K_TILE;           // 2 stages
+    static constexpr int SMEM_P = SMEM_V + 2 * V_TILE;           // 2 stages
+    static constexpr int SMEM_CTRL = SMEM_P + 2 * P_TILE;
+    static constexpr int SMEM_UNION = SMEM_CTRL + 128;  // 256 B: bitmask over up to 2048 key tiles (block-sparse mode)
+    static constexpr int SMEM_XCH = SMEM_CTRL + 512;    // 2 x 128 floats
+    static constexpr int SMEM_TOTAL = SMEM_XCH + 1024 + 1024;
+};
 constexpr int TMEM_COLS = 512;  // S stage 0: [0,128), S stage 1: [128,256), O: [256,384)
 constexpr int TMEM_O = 256;
 constexpr int SOFTMAX_THREADS = 256;  // two threads per query row: warps 0-3 keys 0-63 of a tile, warps 4-7 keys 64-127
@@ -62,6 +71,9 @@ struct AttnArgs {
     const uint64_t* mask;
     int mask_k;
     int window;
+    int exact_window;    // > 0: per-token sliding window (tokens); BIASED instantiations only
+    float bias_exp;      // > 0: distance bias with slopes 2^(-bias_exp * (h + 1) / hq); BIASED instantiations only
+    int out_cols;        // value columns that are stored per head (the rest of DV is padding)
     const uint64_t* blockmask;  // [hkv][tq][bm_words] bits over 64-key blocks, or null
     int bm_words, block_window;
     float scale_log2;
@@ -90,12 +102,14 @@ __device__ __forceinline__ float fast_exp2(float x) {
 // ahead: S(i+1) = Q K(i+1)^T is already in TMEM (two S stages) while the softmax warps work
 // on tile i, and O += P(i) V(i) is issued as soon as P(i) is in shared memory (two P stages),
 // so in steady state an iteration costs one softmax pass.
+template <int DK, int DV, bool BIASED>
 __global__ void __launch_bounds__(NTHREADS, 1)
 tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                  const __grid_constant__ CUtensorMap tm_v, const AttnArgs a) {
+    using C = AttnCfg<DK, DV>;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + SMEM_CTRL);
+    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + C::SMEM_CTRL);
     uint64_t* q_bar = bars;
     uint64_t* k_full = bars + 1;   // [2]
     uint64_t* v_full = bars + 3;   // [2]
@@ -104,7 +118,7 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
     uint64_t* p_ready = bars + 9;  // [2]  P(i) is in shared memory (256 arrivals)
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 11);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-    float* xch = reinterpret_cast<float*>(smem + SMEM_XCH);  // [2][128] row maxima / sums of the two column halves
+    float* xch = reinterpret_cast<float*>(smem + C::SMEM_XCH);  // [2][128] row maxima / sums of the two column halves
 
     const long long pt_kernel = prof_clock();
     const int tid = threadIdx.x;
@@ -144,7 +158,7 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
     ptx::tc_fence_after();
     const uint32_t tmem_base = *tmem_slot;
     const uint32_t lane_sel = static_cast<uint32_t>((warp & 3) * 32) << 16;
-    const uint32_t tmem_o = tmem_base + lane_sel + TMEM_O + ch * 64;  // this thread's 64 output columns
+    const uint32_t tmem_o = tmem_base + lane_sel + TMEM_O + ch * (DV / 2);  // this thread's half of the output columns
     grid_dep_wait();  // everything above overlaps the previous kernel's tail
     const long long pt_dep = prof_clock();
 
@@ -154,7 +168,8 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
     const int t0 = mt * a.tok_per_tile;
     const int t = t0 + row / a.grp;          // query token of this thread's row
     const int qh = h * a.grp + row % a.grp;  // query head of this thread's row
-    const bool row_valid = (t < tq_eff);
+    const bool row_in = !BIASED || row < a.grp * a.tok_per_tile;   // 128 need not be a multiple of grp
+    const bool row_valid = row_in && (t < tq_eff);
     const int causal_base = kv_total - tq_eff;  // token t sees keys < causal_base + t + 1
     int limit = row_valid ? min(kv_total, causal_base + t + 1) : 0;
     if (limit < 0) limit = 0;
@@ -173,6 +188,14 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
         const int lo_blk = (q0 + KEYS - 1) / KEYS - a.window / KEYS;
         if (lo_blk > 0) key_lo = lo_blk * KEYS;
     }
+    int row_lo = key_lo;  // first key this row may see
+    if (BIASED && a.exact_window > 0) {
+        row_lo = max(causal_base + t - a.exact_window + 1, 0);
+        key_lo = max(causal_base + t0 - a.exact_window + 1, 0);
+    }
+    const float slope2 =   // log2(e) * slope of this row's head
+        (BIASED && a.bias_exp > 0.f) ? 1.4426950408889634f * exp2f(-a.bias_exp * static_cast<float>(qh + 1) / static_cast<float>(a.hq)) : 0.f;
+    const float sl2 = BIASED ? 1.f : a.scale_log2;   // biased scores are brought to log2 units as they are read
     const int kt_lo = key_lo / KEYS;
     const int kt_hi = (key_hi + KEYS - 1) / KEYS;
     const int n_kt = max(kt_hi - kt_lo, 0);
@@ -182,7 +205,7 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
 
     // ---- block-sparse mode: union of the tile's tokens' blocks, then this split's share of the set tiles
     const bool sparse = (a.blockmask != nullptr);
-    uint32_t* uni = reinterpret_cast<uint32_t*>(smem + SMEM_UNION);       // 64 words = 2048 key tiles
+    uint32_t* uni = reinterpret_cast<uint32_t*>(smem + C::SMEM_UNION);       // 64 words = 2048 key tiles
     volatile int* sp_info = reinterpret_cast<volatile int*>(abort_flag + 1);  // [0] first tile, [1] count
     // this row's token: first 64-key block always visible, and its mask row
     const int win_left = sparse ? (t + causal_base + 63) / 64 - a.block_window : 0;
@@ -244,32 +267,36 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
     if (is_control) {
         // ================================================= control warp: TMA + MMA issue
         if (lane == 0 && n_it > 0) {
-            const uint32_t q_addr = ptx::smem_u32(smem + SMEM_Q);
-            const uint32_t p_addr = ptx::smem_u32(smem + SMEM_P);
+            const uint32_t q_addr = ptx::smem_u32(smem + C::SMEM_Q);
+            const uint32_t p_addr = ptx::smem_u32(smem + C::SMEM_P);
             constexpr uint32_t idesc_s = ptx::umma_idesc_bf16(ROWS, KEYS, 0, 0);
-            constexpr uint32_t idesc_o = ptx::umma_idesc_bf16(ROWS, D, 0, 1);
+            constexpr uint32_t idesc_o = ptx::umma_idesc_bf16(ROWS, DV, 0, 1);
             int k_tile = kt_begin, v_tile = kt_begin;  // tiles of the next K / V load (issued in iteration order)
             auto load_k = [&](int i) {
                 const int st = i & 1, key0 = k_tile * KEYS;
                 k_tile = next_tile(k_tile);
-                ptx::mbar_arrive_expect_tx(&k_full[st], TILE_BYTES);
-                ptx::tma_load_2d(smem + SMEM_K + st * TILE_BYTES, &tm_k, &k_full[st], h * D, key0);
-                ptx::tma_load_2d(smem + SMEM_K + st * TILE_BYTES + HALF_BYTES, &tm_k, &k_full[st], h * D + 64, key0);
+                ptx::mbar_arrive_expect_tx(&k_full[st], C::K_TILE);
+#pragma unroll
+                for (int c = 0; c < DK / 64; ++c) {
+                    ptx::tma_load_2d(smem + C::SMEM_K + st * C::K_TILE + c * HALF_BYTES, &tm_k, &k_full[st], h * DK + c * 64, key0);
+                }
             };
             auto load_v = [&](int i) {
                 const int st = i & 1, key0 = v_tile * KEYS;
                 v_tile = next_tile(v_tile);
-                ptx::mbar_arrive_expect_tx(&v_full[st], TILE_BYTES);
-                ptx::tma_load_2d(smem + SMEM_V + st * TILE_BYTES, &tm_v, &v_full[st], h * D, key0);
-                ptx::tma_load_2d(smem + SMEM_V + st * TILE_BYTES + HALF_BYTES, &tm_v, &v_full[st], h * D + 64, key0);
+                ptx::mbar_arrive_expect_tx(&v_full[st], C::V_TILE);
+#pragma unroll
+                for (int c = 0; c < DV / 64; ++c) {
+                    ptx::tma_load_2d(smem + C::SMEM_V + st * C::V_TILE + c * HALF_BYTES, &tm_v, &v_full[st], h * DV + c * 64, key0);
+                }
             };
             auto issue_s = [&](int i) -> bool {  // S(i) = Q K(i)^T into S stage i & 1
                 const int st = i & 1;
                 if (!ptx::mbar_wait(&k_full[st], (i >> 1) & 1, abort_flag)) return false;
                 ptx::tc_fence_after();
-                const uint32_t k_addr = ptx::smem_u32(smem + SMEM_K + st * TILE_BYTES);
+                const uint32_t k_addr = ptx::smem_u32(smem + C::SMEM_K + st * C::K_TILE);
 #pragma unroll
-                for (int dh = 0; dh < 2; ++dh) {
+                for (int dh = 0; dh < DK / 64; ++dh) {
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         const uint64_t da = ptx::umma_desc_sw128(q_addr + dh * HALF_BYTES + j * 32, 16, 1024);
@@ -280,9 +307,12 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
                 ptx::umma_commit(&s_bar[st]);
                 return true;
             };
-            ptx::mbar_arrive_expect_tx(q_bar, TILE_BYTES);
-            ptx::tma_load_3d(smem + SMEM_Q, &tm_q, q_bar, 0, h * a.grp, t0);
-            ptx::tma_load_3d(smem + SMEM_Q + HALF_BYTES, &tm_q, q_bar, 64, h * a.grp, t0);
+            // rows of the tile beyond grp * tok_per_tile keep whatever shared memory held; nothing of them is stored
+            ptx::mbar_arrive_expect_tx(q_bar, a.grp * a.tok_per_tile * DK * 2);
+#pragma unroll
+            for (int c = 0; c < DK / 64; ++c) {
+                ptx::tma_load_3d(smem + C::SMEM_Q + c * HALF_BYTES, &tm_q, q_bar, c * 64, h * a.grp, t0);
+            }
             for (int i = 0; i < 2 && i < n_it; ++i) {
                 load_k(i);
                 load_v(i);
@@ -301,8 +331,8 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
                 if (!ptx::mbar_wait(&p_ready[st], ph, abort_flag)) { w = false; break; }
                 if (!ptx::mbar_wait(&v_full[st], ph, abort_flag)) { w = false; break; }
                 ptx::tc_fence_after();
-                const uint32_t v_addr = ptx::smem_u32(smem + SMEM_V + st * TILE_BYTES);
-                const uint32_t pa = p_addr + st * TILE_BYTES;
+                const uint32_t v_addr = ptx::smem_u32(smem + C::SMEM_V + st * C::V_TILE);
+                const uint32_t pa = p_addr + st * C::P_TILE;
 #pragma unroll
                 for (int kk = 0; kk < KEYS / 16; ++kk) {
                     // A: P, K-major: 64-key half (kk / 4), 32 B per 16-key step inside it
@@ -350,15 +380,22 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
             ptx::tmem_ld32(tmem_s, sc);
             ptx::tmem_ld32(tmem_s + 32, sc + 32);
             ptx::tmem_wait_ld();
+            if (BIASED) {
+                const float b0 = slope2 * static_cast<float>(key0 - (causal_base + t));   // <= 0 where the key is visible
+#pragma unroll
+                for (int c = 0; c < 64; ++c) {
+                    sc[c] = __float_as_uint(fmaf(__uint_as_float(sc[c]), a.scale_log2, fmaf(slope2, static_cast<float>(c), b0)));
+                }
+            }
             // visibility of this thread's 64 keys as one 64-bit word: causal bound, window bound, tree-mask bits,
             // block selection.  (A per-key chain of comparisons here made the half-empty last token tile of a
             // verify pass, whose rows see nothing, 2.2 times slower than the full tiles.)
             uint64_t vb = ~0ull;
-            if (!blk_ok || limit <= key0 || key_lo >= key0 + 64) {
+            if (!blk_ok || limit <= key0 || row_lo >= key0 + 64) {
                 vb = 0ull;
             } else {
                 if (limit < key0 + 64) vb &= (1ull << (limit - key0)) - 1ull;
-                if (key_lo > key0) vb &= ~((1ull << (key_lo - key0)) - 1ull);
+                if (row_lo > key0) vb &= ~((1ull << (row_lo - key0)) - 1ull);
                 const int mo = mbeg - key0;  // first column the tree mask applies to (mbeg is huge when there is none)
                 if (mo < 64) {
                     const uint64_t tm = (mo >= 0) ? ((mo > 0 ? (mword << mo) : mword) | ((1ull << mo) - 1ull))
@@ -392,15 +429,15 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
             // and fp32 sums), and O has to be rescaled - which needs the previous PV to have finished and
             // serialises the pipeline - only on such jumps instead of whenever any row of a warp sees a new maximum.
             float m_new = m_run;
-            if (m_tile != -INFINITY && (m_run == -INFINITY || (m_tile - m_run) * a.scale_log2 > 8.f)) m_new = m_tile;
+            if (m_tile != -INFINITY && (m_run == -INFINITY || (m_tile - m_run) * sl2 > 8.f)) m_new = m_tile;
             const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
-            const float alpha = (m_run == -INFINITY) ? 1.f : fast_exp2((m_run - m_use) * a.scale_log2);
+            const float alpha = (m_run == -INFINITY) ? 1.f : fast_exp2((m_run - m_use) * sl2);
             const bool rescale = (i > 0) && __any_sync(0xffffffffu, alpha != 1.f);
             if (rescale) {  // O must hold every product issued so far: wait for PV(i-1)
                 if (!ptx::mbar_wait_warp(&o_bar[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag)) { ok = false; break; }
                 ptx::tc_fence_after();
 #pragma unroll 1
-                for (int c0 = 0; c0 < 64; c0 += 32) {
+                for (int c0 = 0; c0 < DV / 2; c0 += 32) {
                     uint32_t r[32];
                     ptx::tmem_ld32(tmem_o + c0, r);
                     ptx::tmem_wait_ld();
@@ -417,15 +454,15 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
             const long long pc4 = prof_clock();
 
             // ---- P = 2^((s - m) * scale) in bf16 into the swizzled A-operand tile; row sums in fp32
-            const float m_off = m_use * a.scale_log2;
+            const float m_off = m_use * sl2;
             float ls[4] = {0.f, 0.f, 0.f, 0.f};
-            uint8_t* p_half = smem + SMEM_P + st * TILE_BYTES + ch * HALF_BYTES + row * 128;
+            uint8_t* p_half = smem + C::SMEM_P + st * C::P_TILE + ch * HALF_BYTES + row * 128;
 #pragma unroll
             for (int c8 = 0; c8 < 8; ++c8) {
                 float p[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
-                    p[e] = fast_exp2(fmaf(__uint_as_float(sc[c8 * 8 + e]), a.scale_log2, -m_off));
+                    p[e] = fast_exp2(fmaf(__uint_as_float(sc[c8 * 8 + e]), sl2, -m_off));
                     ls[e & 3] += p[e];
                 }
                 uint4 pk;
@@ -463,14 +500,16 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
         ptx::named_bar_sync(1, SOFTMAX_THREADS);
         const float l_row = l_run + xch[(ch ^ 1) * ROWS + row];
         if (ok) {
-            const bool store = (t < a.tq);
+            const bool store = row_in && (t < a.tq);
             const size_t grow = static_cast<size_t>(store ? t : 0) * a.hq + qh;
             const float inv = (nsplit == 1) ? ((l_row > 0.f) ? 1.f / l_row : 0.f) : 1.f;
-            bf16* dst_b = a.out + static_cast<size_t>(store ? t : 0) * a.out_ld + qh * D + ch * 64;
+            bf16* dst_b = a.out + static_cast<size_t>(store ? t : 0) * a.out_ld + qh * (BIASED ? a.out_cols : DV) + ch * (DV / 2);
+            const int cols = BIASED ? a.out_cols - ch * (DV / 2) : DV / 2;   // real columns of this thread's half
+            const bool whole = !BIASED || (a.out_cols % 8 == 0 && a.out_ld % 8 == 0);
             float* dst_f =
-                (nsplit > 1) ? a.ws_o + (static_cast<size_t>(split) * a.tq * a.hq + grow) * D + ch * 64 : nullptr;
+                (nsplit > 1) ? a.ws_o + (static_cast<size_t>(split) * a.tq * a.hq + grow) * DV + ch * (DV / 2) : nullptr;
 #pragma unroll 1
-            for (int c0 = 0; c0 < 64; c0 += 32) {
+            for (int c0 = 0; c0 < DV / 2; c0 += 32) {
                 uint32_t r[32];
                 if (n_it > 0) {  // uniform across the CTA
                     ptx::tmem_ld32(tmem_o + c0, r);
@@ -491,7 +530,15 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
                                                                           __uint_as_float(r[c + e * 2 + 1]) * inv);
                                 w[e] = *reinterpret_cast<uint32_t*>(&b2);
                             }
-                            *reinterpret_cast<uint4*>(dst_b + c0 + c) = pk;
+                            if (!BIASED || (whole && c0 + c < cols)) {
+                                *reinterpret_cast<uint4*>(dst_b + c0 + c) = pk;
+                            } else if (!whole) {   // a head width that 16-byte stores do not fit
+                                const bf16* e8 = reinterpret_cast<const bf16*>(&pk);
+#pragma unroll
+                                for (int e = 0; e < 8; ++e) {
+                                    if (c0 + c + e < cols) dst_b[c0 + c + e] = e8[e];
+                                }
+                            }
                         }
                     } else {
 #pragma unroll
@@ -525,8 +572,9 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
 // Merge split partials: out = sum_s 2^((m_s - M) c) O_s / sum_s 2^((m_s - M) c) l_s.
 // One warp per (token, head) row; lane s first owns split s's (max, sum) pair, then
 // every lane accumulates four output columns with independent loads in flight.
+template <int DV>
 __global__ void attn_combine_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_ml, int nsplit,
-                                    int rows, int hq, float scale_log2, bf16* __restrict__ out, int out_ld) {
+                                    int rows, int hq, float scale_log2, bf16* __restrict__ out, int out_ld, int out_cols) {
     grid_dependency_sync();
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
@@ -534,12 +582,15 @@ __global__ void attn_combine_kernel(const float* __restrict__ ws_o, const float*
     // the first twelve splits' partial outputs are requested before the (max, sum) pairs they are weighted
     // with: both loads are in flight together instead of one L2 round trip after the other
     constexpr int B = 12;
-    const float* base = ws_o + static_cast<size_t>(row) * D + lane * 4;
-    const size_t stride = static_cast<size_t>(rows) * D;
-    float4 o[B];
+    constexpr int CPL = DV / 32;   // output columns per lane
+    using Vec = typename std::conditional<CPL == 4, float4, float2>::type;
+    auto zero = []() { Vec z; memset(&z, 0, sizeof(z)); return z; };
+    const float* base = ws_o + static_cast<size_t>(row) * DV + lane * CPL;
+    const size_t stride = static_cast<size_t>(rows) * DV;
+    Vec o[B];
 #pragma unroll
     for (int j = 0; j < B; ++j) {
-        o[j] = (j < nsplit) ? __ldcg(reinterpret_cast<const float4*>(base + j * stride)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        o[j] = (j < nsplit) ? __ldcg(reinterpret_cast<const Vec*>(base + j * stride)) : zero();
     }
     float m_s = -INFINITY, l_s = 0.f;
     if (lane < nsplit) {
@@ -554,33 +605,44 @@ __global__ void attn_combine_kernel(const float* __restrict__ ws_o, const float*
     float l = w_s * l_s;
 #pragma unroll
     for (int o2 = 16; o2 > 0; o2 >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o2);
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    float acc[CPL];
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) acc[c] = 0.f;
     for (int s0 = 0; s0 < nsplit; s0 += B) {
         if (s0 > 0) {
 #pragma unroll
             for (int j = 0; j < B; ++j) {
                 const int s = s0 + j;
-                o[j] = (s < nsplit) ? __ldcg(reinterpret_cast<const float4*>(base + s * stride)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                o[j] = (s < nsplit) ? __ldcg(reinterpret_cast<const Vec*>(base + s * stride)) : zero();
             }
         }
 #pragma unroll
         for (int j = 0; j < B; ++j) {
             const int s = s0 + j;
             const float w = (s < nsplit) ? __shfl_sync(0xffffffffu, w_s, s & 31) : 0.f;
-            acc.x += w * o[j].x;
-            acc.y += w * o[j].y;
-            acc.z += w * o[j].z;
-            acc.w += w * o[j].w;
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) acc[c] += w * reinterpret_cast<const float*>(&o[j])[c];
         }
     }
     const float inv = (l > 0.f) ? 1.f / l : 0.f;
     const int t = row / hq, qh = row - t * hq;
-    __nv_bfloat162 a0 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
-    __nv_bfloat162 a1 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-    uint2 pk;
-    pk.x = *reinterpret_cast<uint32_t*>(&a0);
-    pk.y = *reinterpret_cast<uint32_t*>(&a1);
-    *reinterpret_cast<uint2*>(out + static_cast<size_t>(t) * out_ld + qh * D + lane * 4) = pk;
+    bf16* dst = out + static_cast<size_t>(t) * out_ld + qh * out_cols + lane * CPL;
+    uint32_t pk[CPL / 2];
+#pragma unroll
+    for (int c = 0; c < CPL; c += 2) {
+        const __nv_bfloat162 b2 = __floats2bfloat162_rn(acc[c] * inv, acc[c + 1] * inv);
+        pk[c / 2] = *reinterpret_cast<const uint32_t*>(&b2);
+    }
+    if (out_cols == DV) {
+        if constexpr (CPL == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(pk[0], pk[1]);
+        else *reinterpret_cast<uint32_t*>(dst) = pk[0];
+    } else {   // padded head width
+        const bf16* e = reinterpret_cast<const bf16*>(pk);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+            if (lane * CPL + c < out_cols) dst[c] = e[c];
+        }
+    }
 }
 
 }  // namespace
@@ -591,29 +653,60 @@ size_t attn_workspace_bytes(int tq, int hq, int d, int splits) {
 
 AttnPlan make_attn_plan(const bf16* q, int q_ld_tokens, const bf16* k_cache, const bf16* v_cache, int budget, int tq,
                         int hq, int hkv, int d, int splits, bf16* out, int out_ld, float* ws_o, float* ws_ml) {
-    CPM_REQUIRE(d == D, "attention: head_dim must be 128");
-    CPM_REQUIRE(hq % hkv == 0, "attention: query heads must be a multiple of kv heads");
-    const int grp = hq / hkv;
-    CPM_REQUIRE(grp <= ROWS && ROWS % grp == 0, "attention: unsupported GQA ratio");
-    CPM_REQUIRE(tq >= 1 && splits >= 1 && splits <= 32, "attention: splits must be in [1,32]");
-    AttnPlan p;
-    p.tq = tq; p.hq = hq; p.hkv = hkv; p.d = d; p.splits = splits;
-    p.out = out; p.out_ld = out_ld; p.ws_o = ws_o; p.ws_ml = ws_ml;
-    p.scale = 1.0f / sqrtf(static_cast<float>(d));
-    p.tm_q = make_tmap_3d(q, d, hq, tq, static_cast<uint64_t>(d) * 2, static_cast<uint64_t>(q_ld_tokens) * 2, 64, grp,
-                          ROWS / grp);
-    p.tm_k = make_tmap_2d(k_cache, static_cast<uint64_t>(hkv) * d, budget, static_cast<uint64_t>(hkv) * d * 2, 64, KEYS);
-    p.tm_v = make_tmap_2d(v_cache, static_cast<uint64_t>(hkv) * d, budget, static_cast<uint64_t>(hkv) * d * 2, 64, KEYS);
+    CPM_REQUIRE(d == 128, "attention: head_dim must be 128");
+    CPM_REQUIRE(hq % hkv == 0 && hq / hkv <= ROWS && ROWS % (hq / hkv) == 0, "attention: unsupported GQA ratio");
+    AttnPlan p = make_biased_attn_plan(q, q_ld_tokens, k_cache, v_cache, budget, tq, hq, hkv, d, d, d, splits,
+                                       1.0f / sqrtf(static_cast<float>(d)), 0, 0.f, out, out_ld, ws_o, ws_ml);
+    p.biased = false;
     return p;
 }
 
-void launch_tree_attention(const AttnPlan& p, cudaStream_t s) {
-    ProfileScope prof(KC_ATTENTION, s);
+bool biased_attn_fits(int hq, int hkv, int dk, int dv) {
+    return (dk == 64 || dk == 128) && (dv == 64 || dv == 128) && hq % hkv == 0 && hq / hkv <= ROWS;
+}
+
+AttnPlan make_biased_attn_plan(const bf16* q, int q_ld_tokens, const bf16* k_cache, const bf16* v_cache, int budget, int tq,
+                               int hq, int hkv, int dk, int dv, int out_cols, int splits, float scale, int exact_window,
+                               float bias_exp, bf16* out, int out_ld, float* ws_o, float* ws_ml) {
+    CPM_REQUIRE(biased_attn_fits(hq, hkv, dk, dv), "attention: unsupported head widths or GQA ratio");
+    CPM_REQUIRE(tq >= 1 && splits >= 1 && splits <= 32, "attention: splits must be in [1,32]");
+    CPM_REQUIRE(out_cols >= 1 && out_cols <= dv, "attention: more output columns than value columns");
+    const int grp = hq / hkv;
+    AttnPlan p;
+    p.tq = tq; p.hq = hq; p.hkv = hkv; p.d = dk; p.dv = dv; p.out_cols = out_cols; p.splits = splits;
+    p.biased = true;
+    p.exact_window = exact_window;
+    p.bias_exp = bias_exp;
+    p.out = out; p.out_ld = out_ld; p.ws_o = ws_o; p.ws_ml = ws_ml;
+    p.scale = scale;
+    p.tm_q = make_tmap_3d(q, dk, hq, tq, static_cast<uint64_t>(dk) * 2, static_cast<uint64_t>(q_ld_tokens) * 2, 64, grp,
+                          ROWS / grp);
+    p.tm_k = make_tmap_2d(k_cache, static_cast<uint64_t>(hkv) * dk, budget, static_cast<uint64_t>(hkv) * dk * 2, 64, KEYS);
+    p.tm_v = make_tmap_2d(v_cache, static_cast<uint64_t>(hkv) * dv, budget, static_cast<uint64_t>(hkv) * dv * 2, 64, KEYS);
+    return p;
+}
+
+namespace {
+template <int DK, int DV, bool BIASED>
+void launch_attn(const AttnPlan& p, const AttnArgs& a, cudaStream_t s) {
     static bool configured = false;
     if (!configured) {
-        CUDA_CHECK(cudaFuncSetAttribute(tree_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL));
+        CUDA_CHECK(cudaFuncSetAttribute(tree_attn_kernel<DK, DV, BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                        AttnCfg<DK, DV>::SMEM_TOTAL));
         configured = true;
     }
+    launch_kernel(tree_attn_kernel<DK, DV, BIASED>, dim3(a.num_mtiles * p.hkv, p.splits), dim3(NTHREADS), AttnCfg<DK, DV>::SMEM_TOTAL,
+                  s, p.tm_q, p.tm_k, p.tm_v, a);
+    if (p.splits > 1) {
+        const int rows = p.tq * p.hq;
+        launch_kernel(attn_combine_kernel<DV>, dim3(ceil_div(rows, 4)), dim3(128), 0, s, p.ws_o, p.ws_ml, p.splits, rows, p.hq,
+                      BIASED ? 1.f : a.scale_log2, p.out, p.out_ld, p.out_cols);
+    }
+}
+}  // namespace
+
+void launch_tree_attention(const AttnPlan& p, cudaStream_t s) {
+    ProfileScope prof(KC_ATTENTION, s);
     AttnArgs a;
     a.tq = p.tq; a.hq = p.hq; a.hkv = p.hkv;
     a.grp = p.hq / p.hkv;
@@ -626,6 +719,7 @@ void launch_tree_attention(const AttnPlan& p, cudaStream_t s) {
     a.n_valid = p.n_valid;
     a.mask = p.mask; a.mask_k = p.mask_k;
     a.window = p.window;
+    a.exact_window = p.exact_window; a.bias_exp = p.bias_exp; a.out_cols = p.out_cols;
     a.blockmask = p.blockmask; a.bm_words = p.bm_words; a.block_window = p.block_window;
     CPM_REQUIRE(p.blockmask == nullptr || (p.bm_words >= 1 && p.bm_words <= 64 && p.block_window >= 1),
                 "attention: block mask needs 1..64 words per row and a local window of at least one block");
@@ -664,11 +758,9 @@ void launch_tree_attention(const AttnPlan& p, cudaStream_t s) {
         }
     }
     CPM_REQUIRE(p.splits == 1 || (p.ws_o != nullptr && p.ws_ml != nullptr), "attention: split-KV needs a workspace");
-    dim3 grid(a.num_mtiles * p.hkv, p.splits);
-    launch_kernel(tree_attn_kernel, grid, dim3(NTHREADS), SMEM_TOTAL, s, p.tm_q, p.tm_k, p.tm_v, a);
-    if (p.splits > 1) {
-        const int rows = p.tq * p.hq;
-        launch_kernel(attn_combine_kernel, dim3(ceil_div(rows, 4)), dim3(128), 0, s, p.ws_o, p.ws_ml, p.splits, rows, p.hq,
-                      a.scale_log2, p.out, p.out_ld);
-    }
+    if (!p.biased) launch_attn<128, 128, false>(p, a, s);
+    else if (p.d == 128 && p.dv == 128) launch_attn<128, 128, true>(p, a, s);
+    else if (p.d == 128) launch_attn<128, 64, true>(p, a, s);
+    else if (p.dv == 128) launch_attn<64, 128, true>(p, a, s);
+    else launch_attn<64, 64, true>(p, a, s);
 }

@@ -82,6 +82,34 @@ int cpmcu_init_minicpm4_eagle_model(int num_layers, int num_iter, int topk_per_i
                                     int frspec_vocab_size, float residual_scale, int use_input_norm,
                                     int use_attn_norm);
 
+/* One layer of a layered model (no reference counterpart). */
+typedef struct {
+    /* mixer: softmax attention; query head h uses key/value head h / (heads / kv_heads) */
+    int heads, kv_heads, dim, vdim;
+    float scale;          /* score = scale * (q . k) - slope_h * (i - j) */
+    int window;           /* > 0: token i sees j with 0 <= i - j < window; 0: all j <= i */
+    float bias_exp;       /* > 0: slope_h = 2^(-bias_exp * (h + 1) / heads); 0: no distance bias */
+    int qk_norm;          /* RMS norms over all query rows and all key rows, before the split into heads */
+    int kv_from;          /* >= 0: keys and values of that earlier layer's cache; -1: its own */
+    /* feed-forward: mixture of experts; experts + identity == 0: the layer has none */
+    int experts;          /* gated experts; the router's outputs are experts + identity */
+    int identity;         /* the last outputs: experts that hand their input on */
+    int top;              /* experts per token */
+    int groups, keep_groups; /* equal groups of neighbouring outputs; only the best keep_groups can be chosen from */
+    float router_scale;
+    int expert_ff;
+    int shared_ff;        /* > 0: an expert of this width that every token uses; 0: none */
+} cpmcu_layer_spec;
+
+/* A decoder described layer by layer, with RMS norms (weights stored as their distance from one) on the sublayers'
+ * outputs and a 32-bit residual stream: x += residual_mult * norm(sublayer(x)).  torch_dtype: 1 = bf16, 2 = fp32 (all
+ * arithmetic in true 32-bit; weights are given as bf16 either way, logits come back in that dtype).
+ * Tensors for cpmcu_load_model: embed [vocab, width], head, final.norm, and for layer i (prefix "l<i>."): norm1, mix.q,
+ * mix.k, mix.v, mix.o, mix.q.norm, mix.k.norm, norm2, mlp.router, mlp.correction, mlp.e<j>.{gate,up,down},
+ * mlp.shared.{gate,up,down}; matrices [out, in] bf16. */
+int cpmcu_init_layered_model(float memory_limit, int vocab_size, int width, float norm_eps, float residual_mult,
+                             int torch_dtype, int chunk_length, int num_layers, const cpmcu_layer_spec* layers);
+
 /* reference: the three spec / hierarchical initialisers, src/entry.cu:344-459.
  * Out of scope for this library: always fail. */
 int cpmcu_init_w4a16_gm_spec_w4a16_gm_model(void);
@@ -103,10 +131,16 @@ int cpmcu_load_model(const char* name, const void* param);
 int cpmcu_prefill(int input_length, int history_length, const int32_t* input, const int32_t* position_ids,
                   void* output);
 
+/* The same, but with the logits of chosen tokens: row i of `output` ([n_want, vocab] in the model dtype) belongs to token
+ * want[i] of this chunk (HOST array; n_want may be 0).  No reference counterpart. */
+int cpmcu_prefill_rows(int input_length, int history_length, const int32_t* input, const int32_t* position_ids,
+                       const int32_t* want, int n_want, void* output);
+
 /* reference: decode, src/entry.cu:474-496.  *cache_length must already include
  * input_length (reference cpmcu/llm.py:263-283); mask_2d may be NULL (causal).
- * `output` is [input_length, vocab] bf16.  padded_length and cuda_graph are
- * accepted for compatibility and ignored. */
+ * `output` is [input_length, vocab] in the model dtype.  padded_length is accepted for
+ * compatibility; cuda_graph matters for layered models only, whose one-token step it captures and
+ * replays while the three device pointers stay the same. */
 int cpmcu_decode(int input_length, int padded_length, const int32_t* input, const int32_t* position_ids,
                  const int32_t* cache_length, const uint64_t* mask_2d, void* output, int cuda_graph);
 
@@ -162,6 +196,14 @@ long cpmcu_total_launches(void);
  * mask, [hkv][rows][words] packed per layer at stride hkv * max(chunk_length, 64) * words, into
  * device_buf (caller-owned device memory; NULL stops it).  Returns words per mask row. */
 int cpmcu_capture_blockmasks(uint64_t* device_buf);
+
+/* Test hook (layered models): from now on every forward pass also copies the residual stream after each layer,
+ * [layers][rows][width] fp32, to device_buf (caller-owned device memory; NULL stops it). */
+int cpmcu_capture_layers(float* device_buf);
+/* Per-launch timing of the forward passes made while it is on: cpmcu_profile(1) starts (decode then runs uncaptured),
+ * cpmcu_profile(0) stops and writes 6 entries each to ms / launches (HOST): linear layers, attention, block selection,
+ * expert products, routing, row-wise kernels. */
+int cpmcu_profile(int on, float* ms, int* launches);
 
 /* Copies the engine-owned tree of the last step to HOST arrays of 64 entries
  * (any pointer may be NULL). */
@@ -252,6 +294,34 @@ int cpmcu_silu_gate(const void* gate_up, void* out, int rows, int inter);
  * both projections rounded to bf16 before the product: bit-identical to cpmcu_linear_bf16 followed by
  * cpmcu_silu_gate.  inter % 64 == 0, K % 64 == 0. */
 int cpmcu_linear_swiglu_bf16(const void* x, const void* w, void* out, int rows, int inter, int K, int grid_limit);
+
+/* ---- mechanisms of layered models, one call each (no reference counterparts).  fp32 != 0: activations are fp32,
+ * otherwise bf16.  Row buffers have `ld` columns, a multiple of 64, zero beyond the real width. */
+
+/* Attention of a layer: q [tq, heads, dk], caches [budget, kv_heads, dk | dv] with dk / dv the head widths rounded up to 64
+ * and zero padded; keys visible = kv_total (HOST value), the last tq of them are the queries' own.  out [tq, heads * vdim].
+ * splits: key splits of the tensor-core kernel; 0 = the plain kernel. */
+int cpmcu_layer_attention(const cpmcu_layer_spec* spec, const void* q, const void* k_cache, const void* v_cache, int budget,
+                          int tq, int kv_total, int splits, int fp32, void* out);
+/* qkv [rows, heads*dim + kv_heads*(dim + vdim)] -> q_out [rows, heads, dk] and cache rows kv_row ..; norms as in the spec. */
+int cpmcu_layer_qkv_norm_append(const cpmcu_layer_spec* spec, const void* qkv, const void* wq, const void* wk, float eps,
+                                int rows, int kv_row, int cache_rows, int fp32, void* q_out, void* k_cache, void* v_cache);
+/* x32 += mult * rms(delta) * (1 + w); xh = x32 in the activation dtype. */
+int cpmcu_layer_out_norm(float* x32, void* xh, const void* delta, float mult, const void* w, int rows, int width, int ld,
+                         float eps, int fp32);
+/* The router: x32 [rows, ld] -> expert / weight [rows, top] (indices >= experts are identity experts). */
+int cpmcu_moe_route(const cpmcu_layer_spec* spec, const float* x32, const void* router, const float* correction, int rows,
+                    int ld, int32_t* expert, float* weight);
+/* The whole feed-forward on x32 [rows, ld] (and its bf16 copy xh): router, expert products, shared and identity experts,
+ * then x32 += mult * rms(sum) * (1 + w), in bf16.  gate_up: [2 * ff, width] per expert (gate rows, then up rows), expert after
+ * expert, the shared expert last; down: [width, ff] likewise. */
+int cpmcu_layer_mixture(const cpmcu_layer_spec* spec, float* x32, void* xh, const void* router, const float* correction,
+                        const void* gate_up, const void* down, float mult, const void* w, int rows, int width, int ld, float eps);
+/* Times the two grouped expert products of a layer (CUDA events, `iters` passes over `copies` weight sets; a random
+ * balanced choice of experts): us[0] = gate/up, us[1] = down. */
+int cpmcu_bench_experts(const cpmcu_layer_spec* spec, int width, int rows, int copies, int iters, float* us);
+/* Times the attention of a layer at `rows` queries behind `kv_total` keys, rotating over 8 caches. */
+int cpmcu_bench_layer_attention(const cpmcu_layer_spec* spec, int rows, int kv_total, int splits, int iters, float* us);
 
 /* Row argmax (lowest index wins ties); reference: torch argmax in
  * cpmcu/speculative/tree_drafter.py:233. */
