@@ -99,9 +99,38 @@ def route(logits, correction, router):
     return idx, wt
 
 
-def mixture(x, mlp, w, p):
+def choice_margin(logits, correction, router):
+    """[rows]: how far the closest call among a row's choices (of groups, then of experts) is from going the other way, as
+    the gap of the two choice scores over the sum of their scores s (and a thousandth of the choice score, whose own last
+    bits count when s is tiny).  Rounding moves s by a small fraction of itself, so rows with a small margin may choose
+    differently in low precision."""
+    s = torch.softmax(logits, dim=-1)
+    choice = s if correction is None else s + correction
+    n = s.shape[-1]
+    groups = router.get("groups") or {"count": 1, "keep": 1}
+    per = n // groups["count"]
+
+    def gap(values, scores, k):
+        if k >= values.shape[-1]:
+            return torch.full(values.shape[:1], float("inf"), dtype=values.dtype)
+        top = values.topk(k + 1, dim=-1)
+        at = top.indices[:, k - 1:k + 1]
+        return (top.values[:, k - 1] - top.values[:, k]) / (scores.gather(1, at).sum(-1) + 1e-3 * top.values[:, k].abs())
+
+    best = choice.view(-1, groups["count"], per).max(dim=-1)
+    best_s = s.view(-1, groups["count"], per).gather(2, best.indices[..., None]).squeeze(-1)
+    margin = gap(best.values, best_s, groups["keep"])
+    keep = torch.zeros_like(best_s, dtype=torch.bool).scatter_(1, best.values.topk(groups["keep"], dim=-1).indices, True)
+    masked = choice.masked_fill(~keep.repeat_interleave(per, dim=1), -1e30)
+    return torch.minimum(margin, gap(masked, s, router["top"]))
+
+
+def mixture(x, mlp, w, p, margins_out=None):
     router = mlp["router"]
-    idx, wt = route(x @ w[p + ".router"].T, w.get(p + ".correction"), router)
+    logits = x @ w[p + ".router"].T
+    idx, wt = route(logits, w.get(p + ".correction"), router)
+    if margins_out is not None:
+        margins_out.append(choice_margin(logits, w.get(p + ".correction"), router))
     out = torch.zeros_like(x)
     for e in range(router["experts"]):
         rows, slot = (idx == e).nonzero(as_tuple=True)
@@ -123,8 +152,9 @@ class Sequence:
         self.kv = {}
 
 
-def forward(config, weights, tokens, seq=None, layers_out=None):
-    """Logits [len(tokens), vocab] of the next tokens of `seq` (a fresh sequence when None)."""
+def forward(config, weights, tokens, seq=None, layers_out=None, margins_out=None):
+    """Logits [len(tokens), vocab] of the next tokens of `seq` (a fresh sequence when None).  layers_out receives the stream
+    after every layer, margins_out the choice margins of every mixture."""
     seq = seq if seq is not None else Sequence()
     w, eps, m = weights, config["norm"]["eps"], config["residual_mult"]
     x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)]
@@ -141,7 +171,7 @@ def forward(config, weights, tokens, seq=None, layers_out=None):
         a = attention(q, k, v, mix["scale"], mask_size(mix), seq.length)
         x = x + m * norm_around_one(a @ w[p + ".mix.o"].T, w[p + ".norm1"], eps)
         if layer.get("mlp"):
-            x = x + m * norm_around_one(mixture(x, layer["mlp"], w, p + ".mlp"), w[p + ".norm2"], eps)
+            x = x + m * norm_around_one(mixture(x, layer["mlp"], w, p + ".mlp", margins_out), w[p + ".norm2"], eps)
         if layers_out is not None:
             layers_out.append(x)
     seq.length += len(tokens)
