@@ -220,15 +220,17 @@ class LLM(torch.nn.Module):
         return self.logits[:n].clone()
 
     def _decode_one(self, token, position):
-        """Logits [1, vocab] after `token`, which becomes row `position` of the cache."""
-        if not hasattr(self, "input_ids"):
-            self.input_ids = torch.tensor([0], dtype=torch.int32, device="cuda")
-            self.position_ids = torch.tensor([0], dtype=torch.int32, device="cuda")
-            self.cache_length = torch.tensor([0], dtype=torch.int32, device="cuda")
-        self.input_ids[0] = token
-        self.position_ids[0] = position
-        self.cache_length[0] = position
-        return self.decode(self.input_ids, self.position_ids, self.cache_length)
+        """Logits [1, vocab] after `token`, which becomes row `position` of the cache.  The next call overwrites them."""
+        if not hasattr(self, "_step_host"):
+            # token id, position and cache length of a step travel in one copy from pinned memory
+            self._step_host = torch.zeros(3, dtype=torch.int32, pin_memory=True)
+            self._step_dev = torch.zeros(3, dtype=torch.int32, device="cuda")
+            self._step_np = self._step_host.numpy()
+        self._step_np[:] = (token, position, position + 1)
+        self._step_dev.copy_(self._step_host, non_blocking=True)
+        at = self._step_dev.data_ptr()
+        C.decode(1, (position + 128) // 128 * 128, at, at + 4, at + 8, 0, self.logits.data_ptr(), self.cuda_graph)
+        return self.logits[:1]
 
     def extend(self, tokens, history, want):
         """Append `tokens` (a list of ids) behind the `history` tokens the cache holds; history 0 starts a new sequence.

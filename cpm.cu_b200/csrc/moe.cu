@@ -30,27 +30,26 @@ struct RouteArgs {
     MoeBuffers b;
 };
 
-__device__ __forceinline__ void warp_argmax(float& v, int& i) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, i, o);
-        if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
-    }
+// Largest of n values in shared memory, lowest index first among equals: values as integers of the same order, so one
+// warp-wide integer maximum and one minimum over the indices do.
+__device__ __forceinline__ uint32_t ordered_bits(float v) {
+    const uint32_t u = __float_as_uint(v + 0.f);   // -0 counts as +0
+    return (u & 0x80000000u) ? ~u : (u | 0x80000000u);
 }
-
-// Largest of n values in shared memory, lowest index first among equals.
 __device__ __forceinline__ int argmax_of(const float* a, int n, int lane) {
-    float v = -INFINITY;
+    uint32_t v = 0u;
     int i = 0x7fffffff;
     for (int e = lane; e < n; e += 32) {
-        if (a[e] > v || i == 0x7fffffff) { v = a[e]; i = e; }
+        const uint32_t u = ordered_bits(a[e]);
+        if (u > v) { v = u; i = e; }
     }
-    warp_argmax(v, i);
-    return i;
+    const uint32_t m = __reduce_max_sync(0xffffffffu, v);
+    return __reduce_min_sync(0xffffffffu, v == m ? i : 0x7fffffff);
 }
 
-// The experts of one row, one warp.  sc: 2 * outputs + 2 * groups floats of scratch.
+// The experts of one row, one warp.  sc: 2 * outputs + 2 * groups floats of scratch.  ALONE: the launch has one row, whose
+// experts' row groups are written here as well.
+template <bool ALONE>
 __device__ void choose_experts(const RouteArgs& a, int row, float* sc, int lane) {
     const int n = a.outputs;
     float* score = sc;
@@ -117,7 +116,17 @@ __device__ void choose_experts(const RouteArgs& a, int row, float* sc, int lane)
         const size_t i = static_cast<size_t>(row) * a.top + lane;
         a.b.expert[i] = mine;
         a.b.weight[i] = weight;
-        a.b.rank[i] = (mine < a.experts) ? atomicAdd(&a.b.counts[mine], 1) : 0;
+        a.b.rank[i] = (!ALONE && mine < a.experts) ? atomicAdd(&a.b.counts[mine], 1) : 0;
+    }
+    if constexpr (ALONE) {
+        const bool real = lane < a.top && mine < a.experts;
+        const uint32_t reals = __ballot_sync(0xffffffffu, real);
+        const int at = __popc(reals & ((1u << lane) - 1u));
+        if (real) {
+            a.b.offset[mine] = at;
+            a.b.entries[at] = make_int4(mine, a.direct ? 0 : at, at, 1);
+        }
+        if (lane == 0) *a.b.n_entries = __popc(reals);
     }
     if (lane == 0) a.b.id_weight[row] = idw;
     __syncwarp();
@@ -201,14 +210,32 @@ moe_route_kernel(const RouteArgs a) {
             }
         }
     }
+    // Sum over the lanes.  With 32 sums or more every exchange hands half of a lane's partial sums to its partner, so
+    // lane l ends up with the sums l * N / 32 ..; the additions are those of a plain butterfly.
+    constexpr int N = EPW * RB;
+    float* v = &acc[0][0];
+    if constexpr (N >= 32) {
 #pragma unroll
-    for (int i = 0; i < EPW; ++i) {
+        for (int o = 16, half = N / 2; o > 0; o >>= 1, half >>= 1) {
+            const bool upper = (lane & o) != 0;
 #pragma unroll
-        for (int r = 0; r < RB; ++r) {
-            float v = acc[i][r];
+            for (int j = 0; j < half; ++j) {
+                const float give = upper ? v[j] : v[j + half], keep = upper ? v[j + half] : v[j];
+                v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+            }
+        }
 #pragma unroll
-            for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-            if (lane == 0 && r < nr && e0 + i < a.outputs) a.b.z[static_cast<size_t>(r0 + r) * a.outputs + e0 + i] = v;
+        for (int j = 0; j < N / 32; ++j) {
+            const int k = lane * (N / 32) + j, i = k / RB, r = k % RB;
+            if (r < nr && e0 + i < a.outputs) a.b.z[static_cast<size_t>(r0 + r) * a.outputs + e0 + i] = v[j];
+        }
+    } else {
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) v[k] += __shfl_xor_sync(0xffffffffu, v[k], o);
+            const int i = k / RB, r = k % RB;
+            if (lane == 0 && r < nr && e0 + i < a.outputs) a.b.z[static_cast<size_t>(r0 + r) * a.outputs + e0 + i] = v[k];
         }
     }
     // the CTA counted last of this block of rows chooses its experts
@@ -226,7 +253,7 @@ moe_route_kernel(const RouteArgs a) {
     if (s_last == 0) return;
     __threadfence();
     const int per_warp = 2 * a.outputs + 2 * a.groups;
-    for (int r = warp; r < nr; r += RT_WARPS) choose_experts(a, r0 + r, sm + warp * per_warp, lane);
+    for (int r = warp; r < nr; r += RT_WARPS) choose_experts<false>(a, r0 + r, sm + warp * per_warp, lane);
     // the CTA counted last of the launch lays out the rows
     __threadfence();
     __syncthreads();
@@ -239,6 +266,62 @@ moe_route_kernel(const RouteArgs a) {
     if (s_last == 0) return;
     __threadfence();
     if (warp == 0) lay_out_rows(a, lane);
+}
+
+// A launch with a single row (decoding): one output per warp, whose weights are on their way before the row exists.  The
+// additions are those of moe_route_kernel.
+constexpr int RT_PRE = 32;   // 128-column pieces of the weights held in registers
+__global__ void __launch_bounds__(RT_WARPS * 32)
+moe_route_one_kernel(const RouteArgs a) {
+    grid_dep_trigger();
+    extern __shared__ float sm[];
+    __shared__ int s_last;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int e = blockIdx.x * RT_WARPS + warp;
+    const bf16* w = a.w + static_cast<size_t>(e < a.outputs ? e : 0) * a.ld;
+    uint2 wv[RT_PRE];
+#pragma unroll
+    for (int j = 0; j < RT_PRE; ++j) {
+        const int c = j * 128 + lane * 4;
+        wv[j] = c < a.ld ? __ldg(reinterpret_cast<const uint2*>(w + c)) : make_uint2(0u, 0u);
+    }
+    grid_dep_wait();
+    float acc = 0.f;
+    auto add = [&](const uint2& wp, const float4& x) {
+        const bf16* b = reinterpret_cast<const bf16*>(&wp);
+        acc = fmaf(x.x, __bfloat162float(b[0]), acc);
+        acc = fmaf(x.y, __bfloat162float(b[1]), acc);
+        acc = fmaf(x.z, __bfloat162float(b[2]), acc);
+        acc = fmaf(x.w, __bfloat162float(b[3]), acc);
+    };
+#pragma unroll
+    for (int j0 = 0; j0 < RT_PRE; j0 += 8) {
+        float4 x[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int c = (j0 + j) * 128 + lane * 4;
+            x[j] = c < a.ld ? *reinterpret_cast<const float4*>(a.x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) add(wv[j0 + j], x[j]);
+    }
+    for (int c = RT_PRE * 128 + lane * 4; c < a.ld; c += 128) {
+        add(*reinterpret_cast<const uint2*>(w + c), *reinterpret_cast<const float4*>(a.x + c));
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+    if (lane == 0 && e < a.outputs) a.b.z[e] = acc;
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        const int last = atomicAdd(&a.b.tickets[0], 1) == static_cast<int>(gridDim.x) - 1;
+        if (last) a.b.tickets[0] = 0;
+        s_last = last;
+    }
+    __syncthreads();
+    if (s_last == 0 || warp != 0) return;
+    __threadfence();
+    choose_experts<true>(a, 0, sm, lane);
 }
 
 // One CTA per token row: its input goes to every chosen expert's slot.
@@ -293,6 +376,8 @@ struct GemmArgs {
     const int32_t* n_entries;
     int* error;
 };
+// The row groups come from the router.  gate/up launches its successor only after its own wait, i.e. when the router has
+// finished; down may therefore read the groups, and ask for their weights, before it waits for gate/up.
 
 // Output tile t: the shared expert's tiles come first, then the experts' row groups; the feature tile runs fastest, so
 // CTAs of a wave share a group's rows and its expert's matrix passes through L2 once for all of the expert's groups.
@@ -351,7 +436,8 @@ moe_gemm_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_cons
 
     const int warp = threadIdx.x >> 5;
     const int lane = threadIdx.x & 31;
-    grid_dep_trigger();
+    constexpr bool kGroupsEarly = !SWIGLU;
+    if (kGroupsEarly) grid_dep_trigger();
     if (threadIdx.x == 0) {
         for (int s = 0; s < C::STAGES; ++s) {
             ptx::mbar_init(&full[s], 1);
@@ -371,28 +457,53 @@ moe_gemm_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_cons
         ptx::tmem_alloc(tmem_slot, C::TMEM_COLS);
         ptx::tmem_relinquish();
     }
-    grid_dep_wait();   // the row groups come from the router
-    const int n_entries = min(*a.n_entries, kMoeMaxEntries);
-    for (int i = threadIdx.x; i < n_entries; i += NUM_THREADS) entries[i] = a.entries[i];
+    auto read_groups = [&]() -> int {
+        const int n = min(__ldcg(a.n_entries), kMoeMaxEntries);
+        for (int i = threadIdx.x; i < n; i += NUM_THREADS) entries[i] = __ldcg(a.entries + i);
+        return n;
+    };
+    int n_entries = kGroupsEarly ? read_groups() : 0;
     ptx::tc_fence_before();
     __syncthreads();
     ptx::tc_fence_after();
     const uint32_t tmem_base = *tmem_slot;
-    const int total = a.groups_s * a.n_tiles_s + n_entries * a.n_tiles;
+    // weights of the first k-blocks, as far as the tiles are known, before the wait for the predecessor
+    const int shared_tiles = a.groups_s * a.n_tiles_s;
+    int pre = 0;
+    if (threadIdx.x == 0) {
+        const int known = shared_tiles + n_entries * a.n_tiles;
+        for (int t = blockIdx.x; t < known && pre < C::STAGES; t += gridDim.x) {
+            const TileJob j = tile_job<SWIGLU>(a, entries, t);
+            for (int kb = 0; kb < j.kblocks && pre < C::STAGES; ++kb, ++pre) {
+                ptx::mbar_arrive_expect_tx(&full[pre], C::STAGE_BYTES);
+                ptx::tma_load_2d(tiles + pre * C::STAGE_BYTES, &tm_w, &full[pre], 0, j.w_row + kb * gemm::BLOCK_N);
+            }
+        }
+    }
+    grid_dep_wait();
+    if (!kGroupsEarly) {
+        grid_dep_trigger();
+        n_entries = read_groups();
+        __syncthreads();
+    }
+    const int total = shared_tiles + n_entries * a.n_tiles;
 
     if (warp == 0) {
         // ------------------------------------------------ TMA producer
         if (lane == 0) {
             int stage = 0;
             uint32_t phase = 0;
+            int issued = 0;
             bool ok = true;
             for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
                 const TileJob j = tile_job<SWIGLU>(a, entries, t);
-                for (int kb = 0; kb < j.kblocks; ++kb) {
-                    if (!ptx::mbar_wait(&empty[stage], phase ^ 1, abort_flag)) { ok = false; break; }
+                for (int kb = 0; kb < j.kblocks; ++kb, ++issued) {
                     uint8_t* dst = tiles + stage * C::STAGE_BYTES;
-                    ptx::mbar_arrive_expect_tx(&full[stage], C::STAGE_BYTES);
-                    ptx::tma_load_2d(dst, &tm_w, &full[stage], 0, j.w_row + kb * gemm::BLOCK_N);
+                    if (issued >= pre) {
+                        if (!ptx::mbar_wait(&empty[stage], phase ^ 1, abort_flag)) { ok = false; break; }
+                        ptx::mbar_arrive_expect_tx(&full[stage], C::STAGE_BYTES);
+                        ptx::tma_load_2d(dst, &tm_w, &full[stage], 0, j.w_row + kb * gemm::BLOCK_N);
+                    }
                     ptx::tma_load_2d(dst + W_TILE_BYTES, j.shared ? &tm_xs : &tm_x, &full[stage], kb * BLOCK_K, j.x_row);
                     if (++stage == C::STAGES) { stage = 0; phase ^= 1; }
                 }
@@ -552,8 +663,11 @@ void launch_moe_route(const LayerSpec& sp, const float* x32, const bf16* w, cons
         launch_kernel(kernel, dim3(ceil_div(rows, rb), ceil_div(a.outputs, RT_WARPS * epw)), dim3(RT_WARPS * 32), smem, s, a);
     };
     static bool c1 = false, c8 = false;
-    if (rows <= 16) run(moe_route_kernel<1, 1>, 1, 1, c1);
-    else run(moe_route_kernel<8, 4>, 8, 4, c8);
+    if (rows == 1) {
+        const size_t smem = (2 * a.outputs + 2 * a.groups) * sizeof(float);   // at most 16 KB
+        launch_kernel(moe_route_one_kernel, dim3(ceil_div(a.outputs, RT_WARPS)), dim3(RT_WARPS * 32), smem, s, a);
+    } else if (rows <= 16) run(moe_route_kernel<1, 1>, 1, 1, c1);
+    else run(moe_route_kernel<8, 8>, 8, 8, c8);
 }
 
 template <typename T>
