@@ -1,13 +1,14 @@
 // Mixture of experts for layered models (layered.cuh): fp32 router with grouped choice and identity experts, the layout
 // of the chosen rows, and the grouped expert products on the tensor cores.
 //
-//   route    fp32 logits (one warp per few outputs, rows staged in shared memory); the CTA counted last of a block of rows
+//   route    fp32 logits (8 rows x 8 outputs per warp, rows staged in shared memory); the CTA counted last of a block of rows
 //            picks its rows' experts; the CTA counted last of the launch cuts every expert's rows into groups
 //   gather   each chosen row's input is copied to its place, expert after expert
 //   gate/up  grouped tcgen05 product, SwiGLU in the epilogue
 //   down     grouped tcgen05 product
 // The weighted sum over a token's experts, the identity part and the output norm are one kernel (out_norm_kernel).
 #include <algorithm>
+#include <type_traits>
 
 #include "gemm_common.cuh"
 #include "layered.cuh"
@@ -17,7 +18,6 @@ namespace {
 
 // ---------------------------------------------------------------- router
 constexpr int RT_WARPS = 8;
-constexpr int RT_KC = 1024;   // columns of x staged at a time
 
 struct RouteArgs {
     const float* x;
@@ -161,82 +161,108 @@ __device__ void lay_out_rows(const RouteArgs& a, int lane) {
     if (lane == 0) *a.b.n_entries = min(entry0, kMoeMaxEntries);
 }
 
-// grid: (row blocks of RB, blocks of RT_WARPS * EPW outputs)
-template <int RB, int EPW>
-__global__ void __launch_bounds__(RT_WARPS * 32)
+// Sums of N values over the lanes of a warp, N a multiple of 32: every exchange hands half of a lane's partial sums to its
+// partner, so lane l ends up with values l * N / 32 .. of v[0 ..]; the additions are those of a plain butterfly.
+template <int N>
+__device__ __forceinline__ void warp_reduce_scatter(float* v, int lane) {
+#pragma unroll
+    for (int o = 16, half = N / 2; o > 0; o >>= 1, half >>= 1) {
+        const bool upper = (lane & o) != 0;
+#pragma unroll
+        for (int j = 0; j < half; ++j) {
+            const float give = upper ? v[j] : v[j + half], keep = upper ? v[j + half] : v[j];
+            v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+}
+
+// A warp computes 8 rows x 8 outputs, lanes along the columns; WE of a CTA's warps are neighbours in the outputs, the rest in
+// the rows.  Rows pass through two shared-memory stages, the next weights are in flight while the current ones are used.
+// grid: (row blocks, blocks of 8 * WE outputs)
+template <int WE>
+struct RouteCfg {
+    static constexpr int WR = RT_WARPS / WE;
+    static constexpr int ROWS = 8 * WR;
+    static constexpr int KC = WR >= 4 ? 128 : 512 / WR;   // columns per stage
+    static constexpr int STAGE = ROWS * KC;               // floats
+};
+template <int WE>
+__global__ void __launch_bounds__(RT_WARPS * 32, 2)
 moe_route_kernel(const RouteArgs a) {
+    using C = RouteCfg<WE>;
     grid_dep_trigger();
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     __shared__ int s_last;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int r0 = blockIdx.x * RB, nr = min(RB, a.rows - r0);
-    const int e0 = (blockIdx.y * RT_WARPS + warp) * EPW;
+    const int r0 = blockIdx.x * C::ROWS, nr = min(C::ROWS, a.rows - r0);
+    const int e0 = (blockIdx.y * WE + warp % WE) * 8, wr = (warp / WE) * 8;
+    const int steps = (a.ld + 127) / 128, stages = (a.ld + C::KC - 1) / C::KC;
+    uint2 next[8];
+    auto load_w = [&](int step) {
+        const int c = step * 128 + lane * 4;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            next[i] = (e0 + i < a.outputs && c < a.ld) ? __ldg(reinterpret_cast<const uint2*>(a.w + static_cast<size_t>(e0 + i) * a.ld + c))
+                                                       : make_uint2(0u, 0u);
+        }
+    };
+    auto load_x = [&](int stage) {
+        float* dst = sm + (stage & 1) * C::STAGE;
+#pragma unroll
+        for (int j = 0; j < C::STAGE / 4; j += RT_WARPS * 32) {
+            const int i = (j + threadIdx.x) * 4, r = i / C::KC, c = stage * C::KC + i % C::KC;
+            const bool in = r < nr && c < a.ld;   // elsewhere zeros are filled in
+            ptx::cp_async16(dst + i, in ? a.x + static_cast<size_t>(r0 + r) * a.ld + c : a.x, in ? 16 : 0);
+        }
+        ptx::cp_async_commit();
+    };
+    load_w(0);   // the weights never depend on the previous kernel
     grid_dep_wait();
-    float acc[EPW][RB];
+    float acc[64];
 #pragma unroll
-    for (int i = 0; i < EPW; ++i) {
-#pragma unroll
-        for (int r = 0; r < RB; ++r) acc[i][r] = 0.f;
-    }
-    for (int k0 = 0; k0 < a.ld; k0 += RT_KC) {
-        const int kn = min(RT_KC, a.ld - k0);   // a multiple of 64
-        __syncthreads();
-        for (int i = threadIdx.x * 4; i < RB * kn; i += RT_WARPS * 32 * 4) {
-            const int r = i / kn, c = i - r * kn;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < nr) v = *reinterpret_cast<const float4*>(a.x + static_cast<size_t>(r0 + r) * a.ld + k0 + c);
-            *reinterpret_cast<float4*>(sm + r * RT_KC + c) = v;
+    for (int i = 0; i < 64; ++i) acc[i] = 0.f;
+    load_x(0);
+    for (int st = 0; st < stages; ++st) {
+        if (st + 1 < stages) {
+            load_x(st + 1);
+            ptx::cp_async_wait<1>();
+        } else {
+            ptx::cp_async_wait<0>();
         }
         __syncthreads();
-        for (int c = lane * 4; c < kn; c += 128) {
-            float w[EPW][4];
+        const float* xs = sm + (st & 1) * C::STAGE + wr * C::KC + lane * 4;
+#pragma unroll 1
+        for (int k = 0; k < C::KC / 128; ++k) {
+            const int step = st * (C::KC / 128) + k;
+            if (step >= steps) break;
+            float w[8][4];
 #pragma unroll
-            for (int i = 0; i < EPW; ++i) {
-                bf16 b[4] = {};
-                if (e0 + i < a.outputs) *reinterpret_cast<uint2*>(b) = *reinterpret_cast<const uint2*>(a.w + static_cast<size_t>(e0 + i) * a.ld + k0 + c);
+            for (int i = 0; i < 8; ++i) {
+                const bf16* b = reinterpret_cast<const bf16*>(&next[i]);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) w[i][e] = __bfloat162float(b[e]);
             }
+            if (step + 1 < steps) load_w(step + 1);
 #pragma unroll
-            for (int r = 0; r < RB; ++r) {
-                const float4 x = *reinterpret_cast<const float4*>(sm + r * RT_KC + c);
+            for (int r = 0; r < 8; ++r) {
+                const float4 x = *reinterpret_cast<const float4*>(xs + r * C::KC + k * 128);
 #pragma unroll
-                for (int i = 0; i < EPW; ++i) {
-                    acc[i][r] = fmaf(x.x, w[i][0], acc[i][r]);
-                    acc[i][r] = fmaf(x.y, w[i][1], acc[i][r]);
-                    acc[i][r] = fmaf(x.z, w[i][2], acc[i][r]);
-                    acc[i][r] = fmaf(x.w, w[i][3], acc[i][r]);
+                for (int i = 0; i < 8; ++i) {
+                    float& s = acc[i * 8 + r];
+                    s = fmaf(x.x, w[i][0], s);
+                    s = fmaf(x.y, w[i][1], s);
+                    s = fmaf(x.z, w[i][2], s);
+                    s = fmaf(x.w, w[i][3], s);
                 }
             }
         }
+        __syncthreads();   // the stage is filled again two iterations on
     }
-    // Sum over the lanes.  With 32 sums or more every exchange hands half of a lane's partial sums to its partner, so
-    // lane l ends up with the sums l * N / 32 ..; the additions are those of a plain butterfly.
-    constexpr int N = EPW * RB;
-    float* v = &acc[0][0];
-    if constexpr (N >= 32) {
+    warp_reduce_scatter<64>(acc, lane);
 #pragma unroll
-        for (int o = 16, half = N / 2; o > 0; o >>= 1, half >>= 1) {
-            const bool upper = (lane & o) != 0;
-#pragma unroll
-            for (int j = 0; j < half; ++j) {
-                const float give = upper ? v[j] : v[j + half], keep = upper ? v[j + half] : v[j];
-                v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
-            }
-        }
-#pragma unroll
-        for (int j = 0; j < N / 32; ++j) {
-            const int k = lane * (N / 32) + j, i = k / RB, r = k % RB;
-            if (r < nr && e0 + i < a.outputs) a.b.z[static_cast<size_t>(r0 + r) * a.outputs + e0 + i] = v[j];
-        }
-    } else {
-#pragma unroll
-        for (int k = 0; k < N; ++k) {
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) v[k] += __shfl_xor_sync(0xffffffffu, v[k], o);
-            const int i = k / RB, r = k % RB;
-            if (lane == 0 && r < nr && e0 + i < a.outputs) a.b.z[static_cast<size_t>(r0 + r) * a.outputs + e0 + i] = v[k];
-        }
+    for (int j = 0; j < 2; ++j) {
+        const int k = lane * 2 + j, e = e0 + k / 8, r = wr + k % 8;
+        if (r < nr && e < a.outputs) a.b.z[static_cast<size_t>(r0 + r) * a.outputs + e] = acc[j];
     }
     // the CTA counted last of this block of rows chooses its experts
     __threadfence();
@@ -269,7 +295,7 @@ moe_route_kernel(const RouteArgs a) {
 }
 
 // A launch with a single row (decoding): one output per warp, whose weights are on their way before the row exists.  The
-// additions are those of moe_route_kernel.
+// additions are those of moe_route_kernel, in the same order.
 constexpr int RT_PRE = 32;   // 128-column pieces of the weights held in registers
 __global__ void __launch_bounds__(RT_WARPS * 32)
 moe_route_one_kernel(const RouteArgs a) {
@@ -422,6 +448,7 @@ __global__ void __launch_bounds__(NUM_THREADS, 1)
 moe_gemm_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x,
                      const __grid_constant__ CUtensorMap tm_xs, const GemmArgs a) {
     using C = Cfg<MT>;
+    constexpr int XBOX = MT < 64 ? MT : 64;   // rows per copy of the row operand (x_box of the maps)
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* tiles = smem;
@@ -474,8 +501,9 @@ moe_gemm_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_cons
         const int known = shared_tiles + n_entries * a.n_tiles;
         for (int t = blockIdx.x; t < known && pre < C::STAGES; t += gridDim.x) {
             const TileJob j = tile_job<SWIGLU>(a, entries, t);
+            const uint32_t bytes = W_TILE_BYTES + (j.rows + XBOX - 1) / XBOX * (XBOX * BLOCK_K * 2);
             for (int kb = 0; kb < j.kblocks && pre < C::STAGES; ++kb, ++pre) {
-                ptx::mbar_arrive_expect_tx(&full[pre], C::STAGE_BYTES);
+                ptx::mbar_arrive_expect_tx(&full[pre], bytes);
                 ptx::tma_load_2d(tiles + pre * C::STAGE_BYTES, &tm_w, &full[pre], 0, j.w_row + kb * gemm::BLOCK_N);
             }
         }
@@ -497,14 +525,19 @@ moe_gemm_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_cons
             bool ok = true;
             for (int t = blockIdx.x; ok && t < total; t += gridDim.x) {
                 const TileJob j = tile_job<SWIGLU>(a, entries, t);
+                const int boxes = (j.rows + XBOX - 1) / XBOX;   // rows nobody asked for are not fetched
+                const uint32_t bytes = W_TILE_BYTES + boxes * (XBOX * BLOCK_K * 2);
                 for (int kb = 0; kb < j.kblocks; ++kb, ++issued) {
                     uint8_t* dst = tiles + stage * C::STAGE_BYTES;
                     if (issued >= pre) {
                         if (!ptx::mbar_wait(&empty[stage], phase ^ 1, abort_flag)) { ok = false; break; }
-                        ptx::mbar_arrive_expect_tx(&full[stage], C::STAGE_BYTES);
+                        ptx::mbar_arrive_expect_tx(&full[stage], bytes);
                         ptx::tma_load_2d(dst, &tm_w, &full[stage], 0, j.w_row + kb * gemm::BLOCK_N);
                     }
-                    ptx::tma_load_2d(dst + W_TILE_BYTES, j.shared ? &tm_xs : &tm_x, &full[stage], kb * BLOCK_K, j.x_row);
+                    for (int b = 0; b < boxes; ++b) {
+                        ptx::tma_load_2d(dst + W_TILE_BYTES + b * (XBOX * BLOCK_K * 2), j.shared ? &tm_xs : &tm_x, &full[stage], kb * BLOCK_K,
+                                         j.x_row + b * XBOX);
+                    }
                     if (++stage == C::STAGES) { stage = 0; phase ^= 1; }
                 }
             }
@@ -654,20 +687,27 @@ void launch_moe_route(const LayerSpec& sp, const float* x32, const bf16* w, cons
     a.b = b;
     CPM_REQUIRE(moe_max_entries(sp, rows, tile) <= kMoeMaxEntries, "mixture of experts: too many row groups");
     const size_t choose = static_cast<size_t>(RT_WARPS) * (2 * a.outputs + 2 * a.groups) * sizeof(float);
-    auto run = [&](auto kernel, int rb, int epw, bool& configured) {
-        const size_t smem = std::max<size_t>(choose, static_cast<size_t>(rb) * RT_KC * sizeof(float));
-        if (!configured) {
-            CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, RT_WARPS * 4 * kMoeMaxOutputs * 4));
-            configured = true;
-        }
-        launch_kernel(kernel, dim3(ceil_div(rows, rb), ceil_div(a.outputs, RT_WARPS * epw)), dim3(RT_WARPS * 32), smem, s, a);
-    };
-    static bool c1 = false, c8 = false;
     if (rows == 1) {
         const size_t smem = (2 * a.outputs + 2 * a.groups) * sizeof(float);   // at most 16 KB
         launch_kernel(moe_route_one_kernel, dim3(ceil_div(a.outputs, RT_WARPS)), dim3(RT_WARPS * 32), smem, s, a);
-    } else if (rows <= 16) run(moe_route_kernel<1, 1>, 1, 1, c1);
-    else run(moe_route_kernel<8, 8>, 8, 8, c8);
+        return;
+    }
+    auto run = [&](auto we) {
+        constexpr int WE = decltype(we)::value;
+        using C = RouteCfg<WE>;
+        static bool configured = false;
+        if (!configured) {
+            CUDA_CHECK(cudaFuncSetAttribute(moe_route_kernel<WE>, cudaFuncAttributeMaxDynamicSharedMemorySize, RT_WARPS * 4 * kMoeMaxOutputs * 4));
+            configured = true;
+        }
+        launch_kernel(moe_route_kernel<WE>, dim3(ceil_div(rows, C::ROWS), ceil_div(a.outputs, 8 * WE)), dim3(RT_WARPS * 32),
+                      std::max<size_t>(choose, 2 * C::STAGE * sizeof(float)), s, a);
+    };
+    // few rows: all warps side by side in the outputs, so that the rows spread over more CTAs
+    if (a.outputs > 32 || rows <= 64) run(std::integral_constant<int, 8>());
+    else if (a.outputs > 16) run(std::integral_constant<int, 4>());
+    else if (a.outputs > 8) run(std::integral_constant<int, 2>());
+    else run(std::integral_constant<int, 1>());
 }
 
 template <typename T>
@@ -689,8 +729,8 @@ MoeGemmPlan make_moe_gate_up_plan(const LayerSpec& sp, const bf16* w, const bf16
     MoeGemmPlan p;
     const int ff = pad64(sp.expert_ff), ffs = pad64(sp.shared_ff);
     p.tm_w = weight_map(w, moe_gate_up_elems(sp, K));
-    p.tm_x = make_tmap_2d(x, K, x_rows, static_cast<uint64_t>(K) * 2, BLOCK_K, tile);
-    p.tm_xs = make_tmap_2d(xs, K, rows, static_cast<uint64_t>(K) * 2, BLOCK_K, tile);
+    p.tm_x = make_tmap_2d(x, K, x_rows, static_cast<uint64_t>(K) * 2, BLOCK_K, std::min(tile, 64));
+    p.tm_xs = make_tmap_2d(xs, K, rows, static_cast<uint64_t>(K) * 2, BLOCK_K, std::min(tile, 64));
     p.tile = tile; p.rows = rows; p.max_entries = moe_max_entries(sp, rows, tile);
     p.swiglu = 1;
     p.n_tiles = ff / 64; p.kblocks = K / BLOCK_K; p.N = ff;
@@ -708,7 +748,7 @@ MoeGemmPlan make_moe_down_plan(const LayerSpec& sp, const bf16* w, const bf16* a
     MoeGemmPlan p;
     const int ff = pad64(sp.expert_ff), ffs = pad64(sp.shared_ff);
     p.tm_w = weight_map(w, moe_down_elems(sp, width));
-    p.tm_x = make_tmap_2d(act, ld_act, act_rows, static_cast<uint64_t>(ld_act) * 2, BLOCK_K, tile);
+    p.tm_x = make_tmap_2d(act, ld_act, act_rows, static_cast<uint64_t>(ld_act) * 2, BLOCK_K, std::min(tile, 64));
     p.tm_xs = p.tm_x;
     p.tile = tile; p.rows = rows; p.max_entries = moe_max_entries(sp, rows, tile);
     p.n_tiles = ceil_div(width, gemm::BLOCK_N); p.kblocks = ff / BLOCK_K; p.N = width;

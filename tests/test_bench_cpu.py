@@ -58,3 +58,17 @@ def test_list_split_feeds_target_then_drafter():
 def test_workload_table_covers_the_four_gpu_configurations():
     assert sorted(bench.WORKLOADS) == ["config2", "config3", "config4", "config5"]
     assert [bench.WORKLOADS[k]["index"] for k in sorted(bench.WORKLOADS)] == [1, 2, 3, 4]
+
+
+def test_layered_work_counts_match_the_hand_count():
+    import bench_layered as b
+    mlp = b._moe(6, 2, 32, 2, (4, 2), 16)
+    cfg = b._model(64, 4, 2, 8, 3, 2, mlp)                     # two layers, the second one shares the first one's cache
+    assert b.active_ff(cfg) == 2 * 32 + 16
+    V = b.VOCAB
+    by, fl = b.bytes_and_flops(cfg, "tipetar", 2, 10)
+    attn = 2 * (2 * 64 * 32) + 2 * 2 * 8 * 64                  # q and o twice, k and v once
+    assert by == {"linear": 2 * (attn + V * 64), "experts": 2 * 2 * 3 * 64 * 80, "attention": 2 * 2 * 3 * 2 * 8 * 2}
+    assert fl["attention"] == 2 * 4 * (3 + 3) * 32 and fl["experts"] == 2 * 2 * 2 * 3 * 64 * 80
+    by, fl = b.bytes_and_flops(cfg, "llama", 2, 10)
+    assert by["experts"] == 0 and fl["attention"] == 2 * 4 * (9 + 10) * 32

@@ -473,15 +473,32 @@ def test_extend_serves_llama_format_models_too():
     C.release()
 
 
+def write_checkpoint(mdir, cfg, w):
+    from safetensors.torch import save_file
+    mdir.mkdir()
+    (mdir / "config.json").write_text(json.dumps(cfg))
+    save_file({k: v.to(torch.bfloat16).contiguous() for k, v in w.items()}, str(mdir / "model.safetensors"))
+
+
+def test_command_line(tmp_path):
+    cfg = case("odd")
+    w = T.random_weights(cfg, seed=12)
+    write_checkpoint(tmp_path / "model", cfg, w)
+    prompt = tokens_of(cfg, 40, seed=3)
+    res = subprocess.run([sys.executable, "-m", "cpmcu", "--model", str(tmp_path / "model"), "--tokens", ",".join(map(str, prompt)), "--max-new", "12",
+                          "--dtype", "float32", "--chunk-length", "64", "--max-tokens", "256"], capture_output=True, text=True, timeout=300,
+                         env=dict(os.environ, PYTHONPATH=os.path.join(ROOT, "cpm.cu_b200")))
+    assert res.returncode == 0, res.stderr[-2000:]
+    assert [int(t) for t in res.stdout.strip().splitlines()[-1].split(",")] == T.greedy(cfg, w, prompt, 12)
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_trace_runner(tmp_path, dtype):
-    from safetensors.torch import save_file
     cfg = case("mixed")
     w = T.random_weights(cfg, seed=11)
     mdir, out = tmp_path / "model", tmp_path / "out"
-    mdir.mkdir(), out.mkdir()
-    (mdir / "config.json").write_text(json.dumps(cfg))
-    save_file({k: v.to(torch.bfloat16).contiguous() for k, v in w.items()}, str(mdir / "model.safetensors"))
+    write_checkpoint(mdir, cfg, w)
+    out.mkdir()
     toks, other = tokens_of(cfg, 80, seed=1), tokens_of(cfg, 9, seed=2)
     steps = [{"entries": [{"id": "x", "tokens": toks[:70], "want": [69, 0]}], "end": []},
              {"entries": [{"id": "x", "tokens": toks[70:71], "want": []}], "end": []},
@@ -500,4 +517,3 @@ def test_trace_runner(tmp_path, dtype):
         e = errors(got, rows)
         assert e.median() < (2e-5 if dt == torch.float32 else 0.03), (i, e)
     assert not (out / "1.f32").exists()
-    assert sys.executable
