@@ -67,7 +67,7 @@ def qkv(mix, tq, keys, seed=0, qgain=1.0):
     return q, k, v
 
 
-ATTN_SHAPES = [attn(4, 1, 64, 64, 100), attn(6, 2, 40, 56, 37, scale=0.3), attn(8, 1, 128, 64, 128), attn(2, 2, 64, 128, 300),
+ATTN_SHAPES = [attn(5, 1, 64, 64, 100), attn(6, 2, 40, 56, 37, scale=0.3), attn(8, 1, 128, 64, 128), attn(2, 2, 64, 128, 300),
                attn(5, 1, 96, 100, 129), attn(16, 2, 128, 128, None), attn(3, 3, 17, 3, 1)]
 
 
@@ -172,7 +172,7 @@ def test_output_norm_and_residual(width, fp32):
 
 
 # ---------------------------------------------------------------- mixture of experts
-ROUTERS = [moe(8, 4, 16, identity=4, groups=(4, 3), scale=2.0), moe(5, 3, 16, identity=3, groups=(4, 2), scale=1.7), moe(1, 1, 16),
+ROUTERS = [moe(11, 5, 16, identity=4, groups=(5, 3), scale=1.4), moe(5, 3, 16, identity=3, groups=(4, 2), scale=1.7), moe(1, 1, 16),
            moe(3, 4, 16, identity=5), moe(250, 8, 16, identity=50, groups=(10, 4), scale=0.3), moe(64, 32, 16, groups=(2, 1)),
            moe(40, 6, 16, identity=8, groups=(48, 7))]
 
