@@ -20,7 +20,16 @@ class LayerSpec(ctypes.Structure):
     _fields_ = [("heads", _c_int), ("kv_heads", _c_int), ("dim", _c_int), ("vdim", _c_int), ("scale", _c_float),
                 ("window", _c_int), ("bias_exp", _c_float), ("qk_norm", _c_int), ("kv_from", _c_int), ("experts", _c_int),
                 ("identity", _c_int), ("top", _c_int), ("groups", _c_int), ("keep_groups", _c_int),
-                ("router_scale", _c_float), ("expert_ff", _c_int), ("shared_ff", _c_int)]
+                ("router_scale", _c_float), ("expert_ff", _c_int), ("shared_ff", _c_int),
+                ("sink", _c_int), ("rot_dims", _c_int), ("attn_scale", _c_float), ("recurrence", _c_int), ("rec_heads", _c_int),
+                ("rec_dim", _c_int), ("rec_vdim", _c_int), ("rec_rank", _c_int), ("rec_scale", _c_float), ("ff", _c_int),
+                ("ff_limit", _c_float), ("ff_alpha", _c_float)]
+
+    def __init__(self, **kw):
+        for name, value in (("kv_from", -1), ("groups", 1), ("keep_groups", 1), ("router_scale", 1.0), ("attn_scale", 1.0),
+                            ("rec_scale", 1.0)):
+            kw.setdefault(name, value)
+        super().__init__(**kw)
 
 
 _SIGNATURES = {
@@ -29,7 +38,7 @@ _SIGNATURES = {
     "cpmcu_init_minicpm4_model": (_c_int, [_c_float] + [_c_int] * 7 + [_c_float, _c_int, _c_int] + [_c_float] * 3 + [_c_int] * 5),
     "cpmcu_init_w4a16_gptq_marlin_base_model": (_c_int, [_c_float] + [_c_int] * 7 + [_c_float, _c_int, _c_int, _c_int] + [_c_float] * 3),
     "cpmcu_init_w4a16_gptq_marlin_minicpm4_model": (_c_int, [_c_float] + [_c_int] * 7 + [_c_float, _c_int, _c_int, _c_int] + [_c_float] * 3 + [_c_int] * 5),
-    "cpmcu_init_layered_model": (_c_int, [_c_float, _c_int, _c_int, _c_float, _c_float] + [_c_int] * 3 + [_c_void_p]),
+    "cpmcu_init_layered_model": (_c_int, [_c_float] + [_c_int] * 3 + [_c_float] * 3 + [_c_int] * 5 + [_c_void_p]),
     "cpmcu_init_eagle_model": (_c_int, [_c_int] * 5),
     "cpmcu_init_minicpm4_eagle_model": (_c_int, [_c_int] * 9 + [_c_float, _c_int, _c_int]),
     "cpmcu_init_w4a16_gm_spec_w4a16_gm_model": (_c_int, []),
@@ -59,7 +68,9 @@ _SIGNATURES = {
     "cpmcu_profile": (_c_int, [_c_int, _c_void_p, _c_void_p]),
     "cpmcu_release": (None, []),
     "cpmcu_layer_attention": (_c_int, [_c_void_p] * 4 + [_c_int] * 5 + [_c_void_p]),
-    "cpmcu_layer_qkv_norm_append": (_c_int, [_c_void_p] * 4 + [_c_float] + [_c_int] * 4 + [_c_void_p] * 3),
+    "cpmcu_layer_qkv_norm_append": (_c_int, [_c_void_p] * 4 + [_c_float, _c_void_p] + [_c_int] * 4 + [_c_void_p] * 3),
+    "cpmcu_layer_scan": (_c_int, [_c_void_p] * 8 + [_c_int] * 3 + [_c_void_p]),
+    "cpmcu_layer_scan_state_floats": (ctypes.c_long, [_c_void_p]),
     "cpmcu_layer_out_norm": (_c_int, [_c_void_p] * 3 + [_c_float, _c_void_p] + [_c_int] * 3 + [_c_float, _c_int]),
     "cpmcu_moe_route": (_c_int, [_c_void_p] * 4 + [_c_int] * 2 + [_c_void_p] * 2),
     "cpmcu_layer_mixture": (_c_int, [_c_void_p] * 7 + [_c_float, _c_void_p] + [_c_int] * 3 + [_c_float]),
@@ -170,11 +181,16 @@ def init_w4a16_gptq_marlin_minicpm4_model(memory_limit, vocab_size, num_hidden_l
          sparse_switch, int(apply_compress_lse))
 
 
-def init_layered_model(memory_limit, vocab_size, width, norm_eps, residual_mult, torch_dtype, chunk_length, layers):
+NORM_OUTPUT_RMS, NORM_DYNAMIC_TANH = 0, 1
+REC_TIME_MIX, REC_LIGHTNING = 1, 2
+
+
+def init_layered_model(memory_limit, vocab_size, width, norm_eps, residual_mult, torch_dtype, chunk_length, layers,
+                       norm=NORM_OUTPUT_RMS, embed_scale=1.0, tied_head=False, side_dim=0):
     """layers: a list of LayerSpec."""
     arr = (LayerSpec * len(layers))(*layers)
-    call("cpmcu_init_layered_model", memory_limit, vocab_size, width, norm_eps, residual_mult, torch_dtype, chunk_length,
-         len(layers), ctypes.cast(arr, _c_void_p))
+    call("cpmcu_init_layered_model", memory_limit, vocab_size, width, norm, norm_eps, residual_mult, embed_scale, int(tied_head),
+         side_dim, torch_dtype, chunk_length, len(layers), ctypes.cast(arr, _c_void_p))
 
 
 def init_eagle_model(num_layers, num_iter, topk_per_iter, tree_size, torch_dtype):
@@ -269,9 +285,9 @@ def profile_step():
 
 def profile(on):
     """profile(True) starts per-launch timing; profile(False) stops and returns {class: (ms, launches)}."""
-    ms, cnt = (ctypes.c_float * 6)(), (ctypes.c_int * 6)()
+    ms, cnt = (ctypes.c_float * 7)(), (ctypes.c_int * 7)()
     call("cpmcu_profile", int(on), ctypes.cast(ms, _c_void_p), ctypes.cast(cnt, _c_void_p))
-    names = ("linear", "attention", "selection", "experts", "routing", "rows")
+    names = ("linear", "attention", "selection", "experts", "routing", "rows", "scan")
     return {n: (ms[i], cnt[i]) for i, n in enumerate(names)}
 
 

@@ -9,7 +9,7 @@ Additions that the reference does not have, all optional:
   * `load_state_dict_tensors()` feeds tensors that are already in memory;
   * `extend()` appends a portion of a sequence and returns the logits of chosen
     tokens of it.
-Other model designs subclass it (`tipetar.py`) and override the three hooks
+Other model designs subclass it (`layered.py`) and override the three hooks
 `_read_config`, `_create_native` and `_load`.
 """
 import glob

@@ -2,12 +2,13 @@
 import json
 import os
 
+from .fabulix import FabulixLLM
 from .llm import LLM
 from .llm_w4a16_gptq_marlin import W4A16GPTQMarlinLLM
 from .tipetar import TipetarLLM
 
 # config.json 'architecture' (or the first of 'architectures') -> class; everything else is Llama-format
-ARCHITECTURES = {"Tipetar": TipetarLLM}
+ARCHITECTURES = {"Fabulix": FabulixLLM, "Tipetar": TipetarLLM}
 
 
 def model_class(config):

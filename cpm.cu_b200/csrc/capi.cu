@@ -169,14 +169,18 @@ LayerSpec to_spec(const cpmcu_layer_spec& c) {
     s.scale = c.scale; s.window = c.window; s.bias_exp = c.bias_exp; s.qk_norm = c.qk_norm; s.kv_from = c.kv_from;
     s.experts = c.experts; s.identity = c.identity; s.top = c.top; s.groups = c.groups; s.keep_groups = c.keep_groups;
     s.router_scale = c.router_scale; s.expert_ff = c.expert_ff; s.shared_ff = c.shared_ff;
+    s.sink = c.sink; s.rot_dims = c.rot_dims; s.attn_scale = c.attn_scale;
+    s.rec = c.recurrence; s.rec_heads = c.rec_heads; s.rec_dim = c.rec_dim; s.rec_vdim = c.rec_vdim; s.rec_rank = c.rec_rank;
+    s.rec_scale = c.rec_scale;
+    s.ff = c.ff; s.ff_limit = c.ff_limit; s.ff_alpha = c.ff_alpha;
     return s;
 }
 }  // namespace
 
 extern "C" {
 
-int cpmcu_init_layered_model(float memory_limit, int vocab_size, int width, float norm_eps, float residual_mult,
-                             int torch_dtype, int chunk_length, int num_layers, const cpmcu_layer_spec* layers) {
+int cpmcu_init_layered_model(float memory_limit, int vocab_size, int width, int norm, float norm_eps, float residual_mult,
+                             float embed_scale, int tied_head, int side_dim, int torch_dtype, int chunk_length, int num_layers, const cpmcu_layer_spec* layers) {
     return guarded([&] {
         CPM_REQUIRE(torch_dtype == 1 || torch_dtype == 2, "layered models run in torch_dtype 1 (bfloat16) or 2 (float32)");
         CPM_REQUIRE(num_layers >= 1 && layers != nullptr, "layered model: no layers");
@@ -188,6 +192,10 @@ int cpmcu_init_layered_model(float memory_limit, int vocab_size, int width, floa
         mc.eps = norm_eps;
         mc.chunk_length = chunk_length;
         mc.scale_residual = residual_mult;
+        mc.norm = norm;
+        mc.scale_embed = embed_scale;
+        mc.tied_head = tied_head != 0;
+        mc.side_dim = side_dim;
         mc.fp32 = torch_dtype == 2;
         for (int i = 0; i < num_layers; ++i) mc.specs.push_back(to_spec(layers[i]));
         g_engine.reset();
@@ -744,6 +752,7 @@ int cpmcu_layer_attention(const cpmcu_layer_spec* spec, const void* q, const voi
                                                splits, sp.scale, sp.window, sp.bias_exp, static_cast<bf16*>(out), out_ld,
                                                static_cast<float*>(ws_o.p), static_cast<float*>(ws_ml.p));
             p.kv_len = static_cast<const int32_t*>(len.p);
+            p.sink = sp.sink; p.out_scale = sp.attn_scale;
             launch_tree_attention(p, s);
             sync_and_check("layer_attention");
             return 0;
@@ -753,6 +762,7 @@ int cpmcu_layer_attention(const cpmcu_layer_spec* spec, const void* q, const voi
         a.tq = tq; a.hq = sp.heads; a.hkv = sp.kv_heads; a.dk = dk; a.dv = dv; a.out_cols = sp.vdim; a.out_ld = out_ld;
         a.kv_len = static_cast<const int32_t*>(len.p); a.kv_len_add = 0;
         a.scale = sp.scale; a.window = sp.window; a.bias_exp = sp.bias_exp;
+        a.sink = sp.sink; a.out_scale = sp.attn_scale;
         if (fp32) launch_plain_attention<float>(a, s);
         else launch_plain_attention<bf16>(a, s);
         sync_and_check("layer_attention");
@@ -761,7 +771,7 @@ int cpmcu_layer_attention(const cpmcu_layer_spec* spec, const void* q, const voi
 }
 
 int cpmcu_layer_qkv_norm_append(const cpmcu_layer_spec* spec, const void* qkv, const void* wq, const void* wk, float eps,
-                                int rows, int kv_row, int cache_rows, int fp32, void* q_out, void* k_cache, void* v_cache) {
+                                const float* inv_freq, int rows, int kv_row, int cache_rows, int fp32, void* q_out, void* k_cache, void* v_cache) {
     return guarded([&] {
         const LayerSpec sp = to_spec(*spec);
         cudaStream_t s = runtime().stream;
@@ -773,6 +783,7 @@ int cpmcu_layer_qkv_norm_append(const cpmcu_layer_spec* spec, const void* qkv, c
         a.heads = sp.heads; a.kv_heads = sp.kv_heads;
         a.dim = sp.dim; a.dim_p = pad64(sp.dim); a.vdim = sp.vdim; a.vdim_p = pad64(sp.vdim);
         a.wq = static_cast<const bf16*>(wq); a.wk = static_cast<const bf16*>(wk); a.eps = eps;
+        a.rot_dims = inv_freq != nullptr ? sp.rot_dims : 0; a.inv_freq = inv_freq;
         a.q_out = q_out; a.k_cache = k_cache; a.v_cache = v_cache;
         a.kv_len = static_cast<const int32_t*>(len.p); a.kv_off = 0; a.cache_rows = cache_rows; a.error = runtime().d_error;
         if (fp32) launch_qkv_norm_append<float>(a, rows, s);
@@ -792,6 +803,35 @@ int cpmcu_layer_out_norm(float* x32, void* xh, const void* delta, float mult, co
         sync_and_check("layer_out_norm");
         return 0;
     });
+}
+
+int cpmcu_layer_scan(const cpmcu_layer_spec* spec, const void* r, const void* k, const void* v, const float* w, const float* decay,
+                     const void* bonus, float* state, int rows, int position, int fp32, float* out) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        CPM_REQUIRE(sp.rec != REC_NONE && scan_fits(sp.rec_dim, sp.rec_vdim) && rows >= 1, "layer_scan: bad sizes");
+        cudaStream_t s = runtime().stream;
+        DeviceBuf len(4), ws(scan_workspace_floats(sp.rec_heads, sp.rec_dim, sp.rec_vdim, rows) * 4);
+        CUDA_CHECK(cudaMemcpyAsync(len.p, &position, 4, cudaMemcpyHostToDevice, s));
+        ScanArgs a;
+        a.r = r; a.k = k; a.v = v;
+        a.heads = sp.rec_heads; a.dim = sp.rec_dim; a.vdim = sp.rec_vdim; a.rows = rows;
+        a.ld_r = a.ld_k = sp.rec_heads * sp.rec_dim; a.ld_v = a.ld_out = sp.rec_heads * sp.rec_vdim;
+        a.silu = sp.rec == REC_LIGHTNING;
+        a.w = w; a.ld_w = a.ld_k; a.decay = decay; a.bonus = static_cast<const bf16*>(bonus);
+        a.state = state; a.ws = static_cast<float*>(ws.p);
+        a.kv_len = static_cast<const int32_t*>(len.p);
+        a.out = out;
+        if (fp32) launch_scan<float>(a, s);
+        else launch_scan<bf16>(a, s);
+        sync_and_check("layer_scan");
+        return 0;
+    });
+}
+
+long cpmcu_layer_scan_state_floats(const cpmcu_layer_spec* spec) {
+    const LayerSpec sp = to_spec(*spec);
+    return static_cast<long>(scan_state_floats(sp.rec_heads, sp.rec_dim, sp.rec_vdim));
 }
 
 }  // extern "C"

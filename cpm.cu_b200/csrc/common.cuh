@@ -55,6 +55,7 @@ enum KernelError : int {
     ERR_BAD_TREE = 4,
     ERR_KV_OVERFLOW = 8,  // a K/V row beyond the cache budget was about to be written (the store is skipped)
     ERR_BAD_TOKEN = 16,   // a token id outside the vocabulary (token 0 was used in its place)
+    ERR_STATE_POS = 32,   // a pass that does not begin where the recurrent state stands (nor at position 0)
 };
 
 enum KernelClass : int {
@@ -64,7 +65,8 @@ enum KernelClass : int {
     KC_MOE = 3,   // grouped expert products
     KC_ROUTE = 4, // router, row layout and gather of a mixture of experts
     KC_ROW = 5,   // row-wise kernels of layered models
-    KC_COUNT = 6
+    KC_SCAN = 6,  // recurrences
+    KC_COUNT = 7
 };
 
 struct Runtime {
@@ -189,6 +191,13 @@ __device__ __forceinline__ float silu_mul(float g, float u) {
     return g * s * u;
 }
 
+// g sigmoid(alpha g) (u + 1) with g cut off above `limit` and u on both sides
+__device__ __forceinline__ float clamped_gate(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+
 struct LinearPlan {
     CUtensorMap tm_w;   // W  [N,K], box 64 x 128
     CUtensorMap tm_x;   // X  [Mrows,K], box 64 x MT
@@ -205,6 +214,7 @@ struct LinearPlan {
     int wave_tiles = 0;          // several token tiles: tiles computed whole, in waves of `grid` (the rest is cut along K)
     int tail_grid = 0;           // CTAs that share the tiles after wave_tiles (0 = all)
     int swiglu = 0;              // SwiGLU epilogue: w = [gate ; up], N = output features, y = silu(gate) * up
+    float gate_limit = 0.f, gate_alpha = 0.f;   // gate_limit > 0: clamped_gate instead of silu_mul
     // W4A16: when wq is set the weights are 4-bit blocks in the streaming layout (see gemm_w4_umma.cu)
     const void* wq = nullptr;
 };
@@ -294,6 +304,8 @@ struct AttnPlan {
     bool biased = false;              // made by make_biased_attn_plan
     int exact_window = 0;             // biased plans: > 0 = per-token sliding window (tokens)
     float bias_exp = 0.f;             // biased plans: > 0 = distance bias with slopes 2^(-bias_exp * (h + 1) / hq)
+    int sink = 0;                     // 1: one more score of 0, without a value, in every softmax
+    float out_scale = 1.f;            // factor of the output
     int splits = 1;
     const int32_t* kv_len = nullptr;  // device scalar
     int kv_len_add = 0;               // keys visible = *kv_len + kv_len_add

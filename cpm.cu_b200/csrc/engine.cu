@@ -653,7 +653,7 @@ void Engine::prefill_rows(int n, int history, const int32_t* ids, const int32_t*
         // CUDA events around every launch of the pass: time per kernel class, and the GEMMs of the last layer
         rt.profile = false;
         CUDA_CHECK(cudaStreamSynchronize(s));
-        const char* names[KC_COUNT] = {"linear", "attention", "other", "experts", "route", "rows"};
+        const char* names[KC_COUNT] = {"linear", "attention", "other", "experts", "route", "rows", "scan"};
         for (int k = 0; k < KC_COUNT; ++k) {
             double sum = 0.0;
             std::vector<float> each;
@@ -937,7 +937,8 @@ void Engine::check_errors(const char* where) {
         }
         throw std::runtime_error(std::string("cpmcu_b200: kernel error flags ") + std::to_string(e) + " raised in " +
                                  where + " (1 = GEMM pipeline timeout, 2 = attention pipeline timeout, 4 = malformed draft tree, "
-                                 "8 = K/V row beyond the cache budget, 16 = token id outside the vocabulary)");
+                                 "8 = K/V row beyond the cache budget, 16 = token id outside the vocabulary, 32 = tokens that do not "
+                                 "follow those the recurrent state has seen)");
     }
 }
 

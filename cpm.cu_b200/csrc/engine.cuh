@@ -6,6 +6,7 @@
 // drafters (EagleImpl src/model/eagle.cuh:262-516, MiniCPM4EagleImpl
 // src/model/minicpm4/minicpm4_eagle.cuh:10-418).
 #pragma once
+#include <algorithm>
 #include <map>
 #include <memory>
 #include <set>
@@ -30,6 +31,9 @@ struct ModelConfig {
     // sublayers' outputs, a 32-bit residual stream scaled by scale_residual
     std::vector<LayerSpec> specs;
     bool fp32 = false;    // activations, caches and logits in fp32 (layered models only)
+    int norm = NORM_OUTPUT_RMS;
+    bool tied_head = false;   // the head is the embedding table
+    int side_dim = 0;         // > 0: every layer adds an input of its own for each token, this wide inside
 };
 
 struct EagleConfig {
@@ -62,19 +66,47 @@ struct KVLayer {
 
 // One layer of a layered model.  bf16 models keep the matrices tile-major (linear_weight_elems), fp32 models row-major.
 struct LayeredWeights {
-    bf16 *qkv = nullptr, *o = nullptr;          // rows q | k | v (q alone with kv_from); o: K = pad64(heads * vdim)
+    bf16* qkv = nullptr;                        // rows q | k | v (q alone with kv_from)
+    bf16* o = nullptr;                          // columns: pad64(heads * vdim) of the attention, then pad64 of the recurrence's
     bf16 *q_norm = nullptr, *k_norm = nullptr, *norm1 = nullptr, *norm2 = nullptr;
     bf16* router = nullptr;                     // [outputs][ld]
     float* correction = nullptr;                // [outputs]
-    bf16 *gate_up = nullptr, *down = nullptr;   // expert after expert, the shared expert last
+    bf16 *gate_up = nullptr, *down = nullptr;   // expert after expert, the shared expert last; or the dense feed-forward's
     void *k = nullptr, *v = nullptr;            // cache rows [budget][kv_heads][pad64(dim) | pad64(vdim)]; kv_from: that layer's
+    float* inv_freq = nullptr;                  // [rot_dims / 2]
+    // dynamic tanh norms before (1, 2) and after (1b, 2b) the sublayers
+    DynTanh tanh1, tanh1b, tanh2, tanh2b;
+    // recurrence.  Time mix: the matrices r, k, v, g one after the other (rec_part elements each), then w1; lightning: one
+    // matrix with rows q | k | v | g
+    bf16* rec_proj = nullptr;
+    size_t rec_part = 0;
+    bf16* w2 = nullptr;                         // [rec_heads * rec_dim][rec_rank], row-major
+    bf16 *w0 = nullptr, *bonus = nullptr, *rec_norm = nullptr;
+    bf16* mu = nullptr;                         // [kMixes][ld]
+    float* decay = nullptr;                     // [rec_heads]
+    float *state = nullptr, *prev = nullptr;    // the recurrent state, and the last token's mixer input
+    // token side input
+    bf16 *side_gate = nullptr, *side_proj = nullptr, *side_norm = nullptr;
+};
+// y[rows][ldy] = x[rows][K] w^T, N columns
+struct LayeredProduct {
+    const void* x = nullptr;
+    const bf16* w = nullptr;
+    int N = 0, K = 0;
+    void* y = nullptr;
+    int ldy = 0;
+    LinearPlan plan;   // bf16
 };
 struct LayeredPlans {
     struct Layer {
-        LinearPlan qkv, o;
+        LayeredProduct qkv, o;
         AttnPlan attn;
         bool tensor_attn = false;   // head widths the tensor-core attention kernel takes
         MoeGemmPlan gate_up, down;
+        std::vector<LayeredProduct> rec;   // lightning: one product; fp32 time mix: r, k, v, g, w1
+        MoeGemmPlan mixes;                 // bf16 time mix: the five in one launch
+        LayeredProduct ff_gate_up, ff_down, side_gate, side_proj;
+        bool ff_fused = false;      // the activation is in the epilogue of ff_gate_up
     };
     int rows = 0, tile = 0;
     std::vector<Layer> layers;
@@ -182,6 +214,29 @@ private:
     void layered_forward(int rows, const int32_t* ids, const int32_t* kv_len, int kv_off, cudaStream_t s);
     template <typename T>
     void layered_mixture(int layer, LayeredPlans& lp, cudaStream_t s);
+    // attention of lx_ and / or the recurrence of its mixes; the outputs lie side by side in lattn_
+    template <typename T>
+    void layered_attention(int layer, LayeredPlans& lp, const int32_t* kv_len, int kv_off, cudaStream_t s);
+    template <typename T>
+    void layered_recurrence(int layer, LayeredPlans& lp, const int32_t* kv_len, int kv_off, cudaStream_t s);
+    template <typename T>
+    void layered_dense(int layer, LayeredPlans& lp, cudaStream_t s);
+    // a layer of a dynamic tanh model from the mixer on: lx_ (and the mixes) hold its first norm already; leaves those of
+    // the next layer where it can (returns whether it did)
+    template <typename T>
+    bool layered_tanh_layer(int layer, LayeredPlans& lp, const int32_t* ids, const int32_t* kv_len, int kv_off, cudaStream_t s);
+    TokenShift token_shift(int layer, int rows, const int32_t* kv_len, int kv_off) const;
+    template <typename T>
+    void run_product(const LayeredProduct& p, int rows, cudaStream_t s);
+    bool has_recurrence() const;
+    void layered_check_errors(const char* where);
+    // columns of a row of the recurrence's projections
+    static int rec_ld(const LayerSpec& s) {
+        return s.rec == REC_TIME_MIX ? pad64(std::max(s.rec_heads * s.rec_dim, s.rec_rank)) : pad64(2 * s.rec_heads * (s.rec_dim + s.rec_vdim));
+    }
+    // columns of the o product: attention's, then the recurrence's
+    static int o_left(const LayerSpec& s) { return s.heads > 0 ? pad64(s.heads * s.vdim) : 0; }
+    static int o_cols(const LayerSpec& s) { return o_left(s) + (s.rec != REC_NONE ? pad64(s.rec_heads * s.rec_vdim) : 0); }
     // logits of n stream rows (rows_idx: device list, null = rows 0..n)
     template <typename T>
     void layered_logits(const int32_t* rows_idx, int n, void* out, cudaStream_t s);
@@ -278,6 +333,12 @@ private:
     void *moe_x_ = nullptr, *moe_gu_ = nullptr, *moe_act_ = nullptr, *moe_y_ = nullptr;
     size_t moe_rows_ = 0;                             // rows of moe_x_ / moe_act_ / moe_y_
     MoeBuffers moe_;
+    void *lmix_ = nullptr, *lrec_ = nullptr;          // [kMixes][rows][ld] and the projections of a recurrence
+    float *ldecay_ = nullptr, *lo_ = nullptr, *rec_ws_ = nullptr;   // decays [R][channels], outputs of a recurrence
+    void *lgu_ = nullptr, *lact_ = nullptr, *lside_ = nullptr, *lsg_ = nullptr;
+    bf16* side_embed_ = nullptr;                      // [vocab][layers * side_dim]
+    DynTanh tanh_final_;
+    int32_t* state_len_ = nullptr;                    // tokens the recurrent states hold
     int32_t* want_ = nullptr;                         // [R] rows whose logits are asked for
     float* layer_capture_ = nullptr;
     cudaGraphExec_t decode_graph_ = nullptr;          // one-token decode for the pointers below

@@ -27,6 +27,7 @@ struct LinearArgs {
     // SwiGLU epilogue (whole tiles only): a weight tile is 64 gate rows followed by the 64 up rows of the same
     // features, N counts output features (the gate half), y[token][feature] = silu(gate) * up.
     int swiglu = 0;
+    float gate_limit = 0.f, gate_alpha = 0.f;   // > 0: clamped_gate of the fp32 projections instead of silu_mul
     int band = 16;   // token tiles per raster band (tile_to_mn)
 };
 
@@ -279,7 +280,8 @@ __device__ __forceinline__ void run_epilogue(const LinearArgs& a, SegIter it, ui
                 if (q < 2) {
 #pragma unroll
                     for (int c = 0; c < 16; ++c) {
-                        xb[(q * 16 + c) * 32 + lane] = __bfloat162float(__float2bfloat16(__uint_as_float(r[c])));
+                        const float gv = __uint_as_float(r[c]);
+                        xb[(q * 16 + c) * 32 + lane] = a.gate_limit > 0.f ? gv : __bfloat162float(__float2bfloat16(gv));
                     }
                 }
                 // the batch after the next one reuses this buffer: its writers pass the next batch's barrier only
@@ -289,9 +291,11 @@ __device__ __forceinline__ void run_epilogue(const LinearArgs& a, SegIter it, ui
 #pragma unroll
                     for (int c = 0; c < 16; ++c) {
                         if (c0 + c < m_cnt) {
-                            const float uv = __bfloat162float(__float2bfloat16(__uint_as_float(r[c])));
+                            const float uv = __uint_as_float(r[c]);
                             const float gv = xb[((q - 2) * 16 + c) * 32 + lane];
-                            a.y[static_cast<size_t>(m_base + c0 + c) * a.ldy + n_out] = __float2bfloat16(silu_mul(gv, uv));
+                            const float av = a.gate_limit > 0.f ? clamped_gate(gv, uv, a.gate_limit, a.gate_alpha)
+                                                                : silu_mul(gv, __bfloat162float(__float2bfloat16(uv)));
+                            a.y[static_cast<size_t>(m_base + c0 + c) * a.ldy + n_out] = __float2bfloat16(av);
                         }
                     }
                 }

@@ -655,6 +655,7 @@ void launch_linear(const LinearPlan& p, cudaStream_t stream) {
     a.wave_tiles = p.wave_tiles;
     a.tail_grid = p.tail_grid;
     a.swiglu = p.swiglu;
+    a.gate_limit = p.gate_limit; a.gate_alpha = p.gate_alpha;
     a.band = raster_band(p.mt, p.K);
     if (p.swiglu) {   // N = output features; a tile covers 64 of them (gate + up rows)
         a.n_tiles = ceil_div(p.N, 64);

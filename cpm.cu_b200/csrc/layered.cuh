@@ -10,29 +10,64 @@
 #pragma once
 #include "common.cuh"
 
+enum RecurrenceKind : int {
+    REC_NONE = 0,
+    REC_TIME_MIX = 1,    // decay per token and key channel, bonus for the current token, inputs mixed with the token before
+    REC_LIGHTNING = 2,   // constant decay per head, silu on queries, keys and values
+};
+
 struct LayerSpec {
-    // ---- mixer: softmax attention
+    // ---- mixer: softmax attention (heads == 0: none) and / or a recurrence; with both, they read the same input side by
+    // side and their outputs are added
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
     float scale = 0.f;
     int window = 0;          // > 0: a token sees itself and the window - 1 tokens before it
     float bias_exp = 0.f;    // > 0: distance bias, slope of head h = 2^(-bias_exp * (h + 1) / heads)
     int qk_norm = 0;         // RMS norm over all query rows and over all key rows at once, before the split into heads
     int kv_from = -1;        // >= 0: the keys and values of that layer's cache
+    int sink = 0;            // one more score of 0, without a value, in every softmax
+    int rot_dims = 0;        // > 0: rotary positions on the first rot_dims of each query and key head (i paired with i + rot_dims / 2)
+    float attn_scale = 1.f;  // factor of the attention's output
+    int rec = REC_NONE;
+    int rec_heads = 0, rec_dim = 0, rec_vdim = 0;   // key / query and value width of a head
+    int rec_rank = 0;        // REC_TIME_MIX: inner width of the decay's two matrices
+    float rec_scale = 1.f;   // factor of the recurrence's output
     // ---- feed-forward: mixture of experts (experts + identity == 0: none)
     int experts = 0, identity = 0, top = 0, groups = 1, keep_groups = 1;
     float router_scale = 1.f;
     int expert_ff = 0;
     int shared_ff = 0;       // > 0: an expert of this width that runs for every token
+    // ---- feed-forward: one dense one (ff == 0: none), y = g sigmoid(ff_alpha g) (u + 1) with g <= ff_limit, |u| <= ff_limit
+    int ff = 0;
+    float ff_limit = 0.f, ff_alpha = 0.f;
+};
+
+// Norms of a layered model
+enum NormKind : int {
+    NORM_OUTPUT_RMS = 0,     // x += m * rms(sublayer(x)) * (1 + w)
+    NORM_DYNAMIC_TANH = 1,   // x += N'(sublayer(N(x))), N(x) = tanh(alpha x) * w + b
+};
+struct DynTanh {
+    const bf16 *w = nullptr, *b = nullptr;
+    float alpha = 0.f;
 };
 
 inline int pad64(int n) { return (n + 63) / 64 * 64; }
 
 // ---------------------------------------------------------------- rows (layered_ops.cu)
-// x32 = embed[id] (fp32), xh the same in T; `ld` columns per row.  Ids outside [0, vocab) raise ERR_BAD_TOKEN.
+// x32 = embed[id] * scale (fp32), xh the same in T; `ld` columns per row.  Ids outside [0, vocab) raise ERR_BAD_TOKEN.
+// state_len (models with recurrent layers): tokens the recurrent state holds; the pass must begin there (*kv_len + kv_off)
+// or at 0, otherwise ERR_STATE_POS; advanced by `rows`.
+struct StateCheck {
+    int32_t* state_len = nullptr;
+    const int32_t* kv_len = nullptr;
+    int kv_off = 0;
+};
 template <typename T>
-void launch_embed_rows(const int32_t* ids, const bf16* table, int vocab, float* x32, T* xh, int ld, int rows, cudaStream_t s);
+void launch_embed_rows(const int32_t* ids, const bf16* table, int vocab, float scale, float* x32, T* xh, int ld, int rows,
+                       const StateCheck& check, cudaStream_t s);
 
-// Query / key norm over the whole projections, then queries to q_out[rows][heads][dim_p] and keys / values to rows
+// Query / key norm over the whole projections, rotation, then queries to q_out[rows][heads][dim_p] and keys / values to rows
 // *kv_len + kv_off + r of the caches ([.][kv_heads][dim_p], [.][kv_heads][vdim_p]).  qkv: [rows][ld] q | k | v.
 struct QkvNormArgs {
     const void* qkv;
@@ -40,6 +75,8 @@ struct QkvNormArgs {
     int heads, kv_heads, dim, dim_p, vdim, vdim_p;
     const bf16 *wq, *wk;     // null: no norm
     float eps;
+    int rot_dims = 0;        // rotated dimensions per query / key head; the position is the cache row
+    const float* inv_freq = nullptr;   // [rot_dims / 2]
     void* q_out;
     void *k_cache, *v_cache; // null: queries only
     const int32_t* kv_len;
@@ -69,6 +106,72 @@ template <typename T>
 void launch_norm_rows(const float* x32, const int32_t* rows_idx, const bf16* w, T* y, int rows, int width, int ld, float eps,
                       cudaStream_t s);
 
+// ---- dynamic tanh models
+// What a time-mix layer reads instead of h itself: out[s][r] = h + (h_before - h) * mu[s], s = r, k, v, g, w; h_before is the
+// row before, or `prev` ([ld] fp32, written with the last row's h) for the first row, zero at position 0.
+constexpr int kMixes = 5;
+struct TokenShift {
+    const bf16* mu = nullptr;    // [kMixes][ld]; null: no mixes
+    void* out = nullptr;         // [kMixes][stride] T
+    size_t stride = 0;           // elements between two mixes
+    float* prev = nullptr;
+    const int32_t* kv_len = nullptr;   // position of the first row = *kv_len + kv_off
+    int kv_off = 0;
+};
+// h[i] = N(x32[rows_idx ? rows_idx[i] : i]) in T, and the mixes
+template <typename T>
+void launch_tanh_norm(const float* x32, const int32_t* rows_idx, const DynTanh& n, T* h, const TokenShift& shift, int rows, int ld,
+                      cudaStream_t s);
+// x32 += post(delta); out = next(x32) in T, or x32 itself where next has no weights
+template <typename T>
+void launch_tanh_residual(float* x32, const T* delta, const DynTanh& post, const DynTanh& next, T* out, int rows, int ld, cudaStream_t s);
+// act = clamped gate of gu (two blocks of ff columns, or interleaved in groups of 64: see launch_silu_gate)
+template <typename T>
+void launch_clamped_gate(const T* gu, int ld_gu, T* act, int ld_act, int rows, int ff, float limit, float alpha, bool interleaved, cudaStream_t s);
+// Token side input: g[r] = gelu_tanh(z[r]) * table[ids[r]][col0 ..], dim columns, zero up to ld
+template <typename T>
+void launch_side_gate(const T* z, int ld, const int32_t* ids, const bf16* table, int table_ld, int col0, int dim, int vocab, T* g, int rows,
+                      cudaStream_t s);
+// x32 += rms(y) * w; with `next`, h = next(x32) in T and, for a single row, its mixes
+template <typename T>
+void launch_side_add(float* x32, const T* y, const bf16* w, const DynTanh& next, T* h, const TokenShift& shift, int rows, int width, int ld,
+                     float eps, cudaStream_t s);
+// Decays of a time-mix layer: out[r][c] = exp(-exp(w2[c] . tanh(x[r]) + w0[c])), c < channels; x: `rank` columns of T, w2
+// [channels][rank]
+template <typename T>
+void launch_decay(const T* x, int ld_x, const bf16* w2, const bf16* w0, int rank, int channels, float* out, int ld_out, int rows, cudaStream_t s);
+// out[r][c] = rms over each group of `group` columns of o[r] * w[c] * gate(g[r][c]) * scale; gate: silu, or sigmoid
+template <typename T>
+void launch_norm_gate(const float* o, int ld_o, int groups, int group, const bf16* w, const T* gate, int ld_gate, bool silu, float eps,
+                      float scale, T* out, int ld_out, int rows, cudaStream_t s);
+
+// ---------------------------------------------------------------- recurrences (recurrence.cu)
+// Per head, with a state S [dim][vdim] in fp32:
+//   bonus != null:  o_t = (S + diag(u) k_t v_t^T)^T r_t,  then S = diag(w_t) S + k_t v_t^T
+//   bonus == null:  S = diag(w_t) S + k_t v_t^T,  then o_t = S^T r_t
+// w_t is given per token and channel, or constant per head.  Everything is fp32 from r, k, v on.
+struct ScanArgs {
+    const void *r = nullptr, *k = nullptr, *v = nullptr;   // T, head after head in a row
+    int ld_r = 0, ld_k = 0, ld_v = 0;
+    bool silu = false;             // r, k, v pass through silu first
+    const float* w = nullptr;      // [rows][ld_w] decays, channel h * dim + c; null: constant decay
+    int ld_w = 0;
+    const float* decay = nullptr;  // [heads]
+    const bf16* bonus = nullptr;   // [heads * dim]
+    int heads = 0, dim = 0, vdim = 0, rows = 0;
+    float* state = nullptr;        // scan_state_floats(heads, dim, vdim)
+    const int32_t* kv_len = nullptr;   // position of the first row = *kv_len + kv_off; at 0 the state starts at zero
+    int kv_off = 0;
+    float* out = nullptr;          // [rows][ld_out], column h * vdim + c
+    int ld_out = 0;
+    float* ws = nullptr;           // scan_workspace_floats(heads, dim, vdim, rows)
+};
+bool scan_fits(int dim, int vdim);
+size_t scan_state_floats(int heads, int dim, int vdim);
+size_t scan_workspace_floats(int heads, int dim, int vdim, int rows);
+template <typename T>
+void launch_scan(const ScanArgs& a, cudaStream_t s);
+
 // Attention of any head width up to 512, one warp per (token, head); q [tq][hq][dk], caches [.][hkv][dk | dv], out rows
 // of hq * out_cols.  The bias, window and kv_len arguments are those of make_biased_attn_plan.
 struct PlainAttnArgs {
@@ -80,6 +183,8 @@ struct PlainAttnArgs {
     float scale;
     int window;
     float bias_exp;
+    int sink = 0;
+    float out_scale = 1.f;
 };
 template <typename T>
 void launch_plain_attention(const PlainAttnArgs& a, cudaStream_t s);
@@ -140,7 +245,12 @@ struct MoeGemmPlan {
     int ldy = 0;
     const int4* entries = nullptr;
     const int32_t* n_entries = nullptr;
+    int uniform = 0;                 // > 0: no router, this many matrices whose rows lie one block of `rows` after the other
 };
+// `n` products of the same shape in one launch: rows [i * rows, (i + 1) * rows) of x times matrix i [N][K], into the same rows
+// of y; with N_s > 0 one more, of N_s outputs, on rows n * rows ... .  w: linear_weight_elems(N, K) per matrix, the extra one
+// last.
+MoeGemmPlan make_grouped_plan(const bf16* w, int n, int N, int N_s, int K, const bf16* x, bf16* y, int ldy, int rows);
 // gate/up with the SwiGLU epilogue: y[row][ff_p columns]; x rows of K = ld columns
 MoeGemmPlan make_moe_gate_up_plan(const LayerSpec& sp, const bf16* w, const bf16* x, int x_rows, const bf16* xs, int K, bf16* act,
                                   int ld_act, int rows, int tile, const MoeBuffers& b);

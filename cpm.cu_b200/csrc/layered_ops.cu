@@ -2,77 +2,21 @@
 // sum, attention scores and weights are fp32 whatever T is.
 #include <algorithm>
 
-#include "layered.cuh"
+#include "row_ops.cuh"
 
 namespace {
 
 template <typename T>
-__device__ __forceinline__ float to_float(T v);
-template <>
-__device__ __forceinline__ float to_float<float>(float v) { return v; }
-template <>
-__device__ __forceinline__ float to_float<bf16>(bf16 v) { return __bfloat162float(v); }
-template <typename T>
-__device__ __forceinline__ T from_float(float v);
-template <>
-__device__ __forceinline__ float from_float<float>(float v) { return v; }
-template <>
-__device__ __forceinline__ bf16 from_float<bf16>(float v) { return __float2bfloat16(v); }
-
-// VEC consecutive elements (8: 16-byte accesses)
-template <int VEC, typename T>
-__device__ __forceinline__ void load_vec(const T* p, float* f) {
-    if constexpr (VEC == 8 && sizeof(T) == 2) {
-        const uint4 v = *reinterpret_cast<const uint4*>(p);
-        const bf16* e = reinterpret_cast<const bf16*>(&v);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = __bfloat162float(e[i]);
-    } else if constexpr (VEC == 8) {
-        const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-        f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-        f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-    } else {
-        f[0] = to_float<T>(*p);
-    }
-}
-template <int VEC, typename T>
-__device__ __forceinline__ void store_vec(T* p, const float* f) {
-    if constexpr (VEC == 8 && sizeof(T) == 2) {
-        uint4 v;
-        bf16* e = reinterpret_cast<bf16*>(&v);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) e[i] = __float2bfloat16(f[i]);
-        *reinterpret_cast<uint4*>(p) = v;
-    } else if constexpr (VEC == 8) {
-        *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-        *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
-    } else {
-        *p = from_float<T>(f[0]);
-    }
-}
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-// sums of two values over the CTA; sh: 64 floats
-__device__ __forceinline__ float2 block_sum2(float a, float b, float* sh) {
-    a = warp_sum(a);
-    b = warp_sum(b);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-    if (lane == 0) { sh[warp] = a; sh[32 + warp] = b; }
-    __syncthreads();
-    a = warp_sum(lane < nw ? sh[lane] : 0.f);
-    b = warp_sum(lane < nw ? sh[32 + lane] : 0.f);
-    return make_float2(a, b);
-}
-
-template <typename T>
-__global__ void embed_rows_kernel(const int32_t* __restrict__ ids, const bf16* __restrict__ table, int vocab, float* __restrict__ x32,
-                                  T* __restrict__ xh, int ld, int* __restrict__ error) {
+__global__ void embed_rows_kernel(const int32_t* __restrict__ ids, const bf16* __restrict__ table, int vocab, float scale, float* __restrict__ x32,
+                                  T* __restrict__ xh, int ld, const StateCheck check, int* __restrict__ error) {
     grid_dependency_sync();
     const size_t row = blockIdx.x;
+    if (check.state_len != nullptr && row == 0 && threadIdx.x == 0) {
+        const int first = *check.kv_len + check.kv_off;
+        const bool ok = first == 0 || first == *check.state_len;
+        if (!ok) atomicOr(error, ERR_STATE_POS);
+        *check.state_len = ok ? first + static_cast<int>(gridDim.x) : -1;
+    }
     int id = ids[row];
     if (id < 0 || id >= vocab) {
         if (threadIdx.x == 0) atomicOr(error, ERR_BAD_TOKEN);
@@ -82,6 +26,8 @@ __global__ void embed_rows_kernel(const int32_t* __restrict__ ids, const bf16* _
     for (int c = threadIdx.x * 8; c < ld; c += blockDim.x * 8) {
         float f[8];
         load_vec<8>(src + c, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] *= scale;
         store_vec<8>(x32 + row * ld + c, f);
         store_vec<8>(xh + row * ld + c, f);
     }
@@ -92,6 +38,7 @@ template <typename T, int VEC>
 __global__ void qkv_norm_append_kernel(const QkvNormArgs a) {
     grid_dependency_sync();
     __shared__ float sh[64];
+    __shared__ float2 turn[256];   // cos, sin of the row's angles
     const int r = blockIdx.x;
     const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
     const T* row = static_cast<const T*>(a.qkv) + static_cast<size_t>(r) * a.ld;
@@ -99,6 +46,16 @@ __global__ void qkv_norm_append_kernel(const QkvNormArgs a) {
     const long long kv_row = own_kv ? static_cast<long long>(*a.kv_len) + a.kv_off + r : 0;
     const bool store_kv = own_kv && kv_row >= 0 && kv_row < a.cache_rows;
     if (own_kv && !store_kv && threadIdx.x == 0) atomicOr(a.error, ERR_KV_OVERFLOW);
+    const int half = a.rot_dims / 2;
+    if (half > 0) {
+        const float pos = static_cast<float>(*a.kv_len + a.kv_off + r);
+        for (int i = threadIdx.x; i < half; i += blockDim.x) {
+            float sn, cs;
+            sincosf(pos * a.inv_freq[i], &sn, &cs);
+            turn[i] = make_float2(cs, sn);
+        }
+        __syncthreads();
+    }
     float rq = 1.f, rk = 1.f;
     if (a.wq != nullptr) {
         float sq = 0.f, sk = 0.f, f[VEC];
@@ -118,7 +75,7 @@ __global__ void qkv_norm_append_kernel(const QkvNormArgs a) {
         rq = rsqrtf(t.x / nq + a.eps);
         if (own_kv) rk = rsqrtf(t.y / nk + a.eps);
     }
-    auto place = [&](const T* src, const bf16* w, float rs, int n_heads, int d, int dp, T* dst, bool pad) {
+    auto place = [&](const T* src, const bf16* w, float rs, int n_heads, int d, int dp, T* dst, bool pad, int rot) {
         const int per = (pad ? dp : d) / VEC;
         for (int i = threadIdx.x; i < n_heads * per; i += blockDim.x) {
             const int h = i / per, c = (i - h * per) * VEC;
@@ -131,6 +88,23 @@ __global__ void qkv_norm_append_kernel(const QkvNormArgs a) {
 #pragma unroll
                     for (int e = 0; e < VEC; ++e) f[e] = f[e] * rs * g[e];
                 }
+                if (c < 2 * rot) {   // rot is a multiple of VEC
+                    const bool upper = c >= rot;
+                    const int other = upper ? c - rot : c + rot, i0 = upper ? c - rot : c;
+                    float p[VEC];
+                    load_vec<VEC>(src + h * d + other, p);
+                    if (w != nullptr) {
+                        float g[VEC];
+                        load_vec<VEC>(w + h * d + other, g);
+#pragma unroll
+                        for (int e = 0; e < VEC; ++e) p[e] = p[e] * rs * g[e];
+                    }
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        const float2 cs = turn[i0 + e];
+                        f[e] = upper ? f[e] * cs.x + p[e] * cs.y : f[e] * cs.x - p[e] * cs.y;
+                    }
+                }
             } else {
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) f[e] = 0.f;
@@ -139,12 +113,12 @@ __global__ void qkv_norm_append_kernel(const QkvNormArgs a) {
         }
     };
     // the query buffer is shared by layers of different widths, so its padding is written; a cache's padding stays zero
-    place(row, a.wq, rq, a.heads, a.dim, a.dim_p, static_cast<T*>(a.q_out) + static_cast<size_t>(r) * a.heads * a.dim_p, true);
+    place(row, a.wq, rq, a.heads, a.dim, a.dim_p, static_cast<T*>(a.q_out) + static_cast<size_t>(r) * a.heads * a.dim_p, true, half);
     if (store_kv) {
         place(row + nq, a.wk, rk, a.kv_heads, a.dim, a.dim_p,
-              static_cast<T*>(a.k_cache) + static_cast<size_t>(kv_row) * a.kv_heads * a.dim_p, false);
+              static_cast<T*>(a.k_cache) + static_cast<size_t>(kv_row) * a.kv_heads * a.dim_p, false, half);
         place(row + nq + nk, nullptr, 1.f, a.kv_heads, a.vdim, a.vdim_p,
-              static_cast<T*>(a.v_cache) + static_cast<size_t>(kv_row) * a.kv_heads * a.vdim_p, false);
+              static_cast<T*>(a.v_cache) + static_cast<size_t>(kv_row) * a.kv_heads * a.vdim_p, false, 0);
         (void)nv;
     }
 }
@@ -312,7 +286,8 @@ __global__ void plain_attention_kernel(const PlainAttnArgs a) {
         }
     }
     T* out = static_cast<T*>(a.out) + static_cast<size_t>(t) * a.out_ld + static_cast<size_t>(h) * a.out_cols;
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    if (a.sink != 0) l += expf(-m);
+    const float inv = l > 0.f ? a.out_scale / l : 0.f;
 #pragma unroll
     for (int c = 0; c < PA_MAX_D / 32; ++c) {
         if (c * 32 + lane < a.out_cols) out[c * 32 + lane] = from_float<T>(acc[c] * inv);
@@ -381,15 +356,17 @@ __global__ void silu_f32_kernel(const float* __restrict__ gu, int ld_gu, float* 
 }  // namespace
 
 template <typename T>
-void launch_embed_rows(const int32_t* ids, const bf16* table, int vocab, float* x32, T* xh, int ld, int rows, cudaStream_t s) {
+void launch_embed_rows(const int32_t* ids, const bf16* table, int vocab, float scale, float* x32, T* xh, int ld, int rows,
+                       const StateCheck& check, cudaStream_t s) {
     ProfileScope prof(KC_ROW, s);
-    launch_kernel(embed_rows_kernel<T>, dim3(rows), dim3(128), 0, s, ids, table, vocab, x32, xh, ld, runtime().d_error);
+    launch_kernel(embed_rows_kernel<T>, dim3(rows), dim3(128), 0, s, ids, table, vocab, scale, x32, xh, ld, check, runtime().d_error);
 }
 
 template <typename T>
 void launch_qkv_norm_append(const QkvNormArgs& a, int rows, cudaStream_t s) {
     ProfileScope prof(KC_ROW, s);
-    const bool v8 = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0;
+    CPM_REQUIRE(a.rot_dims % 2 == 0 && a.rot_dims <= a.dim && a.rot_dims <= 512, "layered model: bad number of rotated dimensions");
+    const bool v8 = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && (a.rot_dims / 2) % 8 == 0;
     if (v8) launch_kernel(qkv_norm_append_kernel<T, 8>, dim3(rows), dim3(256), 0, s, a);
     else launch_kernel(qkv_norm_append_kernel<T, 1>, dim3(rows), dim3(256), 0, s, a);
 }
@@ -440,7 +417,7 @@ void launch_silu_f32(const float* gu, int ld_gu, float* act, int ld_act, int row
 }
 
 #define CPM_INSTANTIATE(T)                                                                                                          \
-    template void launch_embed_rows<T>(const int32_t*, const bf16*, int, float*, T*, int, int, cudaStream_t);                       \
+    template void launch_embed_rows<T>(const int32_t*, const bf16*, int, float, float*, T*, int, int, const StateCheck&, cudaStream_t); \
     template void launch_qkv_norm_append<T>(const QkvNormArgs&, int, cudaStream_t);                                                 \
     template void launch_out_norm<T>(float*, T*, const T*, const MoeMix&, float, const bf16*, int, int, int, float, cudaStream_t);  \
     template void launch_norm_rows<T>(const float*, const int32_t*, const bf16*, T*, int, int, int, float, cudaStream_t);           \

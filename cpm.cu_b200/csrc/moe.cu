@@ -400,6 +400,7 @@ struct GemmArgs {
     int ldy;
     const int4* entries;
     const int32_t* n_entries;
+    int uniform;           // > 0: the groups are not the router's, every one of this many matrices has all rows
     int* error;
 };
 // The row groups come from the router.  gate/up launches its successor only after its own wait, i.e. when the router has
@@ -485,6 +486,14 @@ moe_gemm_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_cons
         ptx::tmem_relinquish();
     }
     auto read_groups = [&]() -> int {
+        if (a.uniform > 0) {
+            const int per = (a.rows + a.tile - 1) / a.tile, n = a.uniform * per;
+            for (int i = threadIdx.x; i < n; i += NUM_THREADS) {
+                const int m = i / per, r = (i - m * per) * a.tile;
+                entries[i] = make_int4(m, m * a.rows + r, m * a.rows + r, min(a.tile, a.rows - r));
+            }
+            return n;
+        }
         const int n = min(__ldcg(a.n_entries), kMoeMaxEntries);
         for (int i = threadIdx.x; i < n; i += NUM_THREADS) entries[i] = __ldcg(a.entries + i);
         return n;
@@ -723,6 +732,27 @@ size_t moe_gate_up_elems(const LayerSpec& sp, int K) { return moe_gate_up_offset
 size_t moe_down_offset(const LayerSpec& sp, int width, int expert) { return static_cast<size_t>(expert) * linear_weight_elems(width, pad64(sp.expert_ff)); }
 size_t moe_down_elems(const LayerSpec& sp, int width) { return moe_down_offset(sp, width, sp.experts) + linear_weight_elems(width, pad64(sp.shared_ff)); }
 
+MoeGemmPlan make_grouped_plan(const bf16* w, int n, int N, int N_s, int K, const bf16* x, bf16* y, int ldy, int rows) {
+    CPM_REQUIRE(K % BLOCK_K == 0 && n >= 1 && N >= 1 && rows >= 1, "grouped product: bad sizes");
+    MoeGemmPlan p;
+    p.tile = 16;
+    while (p.tile < 256 && p.tile < rows) p.tile *= 2;
+    const size_t one = linear_weight_elems(N, K);
+    p.tm_w = weight_map(w, n * one + (N_s > 0 ? linear_weight_elems(N_s, K) : 0));
+    p.tm_x = make_tmap_2d(x, K, static_cast<uint64_t>(n + (N_s > 0 ? 1 : 0)) * rows, static_cast<uint64_t>(K) * 2, BLOCK_K, std::min(p.tile, 64));
+    p.tm_xs = p.tm_x;
+    p.rows = rows;
+    p.uniform = n;
+    p.max_entries = n * ceil_div(rows, p.tile);
+    CPM_REQUIRE(p.max_entries <= kMoeMaxEntries, "grouped product: too many row groups");
+    p.n_tiles = ceil_div(N, gemm::BLOCK_N); p.kblocks = K / BLOCK_K; p.N = N;
+    p.n_tiles_s = N_s > 0 ? ceil_div(N_s, gemm::BLOCK_N) : 0; p.kblocks_s = p.kblocks; p.N_s = N_s;
+    p.w_row_s = static_cast<long long>(n * one / BLOCK_K);
+    p.xs_row0 = p.ys_row0 = n * rows;
+    p.y = y; p.ldy = ldy;
+    return p;
+}
+
 MoeGemmPlan make_moe_gate_up_plan(const LayerSpec& sp, const bf16* w, const bf16* x, int x_rows, const bf16* xs, int K, bf16* act,
                                   int ld_act, int rows, int tile, const MoeBuffers& b) {
     CPM_REQUIRE(K % BLOCK_K == 0 && ld_act % BLOCK_K == 0, "mixture of experts: padded widths must be multiples of 64");
@@ -761,7 +791,7 @@ MoeGemmPlan make_moe_down_plan(const LayerSpec& sp, const bf16* w, const bf16* a
 }
 
 void launch_moe_gemm(const MoeGemmPlan& p, cudaStream_t s) {
-    ProfileScope prof(KC_MOE, s);
+    ProfileScope prof(p.uniform > 0 ? KC_LINEAR : KC_MOE, s);
     GemmArgs a;
     a.n_tiles = p.n_tiles; a.kblocks = p.kblocks; a.N = p.N;
     a.n_tiles_s = p.n_tiles_s; a.kblocks_s = p.kblocks_s; a.N_s = p.N_s;
@@ -771,6 +801,7 @@ void launch_moe_gemm(const MoeGemmPlan& p, cudaStream_t s) {
     a.w_row_s = p.w_row_s; a.xs_row0 = p.xs_row0; a.ys_row0 = p.ys_row0;
     a.y = p.y; a.ldy = p.ldy;
     a.entries = p.entries; a.n_entries = p.n_entries;
+    a.uniform = p.uniform;
     a.error = runtime().d_error;
     const long long most = static_cast<long long>(a.groups_s) * a.n_tiles_s + static_cast<long long>(p.max_entries) * p.n_tiles;
     const int grid = static_cast<int>(std::max<long long>(1, std::min<long long>(most, runtime().num_sms)));

@@ -1,0 +1,307 @@
+// Row-wise kernels of dynamic-tanh models: norms, token shift, residual sums, clamped gate, token side input, output norm
+// and gate of recurrences.  Everything is computed in fp32; T is the dtype of the activations.
+#include <algorithm>
+
+#include "row_ops.cuh"
+
+namespace {
+
+__device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) { return tanhf(alpha * x) * w + b; }
+
+__device__ __forceinline__ void tanh_norm8(const float* x, const DynTanh& n, int c, float* h) {
+    float w[8], b[8];
+    load_vec<8>(n.w + c, w);
+    load_vec<8>(n.b + c, b);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) h[e] = tanh_norm(x[e], n.alpha, w[e], b[e]);
+}
+
+// the mixes of row r, columns c .. c + 7, from its h and the h before it
+template <typename T>
+__device__ __forceinline__ void store_mixes(const TokenShift& t, int r, int ld, int c, const float* h, const float* before) {
+#pragma unroll
+    for (int m = 0; m < kMixes; ++m) {
+        float mu[8], f[8];
+        load_vec<8>(t.mu + static_cast<size_t>(m) * ld + c, mu);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = h[e] + (before[e] - h[e]) * mu[e];
+        store_vec<8>(static_cast<T*>(t.out) + m * t.stride + static_cast<size_t>(r) * ld + c, f);
+    }
+}
+
+// columns c .. c + 7 of the h before the first row
+__device__ __forceinline__ void load_before(const TokenShift& t, int c, float* before) {
+    if (*t.kv_len + t.kv_off == 0) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) before[e] = 0.f;
+    } else {
+        load_vec<8>(t.prev + c, before);
+    }
+}
+
+// CTA b takes row b; with mixes the last row belongs to CTA 0 as well, which has then read `prev` before it is written.
+template <typename T>
+__global__ void tanh_norm_kernel(const float* __restrict__ x32, const int32_t* __restrict__ rows_idx, const DynTanh n, T* __restrict__ hout,
+                                 const TokenShift t, int rows, int ld) {
+    grid_dependency_sync();
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < ld; c += gridDim.y * blockDim.x * 8) {
+        for (int r = blockIdx.x; r < rows; r += rows - 1 > 0 && blockIdx.x == 0 && t.mu != nullptr ? rows - 1 : rows) {
+            const size_t at = static_cast<size_t>(rows_idx ? rows_idx[r] : r) * ld + c;
+            float x[8], h[8];
+            load_vec<8>(x32 + at, x);
+            tanh_norm8(x, n, c, h);
+            store_vec<8>(hout + static_cast<size_t>(r) * ld + c, h);
+            if (t.mu == nullptr) continue;
+            float before[8];
+            if (r == 0) {
+                load_before(t, c, before);
+            } else {
+                load_vec<8>(x32 + at - ld, x);
+                tanh_norm8(x, n, c, before);
+            }
+            store_mixes<T>(t, r, ld, c, h, before);
+            if (r == rows - 1) store_vec<8>(t.prev + c, h);
+        }
+    }
+}
+
+template <typename T>
+__global__ void tanh_residual_kernel(float* __restrict__ x32, const T* __restrict__ delta, const DynTanh post, const DynTanh next,
+                                     T* __restrict__ out, int rows, int ld) {
+    grid_dependency_sync();
+    const size_t base = static_cast<size_t>(blockIdx.x) * ld;
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < ld; c += gridDim.y * blockDim.x * 8) {
+        float x[8], d[8], y[8];
+        load_vec<8>(x32 + base + c, x);
+        load_vec<8>(delta + base + c, d);
+        tanh_norm8(d, post, c, y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += y[e];
+        store_vec<8>(x32 + base + c, x);
+        if (next.w != nullptr) tanh_norm8(x, next, c, x);
+        store_vec<8>(out + base + c, x);
+    }
+}
+
+template <typename T>
+__global__ void clamped_gate_kernel(const T* __restrict__ gu, int ld_gu, T* __restrict__ act, int ld_act, int ff, float limit, float alpha,
+                                    int interleaved) {
+    grid_dependency_sync();
+    const T* g = gu + static_cast<size_t>(blockIdx.x) * ld_gu;
+    for (int c = threadIdx.x * 8; c < ff; c += blockDim.x * 8) {   // ff is a multiple of 64
+        const int at = interleaved ? (c >> 6) * 128 + (c & 63) : c;
+        float gv[8], uv[8];
+        load_vec<8>(g + at, gv);
+        load_vec<8>(g + at + (interleaved ? 64 : ff), uv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) gv[e] = clamped_gate(gv[e], uv[e], limit, alpha);
+        store_vec<8>(act + static_cast<size_t>(blockIdx.x) * ld_act + c, gv);
+    }
+}
+
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+template <typename T>
+__global__ void side_gate_kernel(const T* __restrict__ z, int ld, const int32_t* __restrict__ ids, const bf16* __restrict__ table, int table_ld,
+                                 int col0, int dim, int vocab, T* __restrict__ g) {
+    grid_dependency_sync();
+    int id = ids[blockIdx.x];
+    if (id < 0 || id >= vocab) id = 0;   // reported by the embedding
+    const bf16* e = table + static_cast<size_t>(id) * table_ld + col0;
+    const size_t base = static_cast<size_t>(blockIdx.x) * ld;
+    for (int c = threadIdx.x; c < ld; c += blockDim.x) {
+        g[base + c] = from_float<T>(c < dim ? gelu_tanh(to_float<T>(z[base + c])) * __bfloat162float(e[c]) : 0.f);
+    }
+}
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(512)
+side_add_kernel(float* __restrict__ x32, const T* __restrict__ y, const bf16* __restrict__ w, const DynTanh next, T* __restrict__ hout,
+                const TokenShift t, int width, int ld, float eps) {
+    grid_dependency_sync();
+    __shared__ float sh[64];
+    const size_t base = static_cast<size_t>(blockIdx.x) * ld;
+    float yv[VPT][8], ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int c = (threadIdx.x + j * blockDim.x) * 8;
+        if (c >= ld) continue;
+        load_vec<8>(y + base + c, yv[j]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += yv[j][e] * yv[j][e];   // padding columns are zero
+    }
+    const float rs = rsqrtf(block_sum2(ss, 0.f, sh).x / width + eps);
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int c = (threadIdx.x + j * blockDim.x) * 8;
+        if (c >= ld) continue;
+        float x[8], wv[8];
+        load_vec<8>(x32 + base + c, x);
+        load_vec<8>(w + c, wv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += yv[j][e] * rs * wv[e];
+        store_vec<8>(x32 + base + c, x);
+        if (next.w == nullptr) continue;
+        float h[8];
+        tanh_norm8(x, next, c, h);
+        store_vec<8>(hout + base + c, h);
+        if (t.mu != nullptr) {   // a single row
+            float before[8];
+            load_before(t, c, before);
+            store_mixes<T>(t, 0, ld, c, h, before);
+            store_vec<8>(t.prev + c, h);
+        }
+    }
+}
+
+// kDecayRows tokens x 256 channels per CTA, one channel per thread.
+constexpr int kDecayRows = 8;
+
+template <typename T>
+__global__ void decay_kernel(const T* __restrict__ x, int ld_x, const bf16* __restrict__ w2, const bf16* __restrict__ w0, int rank, int channels,
+                             float* __restrict__ out, int ld_out, int rows) {
+    extern __shared__ float inner[];   // [rank][kDecayRows]
+    const int row0 = blockIdx.y * kDecayRows, n = min(kDecayRows, rows - row0);
+    grid_dependency_sync();
+    for (int i = threadIdx.x; i < kDecayRows * rank; i += blockDim.x) {
+        const int t = i / rank, k = i - t * rank;
+        inner[k * kDecayRows + t] = t < n ? tanhf(to_float<T>(x[static_cast<size_t>(row0 + t) * ld_x + k])) : 0.f;
+    }
+    __syncthreads();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= channels) return;
+    const float b = __bfloat162float(w0[c]);
+    float z[kDecayRows];
+#pragma unroll
+    for (int t = 0; t < kDecayRows; ++t) z[t] = b;
+    const bf16* w = w2 + static_cast<size_t>(c) * rank;
+    auto add = [&](float wk, int k) {
+        const float4 p = *reinterpret_cast<const float4*>(inner + k * kDecayRows), q = *reinterpret_cast<const float4*>(inner + k * kDecayRows + 4);
+        z[0] = fmaf(wk, p.x, z[0]); z[1] = fmaf(wk, p.y, z[1]); z[2] = fmaf(wk, p.z, z[2]); z[3] = fmaf(wk, p.w, z[3]);
+        z[4] = fmaf(wk, q.x, z[4]); z[5] = fmaf(wk, q.y, z[5]); z[6] = fmaf(wk, q.z, z[6]); z[7] = fmaf(wk, q.w, z[7]);
+    };
+    if (rank % 8 == 0) {
+        for (int k = 0; k < rank; k += 8) {
+            float f[8];
+            load_vec<8>(w + k, f);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) add(f[e], k + e);
+        }
+    } else {
+        for (int k = 0; k < rank; ++k) add(__bfloat162float(w[k]), k);
+    }
+    for (int t = 0; t < n; ++t) out[static_cast<size_t>(row0 + t) * ld_out + c] = expf(-expf(z[t]));
+}
+
+// One CTA per row; one warp per group, or the whole CTA for a single group.
+template <typename T>
+__global__ void norm_gate_kernel(const float* __restrict__ o, int ld_o, int groups, int group, const bf16* __restrict__ w,
+                                 const T* __restrict__ gate, int ld_gate, int silu, float eps, float scale, T* __restrict__ out, int ld_out) {
+    grid_dependency_sync();
+    __shared__ float sh[64];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    o += static_cast<size_t>(blockIdx.x) * ld_o;
+    gate += static_cast<size_t>(blockIdx.x) * ld_gate;
+    out += static_cast<size_t>(blockIdx.x) * ld_out;
+    auto finish = [&](int c, float rs) {
+        const float g = to_float<T>(gate[c]), s = 1.f / (1.f + expf(-g));
+        out[c] = from_float<T>(o[c] * rs * __bfloat162float(w[c]) * (silu ? g * s : s) * scale);
+    };
+    if (groups == 1) {
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < group; c += blockDim.x) ss += o[c] * o[c];
+        const float rs = rsqrtf(block_sum2(ss, 0.f, sh).x / group + eps);
+        for (int c = threadIdx.x; c < group; c += blockDim.x) finish(c, rs);
+    } else {
+        for (int g = warp; g < groups; g += blockDim.x >> 5) {
+            float ss = 0.f;
+            for (int c = g * group + lane; c < (g + 1) * group; c += 32) ss += o[c] * o[c];
+            const float rs = rsqrtf(warp_sum(ss) / group + eps);
+            for (int c = g * group + lane; c < (g + 1) * group; c += 32) finish(c, rs);
+        }
+    }
+}
+
+// Grid and block of an element-wise kernel over rows of ld / 8 vectors: few rows spread over column blocks.
+inline void row_grid(int rows, int ld, dim3& grid, dim3& block) {
+    const int vecs = ld / 8;
+    const int threads = std::min(rows < 64 ? 64 : 256, (vecs + 31) / 32 * 32);
+    grid = dim3(rows, rows < 64 ? ceil_div(vecs, threads) : 1);
+    block = dim3(threads);
+}
+
+}  // namespace
+
+template <typename T>
+void launch_tanh_norm(const float* x32, const int32_t* rows_idx, const DynTanh& n, T* h, const TokenShift& shift, int rows, int ld,
+                      cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    CPM_REQUIRE(ld % 64 == 0 && (shift.mu == nullptr || rows_idx == nullptr), "tanh_norm: bad arguments");
+    dim3 grid, block;
+    row_grid(rows, ld, grid, block);
+    if (shift.mu != nullptr && rows > 1) grid.x = rows - 1;
+    launch_kernel(tanh_norm_kernel<T>, grid, block, 0, s, x32, rows_idx, n, h, shift, rows, ld);
+}
+
+template <typename T>
+void launch_tanh_residual(float* x32, const T* delta, const DynTanh& post, const DynTanh& next, T* out, int rows, int ld, cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    dim3 grid, block;
+    row_grid(rows, ld, grid, block);
+    launch_kernel(tanh_residual_kernel<T>, grid, block, 0, s, x32, delta, post, next, out, rows, ld);
+}
+
+template <typename T>
+void launch_clamped_gate(const T* gu, int ld_gu, T* act, int ld_act, int rows, int ff, float limit, float alpha, bool interleaved, cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    CPM_REQUIRE(ff % 64 == 0 && ld_act % 8 == 0 && ld_gu % 8 == 0, "clamped gate: widths must be multiples of 64");
+    launch_kernel(clamped_gate_kernel<T>, dim3(rows), dim3(256), 0, s, gu, ld_gu, act, ld_act, ff, limit, alpha, interleaved ? 1 : 0);
+}
+
+template <typename T>
+void launch_side_gate(const T* z, int ld, const int32_t* ids, const bf16* table, int table_ld, int col0, int dim, int vocab, T* g, int rows,
+                      cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    launch_kernel(side_gate_kernel<T>, dim3(rows), dim3(64), 0, s, z, ld, ids, table, table_ld, col0, dim, vocab, g);
+}
+
+template <typename T>
+void launch_side_add(float* x32, const T* y, const bf16* w, const DynTanh& next, T* h, const TokenShift& shift, int rows, int width, int ld,
+                     float eps, cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    CPM_REQUIRE(ld % 64 == 0 && ld <= 512 * 8 * 4 && (shift.mu == nullptr || rows == 1), "side_add: bad arguments");
+    const int vecs = ld / 8;
+    const int threads = vecs >= 512 ? 512 : (vecs + 31) / 32 * 32;
+    if (vecs <= 512) launch_kernel(side_add_kernel<T, 1>, dim3(rows), dim3(threads), 0, s, x32, y, w, next, h, shift, width, ld, eps);
+    else launch_kernel(side_add_kernel<T, 4>, dim3(rows), dim3(threads), 0, s, x32, y, w, next, h, shift, width, ld, eps);
+}
+
+template <typename T>
+void launch_decay(const T* x, int ld_x, const bf16* w2, const bf16* w0, int rank, int channels, float* out, int ld_out, int rows, cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    CPM_REQUIRE(rank >= 1 && rank <= 1024, "time mix: inner width of the decay must be in [1, 1024]");
+    launch_kernel(decay_kernel<T>, dim3(ceil_div(channels, 256), ceil_div(rows, kDecayRows)), dim3(256), rank * kDecayRows * sizeof(float), s, x, ld_x,
+                  w2, w0, rank, channels, out, ld_out, rows);
+}
+
+template <typename T>
+void launch_norm_gate(const float* o, int ld_o, int groups, int group, const bf16* w, const T* gate, int ld_gate, bool silu, float eps,
+                      float scale, T* out, int ld_out, int rows, cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    launch_kernel(norm_gate_kernel<T>, dim3(rows), dim3(256), 0, s, o, ld_o, groups, group, w, gate, ld_gate, silu ? 1 : 0, eps, scale, out,
+                  ld_out);
+}
+
+#define CPM_INSTANTIATE(T)                                                                                                                  \
+    template void launch_tanh_norm<T>(const float*, const int32_t*, const DynTanh&, T*, const TokenShift&, int, int, cudaStream_t);         \
+    template void launch_tanh_residual<T>(float*, const T*, const DynTanh&, const DynTanh&, T*, int, int, cudaStream_t);                    \
+    template void launch_clamped_gate<T>(const T*, int, T*, int, int, int, float, float, bool, cudaStream_t);                               \
+    template void launch_side_gate<T>(const T*, int, const int32_t*, const bf16*, int, int, int, int, T*, int, cudaStream_t);               \
+    template void launch_side_add<T>(float*, const T*, const bf16*, const DynTanh&, T*, const TokenShift&, int, int, int, float,            \
+                                     cudaStream_t);                                                                                         \
+    template void launch_decay<T>(const T*, int, const bf16*, const bf16*, int, int, float*, int, int, cudaStream_t);                       \
+    template void launch_norm_gate<T>(const float*, int, int, int, const bf16*, const T*, int, bool, float, float, T*, int, int, cudaStream_t);
+CPM_INSTANTIATE(bf16)
+CPM_INSTANTIATE(float)

@@ -73,6 +73,8 @@ struct AttnArgs {
     int window;
     int exact_window;    // > 0: per-token sliding window (tokens); BIASED instantiations only
     float bias_exp;      // > 0: distance bias with slopes 2^(-bias_exp * (h + 1) / hq); BIASED instantiations only
+    int sink;            // 1: exp(0) is added to every row's sum
+    float out_scale;     // factor of the output
     int out_cols;        // value columns that are stored per head (the rest of DV is padding)
     const uint64_t* blockmask;  // [hkv][tq][bm_words] bits over 64-key blocks, or null
     int bm_words, block_window;
@@ -195,7 +197,8 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
     }
     const float slope2 =   // log2(e) * slope of this row's head
         (BIASED && a.bias_exp > 0.f) ? 1.4426950408889634f * exp2f(-a.bias_exp * static_cast<float>(qh + 1) / static_cast<float>(a.hq)) : 0.f;
-    const float sl2 = BIASED ? 1.f : a.scale_log2;   // biased scores are brought to log2 units as they are read
+    const bool biased = BIASED && a.bias_exp > 0.f;
+    const float sl2 = biased ? 1.f : a.scale_log2;   // biased scores are brought to log2 units as they are read
     const int kt_lo = key_lo / KEYS;
     const int kt_hi = (key_hi + KEYS - 1) / KEYS;
     const int n_kt = max(kt_hi - kt_lo, 0);
@@ -380,7 +383,7 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
             ptx::tmem_ld32(tmem_s, sc);
             ptx::tmem_ld32(tmem_s + 32, sc + 32);
             ptx::tmem_wait_ld();
-            if (BIASED) {
+            if (biased) {
                 const float b0 = slope2 * static_cast<float>(key0 - (causal_base + t));   // <= 0 where the key is visible
 #pragma unroll
                 for (int c = 0; c < 64; ++c) {
@@ -498,11 +501,13 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
         // and only the global stores depend on whether the row exists.
         xch[ch * ROWS + row] = l_run;
         ptx::named_bar_sync(1, SOFTMAX_THREADS);
-        const float l_row = l_run + xch[(ch ^ 1) * ROWS + row];
+        float l_row = l_run + xch[(ch ^ 1) * ROWS + row];
+        // the sink joins the sum once: here, or when the splits' sums are merged
+        if (BIASED && a.sink != 0 && nsplit == 1 && m_run != -INFINITY) l_row += exp2f(-m_run * sl2);
         if (ok) {
             const bool store = row_in && (t < a.tq);
             const size_t grow = static_cast<size_t>(store ? t : 0) * a.hq + qh;
-            const float inv = (nsplit == 1) ? ((l_row > 0.f) ? 1.f / l_row : 0.f) : 1.f;
+            const float inv = (nsplit == 1) ? ((l_row > 0.f) ? (BIASED ? a.out_scale : 1.f) / l_row : 0.f) : 1.f;
             bf16* dst_b = a.out + static_cast<size_t>(store ? t : 0) * a.out_ld + qh * (BIASED ? a.out_cols : DV) + ch * (DV / 2);
             const int cols = BIASED ? a.out_cols - ch * (DV / 2) : DV / 2;   // real columns of this thread's half
             const bool whole = !BIASED || (a.out_cols % 8 == 0 && a.out_ld % 8 == 0);
@@ -574,7 +579,8 @@ tree_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
 // every lane accumulates four output columns with independent loads in flight.
 template <int DV>
 __global__ void attn_combine_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_ml, int nsplit,
-                                    int rows, int hq, float scale_log2, bf16* __restrict__ out, int out_ld, int out_cols) {
+                                    int rows, int hq, float scale_log2, bf16* __restrict__ out, int out_ld, int out_cols,
+                                    int sink, float out_scale) {
     grid_dependency_sync();
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
@@ -624,7 +630,8 @@ __global__ void attn_combine_kernel(const float* __restrict__ ws_o, const float*
             for (int c = 0; c < CPL; ++c) acc[c] += w * reinterpret_cast<const float*>(&o[j])[c];
         }
     }
-    const float inv = (l > 0.f) ? 1.f / l : 0.f;
+    if (sink != 0 && M != -INFINITY) l += exp2f(-M * scale_log2);
+    const float inv = (l > 0.f) ? out_scale / l : 0.f;
     const int t = row / hq, qh = row - t * hq;
     bf16* dst = out + static_cast<size_t>(t) * out_ld + qh * out_cols + lane * CPL;
     uint32_t pk[CPL / 2];
@@ -700,7 +707,7 @@ void launch_attn(const AttnPlan& p, const AttnArgs& a, cudaStream_t s) {
     if (p.splits > 1) {
         const int rows = p.tq * p.hq;
         launch_kernel(attn_combine_kernel<DV>, dim3(ceil_div(rows, 4)), dim3(128), 0, s, p.ws_o, p.ws_ml, p.splits, rows, p.hq,
-                      BIASED ? 1.f : a.scale_log2, p.out, p.out_ld, p.out_cols);
+                      BIASED && p.bias_exp > 0.f ? 1.f : a.scale_log2, p.out, p.out_ld, p.out_cols, p.sink, p.out_scale);
     }
 }
 }  // namespace
@@ -720,6 +727,7 @@ void launch_tree_attention(const AttnPlan& p, cudaStream_t s) {
     a.mask = p.mask; a.mask_k = p.mask_k;
     a.window = p.window;
     a.exact_window = p.exact_window; a.bias_exp = p.bias_exp; a.out_cols = p.out_cols;
+    a.sink = p.sink; a.out_scale = p.out_scale;
     a.blockmask = p.blockmask; a.bm_words = p.bm_words; a.block_window = p.block_window;
     CPM_REQUIRE(p.blockmask == nullptr || (p.bm_words >= 1 && p.bm_words <= 64 && p.block_window >= 1),
                 "attention: block mask needs 1..64 words per row and a local window of at least one block");

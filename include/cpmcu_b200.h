@@ -84,7 +84,7 @@ int cpmcu_init_minicpm4_eagle_model(int num_layers, int num_iter, int topk_per_i
 
 /* One layer of a layered model (no reference counterpart). */
 typedef struct {
-    /* mixer: softmax attention; query head h uses key/value head h / (heads / kv_heads) */
+    /* mixer: softmax attention (heads == 0: none); query head h uses key/value head h / (heads / kv_heads) */
     int heads, kv_heads, dim, vdim;
     float scale;          /* score = scale * (q . k) - slope_h * (i - j) */
     int window;           /* > 0: token i sees j with 0 <= i - j < window; 0: all j <= i */
@@ -99,16 +99,35 @@ typedef struct {
     float router_scale;
     int expert_ff;
     int shared_ff;        /* > 0: an expert of this width that every token uses; 0: none */
+    /* more of the attention */
+    int sink;             /* 1: every softmax has one more score of 0, without a value */
+    int rot_dims;         /* > 0: rotary positions on the first rot_dims of each head, i paired with i + rot_dims / 2 */
+    float attn_scale;     /* factor of its output */
+    /* mixer: a recurrence, alone or beside the attention (their outputs are added).  0: none; 1: time mix, decays per token
+     * and channel; 2: lightning, one constant decay per head */
+    int recurrence, rec_heads, rec_dim, rec_vdim;
+    int rec_rank;         /* time mix: rows of w1 */
+    float rec_scale;      /* factor of its output */
+    /* feed-forward: a dense one of this width (0: none), g sigmoid(ff_alpha g) (u + 1), g <= ff_limit, |u| <= ff_limit */
+    int ff;
+    float ff_limit, ff_alpha;
 } cpmcu_layer_spec;
 
-/* A decoder described layer by layer, with RMS norms (weights stored as their distance from one) on the sublayers'
- * outputs and a 32-bit residual stream: x += residual_mult * norm(sublayer(x)).  torch_dtype: 1 = bf16, 2 = fp32 (all
- * arithmetic in true 32-bit; weights are given as bf16 either way, logits come back in that dtype).
- * Tensors for cpmcu_load_model: embed [vocab, width], head, final.norm, and for layer i (prefix "l<i>."): norm1, mix.q,
- * mix.k, mix.v, mix.o, mix.q.norm, mix.k.norm, norm2, mlp.router, mlp.correction, mlp.e<j>.{gate,up,down},
- * mlp.shared.{gate,up,down}; matrices [out, in] bf16. */
-int cpmcu_init_layered_model(float memory_limit, int vocab_size, int width, float norm_eps, float residual_mult,
-                             int torch_dtype, int chunk_length, int num_layers, const cpmcu_layer_spec* layers);
+/* A decoder described layer by layer on a 32-bit residual stream that starts as embed_scale * embed[token].  torch_dtype:
+ * 1 = bf16, 2 = fp32 (all arithmetic in true 32-bit; weights are given as bf16 either way, logits come back in that dtype).
+ * norm 0: RMS norms (weights stored as their distance from one) on the sublayers' outputs, x += residual_mult * norm(sublayer(x)).
+ * norm 1: N(x) = tanh(alpha x) * w + b before and after, x += Nb(sublayer(N(x))).
+ * tied_head: the head is the embedding table.  side_dim > 0 (norm 1): after every layer i
+ * x += rms(P (gelu_tanh(G x) * side.embed[token][i * side_dim ..])) * w.
+ * Tensors for cpmcu_load_model: embed [vocab, width], head (unless tied), final.norm, and for layer i (prefix "l<i>."):
+ * norm1, norm2 and with norm 1 norm1b, norm2b, each norm with .b and .alpha; attention mix.{q,k,v,o}, mix.q.norm, mix.k.norm,
+ * mix.inv_freq (fp32, base^(-2 i / rot_dims)); time mix mix.{r,k,v,g,o,norm,u,w0,w1,w2}, mix.mu.{r,k,v,g,w}; lightning
+ * mix.{q,k,v,g,o,norm}, mix.decay (fp32); attention beside a recurrence is mix.left, the recurrence mix.right; mlp.{gate,up,down},
+ * or mlp.router, mlp.correction, mlp.e<j>.{gate,up,down}, mlp.shared.{gate,up,down}; side.embed [vocab, layers * side_dim],
+ * l<i>.side.{gate,proj,norm}.  Matrices are [out, in] bf16. */
+int cpmcu_init_layered_model(float memory_limit, int vocab_size, int width, int norm, float norm_eps, float residual_mult,
+                             float embed_scale, int tied_head, int side_dim, int torch_dtype, int chunk_length, int num_layers,
+                             const cpmcu_layer_spec* layers);
 
 /* reference: the three spec / hierarchical initialisers, src/entry.cu:344-459.
  * Out of scope for this library: always fail. */
@@ -201,8 +220,8 @@ int cpmcu_capture_blockmasks(uint64_t* device_buf);
  * [layers][rows][width] fp32, to device_buf (caller-owned device memory; NULL stops it). */
 int cpmcu_capture_layers(float* device_buf);
 /* Per-launch timing of the forward passes made while it is on: cpmcu_profile(1) starts (decode then runs uncaptured),
- * cpmcu_profile(0) stops and writes 6 entries each to ms / launches (HOST): linear layers, attention, block selection,
- * expert products, routing, row-wise kernels. */
+ * cpmcu_profile(0) stops and writes 7 entries each to ms / launches (HOST): linear layers, attention, block selection,
+ * expert products, routing, row-wise kernels, recurrences. */
 int cpmcu_profile(int on, float* ms, int* launches);
 
 /* Copies the engine-owned tree of the last step to HOST arrays of 64 entries
@@ -303,9 +322,17 @@ int cpmcu_linear_swiglu_bf16(const void* x, const void* w, void* out, int rows, 
  * splits: key splits of the tensor-core kernel; 0 = the plain kernel. */
 int cpmcu_layer_attention(const cpmcu_layer_spec* spec, const void* q, const void* k_cache, const void* v_cache, int budget,
                           int tq, int kv_total, int splits, int fp32, void* out);
-/* qkv [rows, heads*dim + kv_heads*(dim + vdim)] -> q_out [rows, heads, dk] and cache rows kv_row ..; norms as in the spec. */
+/* qkv [rows, heads*dim + kv_heads*(dim + vdim)] -> q_out [rows, heads, dk] and cache rows kv_row ..; norms as in the spec
+ * (wq null: none), rotation with inv_freq [rot_dims / 2] (null: none). */
 int cpmcu_layer_qkv_norm_append(const cpmcu_layer_spec* spec, const void* qkv, const void* wq, const void* wk, float eps,
-                                int rows, int kv_row, int cache_rows, int fp32, void* q_out, void* k_cache, void* v_cache);
+                                const float* inv_freq, int rows, int kv_row, int cache_rows, int fp32, void* q_out, void* k_cache, void* v_cache);
+/* The recurrence of a layer over `rows` tokens from `position` on (0: from a zero state): r (or q), k [rows, heads * dim], v
+ * [rows, heads * vdim] in the activation dtype (lightning: before their silu), time mix: decays w [rows, heads * dim] and bonus
+ * [heads * dim] (bf16), lightning: decay [heads].  state: cpmcu_layer_scan_state_floats() floats, read and replaced.
+ * out [rows, heads * vdim] fp32. */
+int cpmcu_layer_scan(const cpmcu_layer_spec* spec, const void* r, const void* k, const void* v, const float* w, const float* decay,
+                     const void* bonus, float* state, int rows, int position, int fp32, float* out);
+long cpmcu_layer_scan_state_floats(const cpmcu_layer_spec* spec);
 /* x32 += mult * rms(delta) * (1 + w); xh = x32 in the activation dtype. */
 int cpmcu_layer_out_norm(float* x32, void* xh, const void* delta, float mult, const void* w, int rows, int width, int ld,
                          float eps, int fp32);

@@ -141,7 +141,7 @@ def test_qkv_norm_over_the_whole_projection(mix, fp32):
     q = torch.full((rows, H, pad64(d)), 5.0, dtype=dt, device="cuda")
     kc, vc = (torch.zeros(budget, G, pad64(n), dtype=dt, device="cuda") for n in (d, dv))
     xc, wqc, wkc = x.cuda(), wq.cuda(), wk.cuda()
-    C.call("cpmcu_layer_qkv_norm_append", ctypes.byref(spec_of(mix)), xc.data_ptr(), wqc.data_ptr(), wkc.data_ptr(), eps, rows, at,
+    C.call("cpmcu_layer_qkv_norm_append", ctypes.byref(spec_of(mix)), xc.data_ptr(), wqc.data_ptr(), wkc.data_ptr(), eps, None, rows, at,
            budget, int(fp32), q.data_ptr(), kc.data_ptr(), vc.data_ptr())
     f = x.double()
     rq = T.norm_plain(f[:, :H * d], wq.double(), eps).view(rows, H, d)
@@ -152,7 +152,7 @@ def test_qkv_norm_over_the_whole_projection(mix, fp32):
     assert torch.equal(vc[at:at + rows, :, :dv].cpu(), x[:, (H + G) * d:].view(rows, G, dv))
     assert (q[..., d:] == 0).all() and (kc[..., d:] == 0).all() and (kc[:at] == 0).all() and (kc[at + rows:] == 0).all()
     with pytest.raises(RuntimeError):        # the last row would fall behind the cache: refused, nothing written there
-        C.call("cpmcu_layer_qkv_norm_append", ctypes.byref(spec_of(mix)), xc.data_ptr(), wqc.data_ptr(), wkc.data_ptr(), eps, rows,
+        C.call("cpmcu_layer_qkv_norm_append", ctypes.byref(spec_of(mix)), xc.data_ptr(), wqc.data_ptr(), wkc.data_ptr(), eps, None, rows,
                budget - rows + 1, budget, int(fp32), q.data_ptr(), kc.data_ptr(), vc.data_ptr())
 
 
