@@ -683,7 +683,7 @@ def main():
                     help="config2 = the headline bf16 workload; config3 = the same with an FR-Spec draft vocabulary of 32768; "
                          "config4 = the same with a W4A16 GPTQ-Marlin target; config5 = 32768-token prompt, InfLLM-v2 "
                          "sparse target, draft window 1024")
-    ap.add_argument("--model", default=None, choices=["tipetar"],
+    ap.add_argument("--model", default=None, choices=["tipetar", "fabulix"],
                     help="instead of the speculative-decoding workload: prefill and decode throughput of this model design "
                          "beside the Llama-format model of equal size (bench_layered.py)")
     ap.add_argument("--sizes", default="", help="with --model: the sizes to run, with commas between them")

@@ -199,7 +199,7 @@ void Engine::lay_out_layered(Pool& p) {
     lact_ = p.take(R * ff * es);
     lside_ = p.take(R * side_ld * es);
     lsg_ = p.take(R * side_ld * es);
-    state_len_ = take<int32_t>(p, 1);
+    state_len_ = take<int32_t>(p, 2);   // and the counter of a one-token recurrence
     moe_rows_ = slots;
     moe_x_ = p.take(x_slots * L * es);
     moe_act_ = p.take(slots * act_ld * es);
@@ -607,9 +607,12 @@ void Engine::layered_recurrence(int i, LayeredPlans& lp, const int32_t* kv_len, 
     a.kv_len = kv_len; a.kv_off = kv_off;
     a.out = lo_; a.ld_out = nv;
     const T* gate;
-    if (sp.rec == REC_TIME_MIX) {
+    const bool per_head = sp.rec == REC_TIME_MIX;
+    T* out = static_cast<T*>(lattn_) + o_left(sp);
+    const bool step = rows == 1 && scan_step_fits(sp.rec_dim, sp.rec_vdim, per_head);
+    if (per_head) {
         const size_t part = static_cast<size_t>(rows) * ldr;
-        launch_decay<T>(proj + 4 * part, ldr, w.w2, w.w0, sp.rec_rank, nk, ldecay_, nk, rows, s);
+        if (!step) launch_decay<T>(proj + 4 * part, ldr, w.w2, w.w0, sp.rec_rank, nk, ldecay_, nk, rows, s);
         a.r = proj; a.k = proj + part; a.v = proj + 2 * part;
         gate = proj + 3 * part;
         a.w = ldecay_; a.ld_w = nk;
@@ -620,10 +623,21 @@ void Engine::layered_recurrence(int i, LayeredPlans& lp, const int32_t* kv_len, 
         a.silu = true;
         a.decay = w.decay;
     }
+    if (step) {
+        ScanStepArgs st;
+        st.scan = a;
+        st.inner = proj + 4 * static_cast<size_t>(ldr);
+        st.w2 = w.w2; st.w0 = w.w0; st.rank = sp.rec_rank;
+        st.norm = w.rec_norm; st.gate = gate;
+        st.eps = mc_.eps; st.scale = sp.rec_scale;
+        st.out = out;
+        st.ticket = state_len_ + 1;
+        launch_scan_step<T>(st, s);
+        return;
+    }
     launch_scan<T>(a, s);
-    const bool per_head = sp.rec == REC_TIME_MIX;
-    launch_norm_gate<T>(lo_, nv, per_head ? sp.rec_heads : 1, per_head ? sp.rec_vdim : nv, w.rec_norm, gate, ldr, per_head, mc_.eps, sp.rec_scale,
-                        static_cast<T*>(lattn_) + o_left(sp), o_cols(sp), rows, s);
+    launch_norm_gate<T>(lo_, nv, per_head ? sp.rec_heads : 1, per_head ? sp.rec_vdim : nv, w.rec_norm, gate, ldr, per_head, mc_.eps, sp.rec_scale, out,
+                        o_cols(sp), rows, s);
 }
 
 template <typename T>
@@ -661,20 +675,35 @@ bool Engine::layered_tanh_layer(int i, LayeredPlans& lp, const int32_t* ids, con
     if (sp.heads > 0) layered_attention<T>(i, lp, kv_len, kv_off, s);
     if (sp.rec != REC_NONE) layered_recurrence<T>(i, lp, kv_len, kv_off, s);
     run_product<T>(l.o, rows, s);
-    launch_tanh_residual<T>(x32_, delta, w.tanh1b, sp.ff > 0 ? w.tanh2 : DynTanh(), x, rows, L, s);
+    // a row's mixes need the row before it, which only a single row has at hand at a layer's end
+    const bool next = i + 1 < layers && mc_.side_dim > 0 && (rows == 1 || mc_.specs[i + 1].rec != REC_TIME_MIX);
+    const DynTanh next_norm = next ? lw_[i + 1].tanh1 : DynTanh();
+    const TokenShift next_shift = next ? token_shift(i + 1, rows, kv_len, kv_off) : TokenShift();
+    const bool side_step = rows == 1 && mc_.side_dim > 0 && mc_.side_dim <= 4096;
     if (sp.ff > 0) {
+        launch_tanh_residual<T>(x32_, delta, w.tanh1b, w.tanh2, x, rows, L, s);
         layered_dense<T>(i, lp, s);
-        launch_tanh_residual<T>(x32_, delta, w.tanh2b, DynTanh(), x, rows, L, s);
     }
+    const DynTanh& last = sp.ff > 0 ? w.tanh2b : w.tanh1b;
+    if (side_step) {
+        SideStepArgs a;
+        a.x32 = x32_; a.delta = ldelta_;
+        a.post = last;
+        a.gate = w.side_gate; a.proj = w.side_proj; a.norm = w.side_norm;
+        a.ids = ids; a.table = side_embed_; a.table_ld = layers * mc_.side_dim; a.col0 = i * mc_.side_dim;
+        a.dim = mc_.side_dim; a.vocab = mc_.vocab;
+        a.next = next_norm; a.h = lx_; a.shift = next_shift;
+        a.width = W; a.ld = L; a.eps = mc_.eps;
+        launch_side_step<T>(a, s);
+        return next;
+    }
+    launch_tanh_residual<T>(x32_, delta, last, DynTanh(), x, rows, L, s);
     if (mc_.side_dim == 0) return false;
     run_product<T>(l.side_gate, rows, s);
     launch_side_gate<T>(static_cast<const T*>(lside_), pad64(mc_.side_dim), ids, side_embed_, layers * mc_.side_dim, i * mc_.side_dim, mc_.side_dim,
                         mc_.vocab, static_cast<T*>(lsg_), rows, s);
     run_product<T>(l.side_proj, rows, s);
-    // a row's mixes need the row before it, which only a single row has at hand here
-    const bool next = i + 1 < layers && (rows == 1 || mc_.specs[i + 1].rec != REC_TIME_MIX);
-    launch_side_add<T>(x32_, delta, w.side_norm, next ? lw_[i + 1].tanh1 : DynTanh(), x, next ? token_shift(i + 1, rows, kv_len, kv_off) : TokenShift(), rows, W,
-                       L, mc_.eps, s);
+    launch_side_add<T>(x32_, delta, w.side_norm, next_norm, x, next_shift, rows, W, L, mc_.eps, s);
     return next;
 }
 

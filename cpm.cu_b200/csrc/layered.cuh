@@ -136,6 +136,24 @@ void launch_side_gate(const T* z, int ld, const int32_t* ids, const bf16* table,
 template <typename T>
 void launch_side_add(float* x32, const T* y, const bf16* w, const DynTanh& next, T* h, const TokenShift& shift, int rows, int width, int ld,
                      float eps, cudaStream_t s);
+// A single row from a sublayer's output to the next layer's input in one launch: x32 += post(delta), then the token side input
+// (gate product, launch_side_gate, projection, launch_side_add).  The two matrices are tile-major for bf16, row-major for fp32.
+struct SideStepArgs {
+    float* x32 = nullptr;
+    const void* delta = nullptr;
+    DynTanh post;
+    const bf16 *gate = nullptr, *proj = nullptr, *norm = nullptr;
+    const int32_t* ids = nullptr;
+    const bf16* table = nullptr;
+    int table_ld = 0, col0 = 0, dim = 0, vocab = 0;
+    DynTanh next;
+    void* h = nullptr;
+    TokenShift shift;
+    int width = 0, ld = 0;
+    float eps = 0.f;
+};
+template <typename T>
+void launch_side_step(const SideStepArgs& a, cudaStream_t s);
 // Decays of a time-mix layer: out[r][c] = exp(-exp(w2[c] . tanh(x[r]) + w0[c])), c < channels; x: `rank` columns of T, w2
 // [channels][rank]
 template <typename T>
@@ -171,6 +189,23 @@ size_t scan_state_floats(int heads, int dim, int vdim);
 size_t scan_workspace_floats(int heads, int dim, int vdim, int rows);
 template <typename T>
 void launch_scan(const ScanArgs& a, cudaStream_t s);
+
+// A single token's recurrence in one launch together with the decays before it (time mix: launch_decay of `inner`; a.w unused) and
+// the norm and gate behind it (launch_norm_gate per head for a time mix, over all heads otherwise).
+struct ScanStepArgs {
+    ScanArgs scan;
+    const void* inner = nullptr;   // T [rank]
+    const bf16 *w2 = nullptr, *w0 = nullptr;
+    int rank = 0;
+    const bf16* norm = nullptr;    // [heads * vdim]
+    const void* gate = nullptr;    // T [heads * vdim]
+    float eps = 0.f, scale = 1.f;
+    void* out = nullptr;           // T [heads * vdim]
+    int32_t* ticket = nullptr;     // zero between launches
+};
+bool scan_step_fits(int dim, int vdim, bool time_mix);
+template <typename T>
+void launch_scan_step(const ScanStepArgs& a, cudaStream_t s);
 
 // Attention of any head width up to 512, one warp per (token, head); q [tq][hq][dk], caches [.][hkv][dk | dv], out rows
 // of hq * out_cols.  The bias, window and kv_len arguments are those of make_biased_attn_plan.

@@ -1,26 +1,29 @@
 // Recurrences with an outer-product state (layered.cuh: ScanArgs) on the fp32 pipes.
 //
 // A warp holds 8 * KG rows (key channels) x 8 * (32 / KG) columns (value channels) of a head's state in registers, 8 x 8 per
-// lane, and walks over the tokens; r, k, w, v of a few tokens at a time lie in shared memory.  The output of a token is a sum
-// over the KG lanes of a column, folded so that every lane ends up with one column.
+// lane as pairs of rows for the packed fp32 instructions, and walks over the tokens; r, k, w, v of a few tokens at a time lie
+// in shared memory, the next ones on their way.  The output of a token is a sum over the KG lanes of a column, folded so that
+// every lane ends up with one column.
 //
-// Long portions are cut into chunks: scan_chunk_kernel adds up what every chunk alone would leave in the state (and its
-// decay), scan_link_kernel runs over the chunks and replaces that by the state each chunk begins with, and scan_kernel then
-// walks all chunks side by side.
+// Long portions are cut into chunks: a first walk over every chunk alone, from a zero state and without outputs, leaves what
+// the chunk adds to the state and its decay, scan_link_kernel runs over the chunks and replaces that by the state each chunk
+// begins with, and a second walk over all chunks side by side gives the outputs.
+//
+// A single token takes scan_step_kernel, which streams the state and does what surrounds the recurrence as well.
 #include <algorithm>
 
 #include "row_ops.cuh"
 
 namespace {
 
-constexpr int kChunk = 64;   // tokens per chunk
+constexpr int kMinChunk = 64;   // tokens per chunk: 64 or, when that gives enough warps, 128
+constexpr int TT = 8;           // tokens in shared memory
 
 template <int KG>
 struct Shape {
     static constexpr int KP = 8 * KG;           // key channels, padded
     static constexpr int VG = 32 / KG;
     static constexpr int CW = 8 * VG;           // value columns per warp
-    static constexpr int TT = KG >= 32 ? 8 : 16;  // tokens in shared memory
 };
 
 struct Geometry {
@@ -44,26 +47,75 @@ struct ScanParams {
     float* chunk_state;      // [chunks][heads][kp][vp]; null: the walk starts from and ends in a.state
     float* chunk_decay;      // [chunks][heads][kp]
     int chunks;
+    int vec_k, vec_v;        // rows of r, k, w / of v can be copied 16 bytes at a time
 };
 
-// tokens row0 .. row0 + n of one operand -> dst[t][width], zero where there is none
-template <typename T>
-__device__ __forceinline__ void stage(const void* src, int ld, int col0, int cols, int row0, int n, int width, bool silu, float* dst) {
-    for (int i = threadIdx.x; i < n * width; i += blockDim.x) {
-        const int t = i / width, c = i - t * width;
-        float v = 0.f;
-        if (c < cols) {
-            v = to_float<T>(static_cast<const T*>(src)[static_cast<size_t>(row0 + t) * ld + col0 + c]);
-            if (silu) v = silu_f32(v);
+// ---- pairs of fp32
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pair(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 unpair(f32x2 p) {
+    float2 f;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(p));
+    return f;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+// rows kg * 4 .. + 3 and kg * 4 + 4 KG .. + 3 as four pairs
+template <int KG>
+__device__ __forceinline__ void lds_pairs(const float* p, f32x2* f) {
+    const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(p), b = *reinterpret_cast<const ulonglong2*>(p + 4 * KG);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+
+__device__ __forceinline__ void copy16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src) : "memory");
+}
+
+// `n` rows of `cols` elements of a global matrix -> dst[t][width] in shared memory as they are
+template <typename E>
+__device__ __forceinline__ void copy_rows(E* dst, int width, const void* src, int ld, size_t row0, int col0, int cols, int n, int vec) {
+    constexpr int PER = 16 / sizeof(E);
+    const E* base = static_cast<const E*>(src) + row0 * ld + col0;
+    if (vec) {
+        const int per = cols / PER;
+        for (int i = threadIdx.x; i < n * per; i += blockDim.x) {
+            const int t = i / per, c = (i - t * per) * PER;
+            copy16(dst + t * width + c, base + static_cast<size_t>(t) * ld + c);
         }
-        dst[i] = v;
+    } else {
+        for (int i = threadIdx.x; i < n * cols; i += blockDim.x) {
+            const int t = i / cols, c = i - t * cols;
+            dst[t * width + c] = base[static_cast<size_t>(t) * ld + c];
+        }
     }
 }
 
-__device__ __forceinline__ void lds8(const float* p, int second, float* f) {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + second);
-    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+// raw rows -> fp32, zero from column `cols` on; width is a multiple of 8
+template <typename T>
+__device__ __forceinline__ void convert_rows(float* dst, const T* raw, int width, int cols, int n, bool silu) {
+    for (int i = threadIdx.x * 8; i < n * width; i += blockDim.x * 8) {
+        const int c = i % width;
+        float f[8];
+        load_vec<8>(raw + i, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            if (silu) f[e] = silu_f32(f[e]);
+            if (c + e >= cols) f[e] = 0.f;
+        }
+        store_vec<8>(dst + i, f);
+    }
 }
 
 // Sum over the KG lanes of a column group.  Afterwards the lane holds the sums of columns fold_column() (+ 1 for KG = 4).
@@ -84,169 +136,186 @@ __device__ __forceinline__ void fold(float* o, int lane) {
 }
 
 template <typename T, int KG, bool CONST_DECAY>
+struct ScanSmem {
+    static constexpr int KP = Shape<KG>::KP;
+    // floats: r, k, v of the tokens being walked over, decays of two batches; then the raw rows of two batches
+    static size_t bytes(int vb, bool out) {
+        const int keys = out ? 2 : 1;
+        return sizeof(float) * TT * (keys * KP + vb + (CONST_DECAY ? 0 : 2 * KP)) + sizeof(T) * 2 * TT * (keys * KP + vb);
+    }
+};
+
+// OUT: outputs from the state a chunk (or the sequence) begins with; otherwise what a chunk alone leaves behind.
+template <typename T, int KG, bool CONST_DECAY, bool OUT>
 __global__ void __launch_bounds__(128)
 scan_kernel(const ScanParams p) {
     using S_ = Shape<KG>;
-    constexpr int KP = S_::KP, TT = S_::TT;
+    constexpr int KP = S_::KP;
     const ScanArgs& a = p.a;
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     const int warps = blockDim.x >> 5, VB = warps * S_::CW;
     float* sr = sm;
-    float* sk = sr + TT * KP;
-    float* sw = sk + TT * KP;                          // no decays for CONST_DECAY
-    float* sv = sw + (CONST_DECAY ? 0 : TT * KP);
-    float* sb = sv + TT * VB;                          // bonus of a token: r . (u k)
+    float* sk = sr + (OUT ? TT * KP : 0);
+    float* sv = sk + TT * KP;
+    float* sw = sv + TT * VB;                          // two batches
+    T* raw = reinterpret_cast<T*>(sw + (CONST_DECAY ? 0 : 2 * TT * KP));
+    const int raw_batch = TT * ((OUT ? 2 : 1) * KP + VB);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int kg = lane % KG, vg = lane / KG;
     const int h = blockIdx.x, v0 = blockIdx.y * VB;
     const int begin = blockIdx.z * p.chunk, end = min(begin + p.chunk, a.rows);
     const int c_a = warp * S_::CW + vg * 4;            // this lane's columns: c_a .. + 3 and c_a + 4 VG .. + 3
+    const int vcols = min(VB, a.vdim - v0);
+    // columns of the raw rows that nothing is copied to: any finite value
+    for (int i = threadIdx.x; i < 2 * raw_batch; i += blockDim.x) raw[i] = from_float<T>(0.f);
+    if (!CONST_DECAY) {
+        for (int i = threadIdx.x; i < 2 * TT * KP; i += blockDim.x) sw[i] = 0.f;
+    }
+    __syncthreads();
     grid_dependency_sync();
 
-    float S[8][8];
-    float* state = (p.chunk_state != nullptr ? p.chunk_state + static_cast<size_t>(blockIdx.z) * a.heads * KP * p.vp : a.state) +
+    auto fetch = [&](int batch, int row0) {
+        const int n = min(TT, end - row0);
+        T* dst = raw + (batch & 1) * raw_batch;
+        if (OUT) copy_rows<T>(dst, KP, a.r, a.ld_r, row0, h * a.dim, a.dim, n, p.vec_k);
+        copy_rows<T>(dst + (OUT ? TT * KP : 0), KP, a.k, a.ld_k, row0, h * a.dim, a.dim, n, p.vec_k);
+        copy_rows<T>(dst + (OUT ? 2 : 1) * TT * KP, VB, a.v, a.ld_v, row0, h * a.vdim + v0, vcols, n, p.vec_v);
+        if (!CONST_DECAY) copy_rows<float>(sw + (batch & 1) * TT * KP, KP, a.w, a.ld_w, row0, h * a.dim, a.dim, n, p.vec_k);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0, begin);
+
+    // S[i][j]: rows 2 i, 2 i + 1 of this lane's eight, column j
+    f32x2 S[4][8], total[4], bonus[4];
+    const bool chunked = p.chunk_state != nullptr;
+    float* state = (chunked ? p.chunk_state + static_cast<size_t>(blockIdx.z) * a.heads * KP * p.vp : a.state) +
                    static_cast<size_t>(h) * KP * p.vp + v0 + c_a;
     auto k_of = [&](int i) { return (i >> 2) * 4 * KG + kg * 4 + (i & 3); };
-    const bool fresh = p.chunk_state == nullptr && *a.kv_len + a.kv_off == 0;
+    const bool zero = !OUT || (!chunked && *a.kv_len + a.kv_off == 0);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        if (fresh) {
+    for (int i = 0; i < 4; ++i) {
+        float f[2][8];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) S[i][j] = 0.f;
-        } else {
-            const float* q = state + static_cast<size_t>(k_of(i)) * p.vp;
-            const float4 x = *reinterpret_cast<const float4*>(q), y = *reinterpret_cast<const float4*>(q + 4 * S_::VG);
-            S[i][0] = x.x; S[i][1] = x.y; S[i][2] = x.z; S[i][3] = x.w;
-            S[i][4] = y.x; S[i][5] = y.y; S[i][6] = y.z; S[i][7] = y.w;
+        for (int e = 0; e < 2; ++e) {
+            const float* q = state + static_cast<size_t>(k_of(2 * i + e)) * p.vp;
+            float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+            if (!zero) {
+                x = *reinterpret_cast<const float4*>(q);
+                y = *reinterpret_cast<const float4*>(q + 4 * S_::VG);
+            }
+            f[e][0] = x.x; f[e][1] = x.y; f[e][2] = x.z; f[e][3] = x.w;
+            f[e][4] = y.x; f[e][5] = y.y; f[e][6] = y.z; f[e][7] = y.w;
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) S[i][j] = pair(f[0][j], f[1][j]);
+        total[i] = pair(1.f, 1.f);
+        if (OUT && !CONST_DECAY) {
+            float u[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int c = k_of(2 * i + e);
+                u[e] = c < a.dim ? __bfloat162float(a.bonus[h * a.dim + c]) : 0.f;
+            }
+            bonus[i] = pair(u[0], u[1]);
         }
     }
-    const float lam = CONST_DECAY ? a.decay[h] : 0.f;
-    for (int row0 = begin; row0 < end; row0 += TT) {
+    f32x2 w[4];
+    if (CONST_DECAY) {
+        const float d = a.decay[h];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) w[i] = pair(d, d);
+    }
+    int batch = 0;
+    for (int row0 = begin; row0 < end; row0 += TT, ++batch) {
         const int n = min(TT, end - row0);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();   // this batch's raw rows are here, the last batch has been walked over
+        if (row0 + TT < end) fetch(batch + 1, row0 + TT);
+        const T* src = raw + (batch & 1) * raw_batch;
+        if (OUT) convert_rows<T>(sr, src, KP, a.dim, n, a.silu);
+        convert_rows<T>(sk, src + (OUT ? TT * KP : 0), KP, a.dim, n, a.silu);
+        convert_rows<T>(sv, src + (OUT ? 2 : 1) * TT * KP, VB, vcols, n, a.silu);
         __syncthreads();
-        stage<T>(a.r, a.ld_r, h * a.dim, a.dim, row0, n, KP, a.silu, sr);
-        stage<T>(a.k, a.ld_k, h * a.dim, a.dim, row0, n, KP, a.silu, sk);
-        stage<T>(a.v, a.ld_v, h * a.vdim + v0, a.vdim - v0, row0, n, VB, a.silu, sv);
-        if (!CONST_DECAY) stage<float>(a.w, a.ld_w, h * a.dim, a.dim, row0, n, KP, false, sw);
-        __syncthreads();
-        if (!CONST_DECAY) {
-            for (int t = warp; t < n; t += warps) {
-                float b = 0.f;
-                for (int c = lane; c < a.dim; c += 32) b += sr[t * KP + c] * __bfloat162float(a.bonus[h * a.dim + c]) * sk[t * KP + c];
-                b = warp_sum(b);
-                if (lane == 0) sb[t] = b;
-            }
-            __syncthreads();
-        }
+        const float* swb = sw + (batch & 1) * TT * KP;
         for (int t = 0; t < n; ++t) {
-            float r[8], k[8], v[8], o[8];
-            lds8(sr + t * KP + kg * 4, 4 * KG, r);
-            lds8(sk + t * KP + kg * 4, 4 * KG, k);
-            lds8(sv + t * VB + c_a, 4 * S_::VG, v);
-            if (CONST_DECAY) {
+            f32x2 r[4], k[4];
+            float v[8], o[8];
+            lds_pairs<KG>(sk + t * KP + kg * 4, k);
+            if (OUT) lds_pairs<KG>(sr + t * KP + kg * 4, r);
+            if (!CONST_DECAY) lds_pairs<KG>(swb + t * KP + kg * 4, w);
+            {
+                const float4 x = *reinterpret_cast<const float4*>(sv + t * VB + c_a),
+                             y = *reinterpret_cast<const float4*>(sv + t * VB + c_a + 4 * S_::VG);
+                v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+                v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+            }
+            float own = 0.f;   // this lane's share of r . (u k)
+            if (OUT && !CONST_DECAY) {
+                f32x2 b = mul2(mul2(r[0], bonus[0]), k[0]);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
+                for (int i = 1; i < 4; ++i) b = fma2(mul2(r[i], bonus[i]), k[i], b);
+                const float2 f = unpair(b);
+                own = f.x + f.y;
+            }
 #pragma unroll
-                    for (int j = 0; j < 8; ++j) S[i][j] = fmaf(lam, S[i][j], k[i] * v[j]);
+            for (int j = 0; j < 8; ++j) {
+                const f32x2 vv = pair(v[j], v[j]);
+                f32x2 acc = 0;
+                if (OUT && !CONST_DECAY) {
+                    acc = mul2(r[0], S[0][j]);
+#pragma unroll
+                    for (int i = 1; i < 4; ++i) acc = fma2(r[i], S[i][j], acc);
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) S[i][j] = fma2(w[i], S[i][j], mul2(k[i], vv));
+                if (OUT && CONST_DECAY) {
+                    acc = mul2(r[0], S[0][j]);
+#pragma unroll
+                    for (int i = 1; i < 4; ++i) acc = fma2(r[i], S[i][j], acc);
+                }
+                if (OUT) {
+                    const float2 f = unpair(acc);
+                    o[j] = CONST_DECAY ? f.x + f.y : fmaf(own, v[j], f.x + f.y);
                 }
             }
+            if constexpr (OUT) {
+                fold<KG>(o, lane);
+                if (KG <= 8 || (lane & (KG - 1) & ~7) == 0) {
+                    const int j0 = KG == 4 ? (lane & 1) * 4 + ((lane >> 1) & 1) * 2 : (lane & 1) * 4 + ((lane >> 1) & 1) * 2 + ((lane >> 2) & 1);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) o[j] = r[0] * S[0][j];
-#pragma unroll
-            for (int i = 1; i < 8; ++i) {
-#pragma unroll
-                for (int j = 0; j < 8; ++j) o[j] = fmaf(r[i], S[i][j], o[j]);
-            }
-            if (!CONST_DECAY) {
-                float w[8];
-                lds8(sw + t * KP + kg * 4, 4 * KG, w);
-#pragma unroll
-                for (int i = 0; i < 8; ++i) {
-#pragma unroll
-                    for (int j = 0; j < 8; ++j) S[i][j] = fmaf(w[i], S[i][j], k[i] * v[j]);
+                    for (int e = 0; e < (KG == 4 ? 2 : 1); ++e) {
+                        const int j = j0 + e, c = c_a + (j >> 2) * 4 * S_::VG + (j & 3);
+                        if (c < vcols) a.out[static_cast<size_t>(row0 + t) * a.ld_out + h * a.vdim + v0 + c] = o[e];
+                    }
                 }
-            }
-            fold<KG>(o, lane);
-            if (KG <= 8 || (lane & (KG - 1) & ~7) == 0) {
-                const int j0 = KG == 4 ? (lane & 1) * 4 + ((lane >> 1) & 1) * 2 : (lane & 1) * 4 + ((lane >> 1) & 1) * 2 + ((lane >> 2) & 1);
+            } else {
 #pragma unroll
-                for (int e = 0; e < (KG == 4 ? 2 : 1); ++e) {
-                    const int j = j0 + e, c = c_a + (j >> 2) * 4 * S_::VG + (j & 3);
-                    float val = o[e];
-                    if (!CONST_DECAY) val += sb[t] * sv[t * VB + c];
-                    if (v0 + c < a.vdim) a.out[static_cast<size_t>(row0 + t) * a.ld_out + h * a.vdim + v0 + c] = val;
-                }
+                for (int i = 0; i < 4; ++i) total[i] = mul2(total[i], w[i]);
             }
         }
     }
-    if (p.chunk_state == nullptr) {
+    if (!OUT || !chunked) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            float* q = state + static_cast<size_t>(k_of(i)) * p.vp;
-            *reinterpret_cast<float4*>(q) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
-            *reinterpret_cast<float4*>(q + 4 * S_::VG) = make_float4(S[i][4], S[i][5], S[i][6], S[i][7]);
+        for (int i = 0; i < 4; ++i) {
+            float2 f[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) f[j] = unpair(S[i][j]);
+            float* q = state + static_cast<size_t>(k_of(2 * i)) * p.vp;
+            *reinterpret_cast<float4*>(q) = make_float4(f[0].x, f[1].x, f[2].x, f[3].x);
+            *reinterpret_cast<float4*>(q + 4 * S_::VG) = make_float4(f[4].x, f[5].x, f[6].x, f[7].x);
+            q += p.vp;   // the next row
+            *reinterpret_cast<float4*>(q) = make_float4(f[0].y, f[1].y, f[2].y, f[3].y);
+            *reinterpret_cast<float4*>(q + 4 * S_::VG) = make_float4(f[4].y, f[5].y, f[6].y, f[7].y);
         }
     }
-}
-
-// What the tokens of one chunk leave in a state that was zero before it, and the decay over the chunk.
-template <typename T, int KG, bool CONST_DECAY>
-__global__ void __launch_bounds__(128)
-scan_chunk_kernel(const ScanParams p) {
-    using S_ = Shape<KG>;
-    constexpr int KP = S_::KP, TT = S_::TT;
-    const ScanArgs& a = p.a;
-    extern __shared__ float sm[];
-    const int warps = blockDim.x >> 5, VB = warps * S_::CW;
-    float* sk = sm;
-    float* sw = sk + TT * KP;
-    float* sv = sw + (CONST_DECAY ? 0 : TT * KP);
-    float* carry = sv + TT * VB;                       // decay from the tokens already added (later ones) to the chunk's end
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int kg = lane % KG, vg = lane / KG;
-    const int h = blockIdx.x, v0 = blockIdx.y * VB;
-    const int begin = blockIdx.z * p.chunk, end = min(begin + p.chunk, a.rows);
-    const int c_a = warp * S_::CW + vg * 4;
-    grid_dependency_sync();
-    const float lam = CONST_DECAY ? a.decay[h] : 0.f;
-    for (int c = threadIdx.x; c < KP; c += blockDim.x) carry[c] = 1.f;
-    float S[8][8] = {};
-    for (int row1 = end; row1 > begin; row1 -= TT) {
-        const int row0 = max(begin, row1 - TT), n = row1 - row0;
-        __syncthreads();
-        stage<T>(a.k, a.ld_k, h * a.dim, a.dim, row0, n, KP, a.silu, sk);
-        stage<T>(a.v, a.ld_v, h * a.vdim + v0, a.vdim - v0, row0, n, VB, a.silu, sv);
-        if (!CONST_DECAY) stage<float>(a.w, a.ld_w, h * a.dim, a.dim, row0, n, KP, false, sw);
-        __syncthreads();
-        for (int c = threadIdx.x; c < KP; c += blockDim.x) {
-            float d = carry[c];
-            for (int t = n - 1; t >= 0; --t) {
-                sk[t * KP + c] *= d;
-                d *= CONST_DECAY ? lam : sw[t * KP + c];
-            }
-            carry[c] = d;
+    if (!OUT && blockIdx.y == 0 && warp == 0 && vg == 0) {
+        float* d = p.chunk_decay + (static_cast<size_t>(blockIdx.z) * a.heads + h) * KP;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = unpair(total[i]);
+            d[k_of(2 * i)] = f.x;
+            d[k_of(2 * i + 1)] = f.y;
         }
-        __syncthreads();
-        for (int t = 0; t < n; ++t) {
-            float k[8], v[8];
-            lds8(sk + t * KP + kg * 4, 4 * KG, k);
-            lds8(sv + t * VB + c_a, 4 * S_::VG, v);
-#pragma unroll
-            for (int i = 0; i < 8; ++i) {
-#pragma unroll
-                for (int j = 0; j < 8; ++j) S[i][j] = fmaf(k[i], v[j], S[i][j]);
-            }
-        }
-    }
-    float* state = p.chunk_state + (static_cast<size_t>(blockIdx.z) * a.heads + h) * KP * p.vp + v0 + c_a;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        float* q = state + static_cast<size_t>((i >> 2) * 4 * KG + kg * 4 + (i & 3)) * p.vp;
-        *reinterpret_cast<float4*>(q) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
-        *reinterpret_cast<float4*>(q + 4 * S_::VG) = make_float4(S[i][4], S[i][5], S[i][6], S[i][7]);
-    }
-    if (blockIdx.y == 0) {
-        for (int c = threadIdx.x; c < KP; c += blockDim.x) p.chunk_decay[(static_cast<size_t>(blockIdx.z) * a.heads + h) * KP + c] = carry[c];
     }
 }
 
@@ -284,24 +353,176 @@ __global__ void scan_link_kernel(const ScanParams p, int kp) {
     reinterpret_cast<float4*>(a.state)[i] = s;
 }
 
+// ---------------------------------------------------------------- one token
+constexpr int STEP_THREADS = 256;
+constexpr int STEP_LOADS = 16;   // 16-byte pieces of the state per thread
+
+struct StepParams {
+    ScanStepArgs a;
+    int kp, vp, cols;   // state rows and columns; columns per CTA
+};
+
+// blockIdx.x: head; blockIdx.y: block of value columns (one for a time mix, whose norm is per head)
+template <typename T, bool TIME_MIX>
+__global__ void __launch_bounds__(STEP_THREADS)
+scan_step_kernel(const StepParams p) {
+    const ScanArgs& a = p.a.scan;
+    extern __shared__ __align__(16) float sm[];
+    float* sr = sm;                       // [kp]
+    float* sk = sr + p.kp;
+    float* sw = sk + p.kp;
+    float* sv = sw + p.kp;                // [cols]
+    float* red = sv + p.cols;             // [row groups][cols]
+    __shared__ float sh[64];
+    __shared__ float s_own;
+    __shared__ int s_last;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = blockIdx.x, v0 = blockIdx.y * p.cols, vcols = min(p.cols, a.vdim - v0);
+    const int cg = p.cols / 4, groups = STEP_THREADS / cg;
+    const int c4 = (tid % cg) * 4, g = tid / cg;
+    grid_dep_trigger();
+    // the state was last written by the step before, which the host has waited for: it is fetched before this kernel's turn
+    float* state = a.state + static_cast<size_t>(h) * p.kp * p.vp + v0 + c4;
+    float4 S[STEP_LOADS];
+#pragma unroll
+    for (int n = 0; n < STEP_LOADS; ++n) {
+        const int i = g + n * groups;
+        S[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (g < groups && i < p.kp) S[n] = *reinterpret_cast<const float4*>(state + static_cast<size_t>(i) * p.vp);
+    }
+    if (TIME_MIX) {
+        const bf16* w = p.a.w2 + static_cast<size_t>(h) * a.dim * p.a.rank;
+        for (int i = tid * 64; i < a.dim * p.a.rank; i += STEP_THREADS * 64) prefetch_l2(w + i);
+        if (tid * 64 < a.dim) {
+            prefetch_l2(p.a.w0 + h * a.dim + tid * 64);
+            prefetch_l2(a.bonus + h * a.dim + tid * 64);
+            prefetch_l2(p.a.norm + h * a.vdim + tid * 64);
+        }
+    }
+    grid_dep_wait();
+    if (*a.kv_len + a.kv_off == 0) {
+#pragma unroll
+        for (int n = 0; n < STEP_LOADS; ++n) S[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    auto put = [&](float* dst, const void* src, int col0, int cols, int width) {
+        for (int c = tid; c < width; c += STEP_THREADS) {
+            float v = 0.f;
+            if (c < cols) {
+                v = to_float<T>(static_cast<const T*>(src)[col0 + c]);
+                if (!TIME_MIX) v = silu_f32(v);
+            }
+            dst[c] = v;
+        }
+    };
+    put(sr, a.r, h * a.dim, a.dim, p.kp);
+    put(sk, a.k, h * a.dim, a.dim, p.kp);
+    put(sv, a.v, h * a.vdim + v0, vcols, p.cols);
+    if (TIME_MIX) {
+        float* inner = red;               // [rank], before red is needed
+        for (int k = tid; k < p.a.rank; k += STEP_THREADS) inner[k] = tanhf(to_float<T>(static_cast<const T*>(p.a.inner)[k]));
+        __syncthreads();
+        for (int c = warp; c < p.kp; c += STEP_THREADS / 32) {
+            float z = 0.f;
+            if (c < a.dim) {
+                const bf16* w = p.a.w2 + (static_cast<size_t>(h) * a.dim + c) * p.a.rank;
+                for (int k = lane; k < p.a.rank; k += 32) z = fmaf(__bfloat162float(w[k]), inner[k], z);
+                z = warp_sum(z) + __bfloat162float(p.a.w0[h * a.dim + c]);
+            }
+            if (lane == 0) sw[c] = c < a.dim ? expf(-expf(z)) : 0.f;
+        }
+        if (warp == 0) {
+            float b = 0.f;
+            for (int c = lane; c < a.dim; c += 32) b += sr[c] * __bfloat162float(a.bonus[h * a.dim + c]) * sk[c];
+            b = warp_sum(b);
+            if (lane == 0) s_own = b;
+        }
+    }
+    __syncthreads();
+    const float lam = TIME_MIX ? 0.f : a.decay[h];
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (g < groups) {
+        const float4 v = *reinterpret_cast<const float4*>(sv + c4);
+#pragma unroll
+        for (int n = 0; n < STEP_LOADS; ++n) {
+            const int i = g + n * groups;
+            if (i < p.kp) {
+                const float r = sr[i], k = sk[i], w = TIME_MIX ? sw[i] : lam;
+                if (TIME_MIX) {
+                    o.x = fmaf(r, S[n].x, o.x); o.y = fmaf(r, S[n].y, o.y); o.z = fmaf(r, S[n].z, o.z); o.w = fmaf(r, S[n].w, o.w);
+                }
+                S[n].x = fmaf(w, S[n].x, k * v.x); S[n].y = fmaf(w, S[n].y, k * v.y);
+                S[n].z = fmaf(w, S[n].z, k * v.z); S[n].w = fmaf(w, S[n].w, k * v.w);
+                if (!TIME_MIX) {
+                    o.x = fmaf(r, S[n].x, o.x); o.y = fmaf(r, S[n].y, o.y); o.z = fmaf(r, S[n].z, o.z); o.w = fmaf(r, S[n].w, o.w);
+                }
+                *reinterpret_cast<float4*>(state + static_cast<size_t>(i) * p.vp) = S[n];
+            }
+        }
+        *reinterpret_cast<float4*>(red + g * p.cols + c4) = o;
+    }
+    __syncthreads();
+    const T* gate = static_cast<const T*>(p.a.gate);
+    T* out = static_cast<T*>(p.a.out);
+    auto gated = [&](float v, int at, float rs) {
+        const float z = to_float<T>(gate[at]), s = 1.f / (1.f + expf(-z));
+        out[at] = from_float<T>(v * rs * __bfloat162float(p.a.norm[at]) * (TIME_MIX ? z * s : s) * p.a.scale);
+    };
+    if (TIME_MIX) {
+        float ss = 0.f;
+        for (int c = tid; c < vcols; c += STEP_THREADS) {
+            float v = s_own * sv[c];
+            for (int n = 0; n < groups; ++n) v += red[n * p.cols + c];
+            sv[c] = v;
+            ss += v * v;
+        }
+        const float rs = rsqrtf(block_sum2(ss, 0.f, sh).x / a.vdim + p.a.eps);
+        for (int c = tid; c < vcols; c += STEP_THREADS) gated(sv[c], h * a.vdim + c, rs);
+    } else {
+        for (int c = tid; c < vcols; c += STEP_THREADS) {
+            float v = 0.f;
+            for (int n = 0; n < groups; ++n) v += red[n * p.cols + c];
+            a.out[h * a.vdim + v0 + c] = v;
+        }
+        // the CTA counted last has everything for the norm over all heads
+        __threadfence();
+        __syncthreads();
+        if (tid == 0) {
+            const int last = atomicAdd(p.a.ticket, 1) == static_cast<int>(gridDim.x * gridDim.y) - 1;
+            if (last) *p.a.ticket = 0;
+            s_last = last;
+        }
+        __syncthreads();
+        if (s_last == 0) return;
+        __threadfence();
+        const int nv = a.heads * a.vdim;
+        float ss = 0.f;
+        for (int c = tid; c < nv; c += STEP_THREADS) {
+            const float v = __ldcg(a.out + c);
+            ss += v * v;
+        }
+        const float rs = rsqrtf(block_sum2(ss, 0.f, sh).x / nv + p.a.eps);
+        for (int c = tid; c < nv; c += STEP_THREADS) gated(__ldcg(a.out + c), c, rs);
+    }
+}
+
 template <typename T, int KG, bool CONST_DECAY>
 void run_scan(const ScanParams& base, const Geometry& g, cudaStream_t s) {
-    using S_ = Shape<KG>;
+    using M = ScanSmem<T, KG, CONST_DECAY>;
     ScanParams p = base;
     const ScanArgs& a = p.a;
-    const int vb = g.warps * S_::CW;
-    const size_t smem = sizeof(float) * (S_::TT * ((CONST_DECAY ? 2 : 3) * S_::KP + vb) + std::max<int>(S_::TT, S_::KP));
+    const int vb = g.warps * Shape<KG>::CW;
     static bool configured = false;
     if (!configured) {
-        CUDA_CHECK(cudaFuncSetAttribute(scan_kernel<T, KG, CONST_DECAY>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
-        CUDA_CHECK(cudaFuncSetAttribute(scan_chunk_kernel<T, KG, CONST_DECAY>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
+        CUDA_CHECK(cudaFuncSetAttribute(scan_kernel<T, KG, CONST_DECAY, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
+        CUDA_CHECK(cudaFuncSetAttribute(scan_kernel<T, KG, CONST_DECAY, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
         configured = true;
     }
     const dim3 block(g.warps * 32);
-    if (a.rows > kChunk) {
-        p.chunk = kChunk;
-        p.chunks = ceil_div(a.rows, kChunk);
-        launch_kernel(scan_chunk_kernel<T, KG, CONST_DECAY>, dim3(a.heads, g.vblocks, p.chunks), block, smem, s, p);
+    if (a.rows > kMinChunk) {
+        const long long warps = static_cast<long long>(a.heads) * g.vblocks * g.warps * ceil_div(a.rows, 2 * kMinChunk);
+        p.chunk = warps >= 8LL * runtime().num_sms ? 2 * kMinChunk : kMinChunk;
+        p.chunks = ceil_div(a.rows, p.chunk);
+        launch_kernel(scan_kernel<T, KG, CONST_DECAY, false>, dim3(a.heads, g.vblocks, p.chunks), block, M::bytes(vb, false), s, p);
         const size_t n4 = static_cast<size_t>(a.heads) * g.kp * g.vp / 4;
         launch_kernel(scan_link_kernel, dim3(static_cast<unsigned>((n4 + 127) / 128)), dim3(128), 0, s, p, g.kp);
     } else {
@@ -309,7 +530,7 @@ void run_scan(const ScanParams& base, const Geometry& g, cudaStream_t s) {
         p.chunks = 1;
         p.chunk_state = p.chunk_decay = nullptr;
     }
-    launch_kernel(scan_kernel<T, KG, CONST_DECAY>, dim3(a.heads, g.vblocks, p.chunks), block, smem, s, p);
+    launch_kernel(scan_kernel<T, KG, CONST_DECAY, true>, dim3(a.heads, g.vblocks, p.chunks), block, M::bytes(vb, true), s, p);
 }
 
 }  // namespace
@@ -323,7 +544,7 @@ size_t scan_state_floats(int heads, int dim, int vdim) {
 
 size_t scan_workspace_floats(int heads, int dim, int vdim, int rows) {
     const Geometry g = geometry(dim, vdim);
-    return static_cast<size_t>(ceil_div(rows, kChunk)) * heads * g.kp * (g.vp + 1);
+    return static_cast<size_t>(ceil_div(rows, kMinChunk)) * heads * g.kp * (g.vp + 1);
 }
 
 template <typename T>
@@ -336,8 +557,13 @@ void launch_scan(const ScanArgs& a, cudaStream_t s) {
     p.a = a;
     p.vp = g.vp;
     p.chunk = p.chunks = 0;
+    auto aligned = [&](const void* q, int ld, int cols, int es) {
+        return reinterpret_cast<uintptr_t>(q) % 16 == 0 && static_cast<size_t>(ld) * es % 16 == 0 && static_cast<size_t>(cols) * es % 16 == 0;
+    };
+    p.vec_k = aligned(a.r, a.ld_r, a.dim, sizeof(T)) && aligned(a.k, a.ld_k, a.dim, sizeof(T)) && (a.w == nullptr || aligned(a.w, a.ld_w, a.dim, 4));
+    p.vec_v = aligned(a.v, a.ld_v, a.vdim, sizeof(T));
     p.chunk_state = a.ws;
-    p.chunk_decay = a.ws + static_cast<size_t>(ceil_div(a.rows, kChunk)) * a.heads * g.kp * g.vp;
+    p.chunk_decay = a.ws + static_cast<size_t>(ceil_div(a.rows, kMinChunk)) * a.heads * g.kp * g.vp;
     auto run = [&](auto kg) {
         constexpr int KG = decltype(kg)::value;
         if (a.decay != nullptr) run_scan<T, KG, true>(p, g, s);
@@ -350,5 +576,37 @@ void launch_scan(const ScanArgs& a, cudaStream_t s) {
         default: run(std::integral_constant<int, 32>()); break;
     }
 }
+bool scan_step_fits(int dim, int vdim, bool time_mix) {
+    const Geometry g = geometry(dim, vdim);
+    return !time_mix || static_cast<long long>(g.kp) * g.vp <= 4LL * STEP_LOADS * STEP_THREADS;
+}
+
+template <typename T>
+void launch_scan_step(const ScanStepArgs& a, cudaStream_t s) {
+    ProfileScope prof(KC_SCAN, s);
+    const ScanArgs& sc = a.scan;
+    const bool time_mix = sc.bonus != nullptr;
+    CPM_REQUIRE(sc.rows == 1 && scan_fits(sc.dim, sc.vdim) && scan_step_fits(sc.dim, sc.vdim, time_mix), "recurrence step: unsupported sizes");
+    const Geometry g = geometry(sc.dim, sc.vdim);
+    StepParams p;
+    p.a = a;
+    p.kp = g.kp; p.vp = g.vp; p.cols = g.vp;
+    int blocks = 1;
+    if (!time_mix) {
+        while (p.cols % 8 == 0 && (p.kp * p.cols > 4 * STEP_LOADS * STEP_THREADS || (p.cols >= 64 && sc.heads * blocks * 2 <= runtime().num_sms))) {
+            p.cols /= 2;
+            blocks *= 2;
+        }
+    }
+    // columns beyond the real ones need no CTA: their state stays zero
+    const dim3 grid(sc.heads, ceil_div(sc.vdim, p.cols));
+    const int groups = STEP_THREADS / (p.cols / 4);
+    CPM_REQUIRE(groups >= 1 && groups * STEP_LOADS >= p.kp, "recurrence step: unsupported sizes");
+    const size_t smem = sizeof(float) * (3 * p.kp + p.cols + std::max(groups * p.cols, a.rank));
+    if (time_mix) launch_kernel(scan_step_kernel<T, true>, grid, dim3(STEP_THREADS), smem, s, p);
+    else launch_kernel(scan_step_kernel<T, false>, grid, dim3(STEP_THREADS), smem, s, p);
+}
+template void launch_scan_step<bf16>(const ScanStepArgs&, cudaStream_t);
+template void launch_scan_step<float>(const ScanStepArgs&, cudaStream_t);
 template void launch_scan<bf16>(const ScanArgs&, cudaStream_t);
 template void launch_scan<float>(const ScanArgs&, cudaStream_t);

@@ -66,6 +66,9 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* sh) {
     return make_float2(a, b);
 }
 
+// asks for the cache line at p ahead of its use (weights, before the wait for the previous kernel)
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 __device__ __forceinline__ float silu_f32(float v) { return v / (1.f + expf(-v)); }
 
 }  // namespace

@@ -2,6 +2,7 @@
 // and gate of recurrences.  Everything is computed in fp32; T is the dtype of the activations.
 #include <algorithm>
 
+#include "ptx.cuh"
 #include "row_ops.cuh"
 
 namespace {
@@ -68,7 +69,19 @@ __global__ void tanh_norm_kernel(const float* __restrict__ x32, const int32_t* _
 template <typename T>
 __global__ void tanh_residual_kernel(float* __restrict__ x32, const T* __restrict__ delta, const DynTanh post, const DynTanh next,
                                      T* __restrict__ out, int rows, int ld) {
-    grid_dependency_sync();
+    grid_dep_trigger();
+    {
+        const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+        if (rows < 64 && c < ld && threadIdx.x % 8 == 0) {
+            prefetch_l2(post.w + c);
+            prefetch_l2(post.b + c);
+            if (next.w != nullptr) {
+                prefetch_l2(next.w + c);
+                prefetch_l2(next.b + c);
+            }
+        }
+    }
+    grid_dep_wait();
     const size_t base = static_cast<size_t>(blockIdx.x) * ld;
     for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < ld; c += gridDim.y * blockDim.x * 8) {
         float x[8], d[8], y[8];
@@ -152,6 +165,138 @@ side_add_kernel(float* __restrict__ x32, const T* __restrict__ y, const bf16* __
             load_before(t, c, before);
             store_mixes<T>(t, 0, ld, c, h, before);
             store_vec<8>(t.prev + c, h);
+        }
+    }
+}
+
+// ---------------------------------------------------------------- one row through the token side input
+constexpr int SIDE_CTAS = 8, SIDE_THREADS = 512;
+
+// element (row, k) of a matrix with K columns: tile-major (linear_weight_elems) or row-major
+template <typename T>
+__device__ __forceinline__ size_t weight_at(int row, int k, int K) {
+    if constexpr (sizeof(T) == 2) {
+        return (static_cast<size_t>(row >> 7) * (K >> 6) + (k >> 6)) * (128 * 64) + static_cast<size_t>(row & 127) * 64 + (k & 63);
+    } else {
+        return static_cast<size_t>(row) * K + k;
+    }
+}
+
+// One cluster of SIDE_CTAS CTAs.  Every CTA takes the residual sum of the whole row; it computes its share of the gate's rows,
+// which go to all CTAs, then its share of the projection's rows = columns of the stream.
+template <typename T>
+__global__ void __launch_bounds__(SIDE_THREADS)
+side_step_kernel(const SideStepArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float sh[64];
+    __shared__ float s_sum[SIDE_CTAS];
+    const int dim_p = (a.dim + 63) / 64 * 64;
+    float* xs = sm;                // [ld] the stream
+    float* sg = xs + a.ld;         // [dim_p] gated side input
+    float* ys = sg + dim_p;        // [ld / SIDE_CTAS] this CTA's columns of the projection
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int rank = static_cast<int>(ptx::cluster_ctarank());
+    const int share = a.ld / SIDE_CTAS, col0 = rank * share;
+    const int per = (a.dim + SIDE_CTAS - 1) / SIDE_CTAS, g0 = rank * per, g1 = min(g0 + per, a.dim);
+    grid_dep_trigger();
+    {
+        const int kb = a.ld / 64, lines = max(g1 - g0, 0) * kb;
+        for (int i = tid; i < lines; i += SIDE_THREADS) prefetch_l2(a.gate + weight_at<T>(g0 + i / kb, (i % kb) * 64, a.ld));
+        const int pb = dim_p / 64, plines = max(min(share, a.width - col0), 0) * pb;
+        for (int i = tid; i < plines; i += SIDE_THREADS) prefetch_l2(a.proj + weight_at<T>(col0 + i / pb, (i % pb) * 64, dim_p));
+        for (int c = col0 + tid * 64; c < col0 + share; c += SIDE_THREADS * 64) {
+            prefetch_l2(a.norm + c);
+            if (a.next.w != nullptr) {
+                prefetch_l2(a.next.w + c);
+                prefetch_l2(a.next.b + c);
+            }
+            if (a.shift.mu != nullptr) {
+                for (int m = 0; m < kMixes; ++m) prefetch_l2(a.shift.mu + static_cast<size_t>(m) * a.ld + c);
+            }
+        }
+        for (int c = tid * 64; c < a.ld; c += SIDE_THREADS * 64) {
+            prefetch_l2(a.post.w + c);
+            prefetch_l2(a.post.b + c);
+        }
+    }
+    for (int k = tid; k < dim_p; k += SIDE_THREADS) sg[k] = 0.f;
+    grid_dep_wait();
+    for (int c = tid * 8; c < a.ld; c += SIDE_THREADS * 8) {
+        float x[8], d[8], y[8];
+        load_vec<8>(a.x32 + c, x);
+        load_vec<8>(static_cast<const T*>(a.delta) + c, d);
+        tanh_norm8(d, a.post, c, y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += y[e];
+        store_vec<8>(xs + c, x);
+    }
+    int id = a.ids[0];
+    if (id < 0 || id >= a.vocab) id = 0;   // reported by the embedding
+    const bf16* side = a.table + static_cast<size_t>(id) * a.table_ld + a.col0;
+    ptx::cluster_sync();   // xs here; sg zeroed in every CTA
+    for (int row = g0 + warp; row < g1; row += SIDE_THREADS / 32) {
+        float z = 0.f;
+#pragma unroll 4
+        for (int k = lane * 8; k < a.ld; k += 256) {
+            float w[8], x[8];
+            load_vec<8>(a.gate + weight_at<T>(row, k, a.ld), w);
+            load_vec<8>(xs + k, x);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) z = fmaf(w[e], to_float<T>(from_float<T>(x[e])), z);
+        }
+        z = to_float<T>(from_float<T>(warp_sum(z)));
+        const float g = to_float<T>(from_float<T>(gelu_tanh(z) * __bfloat162float(side[row])));
+        if (lane < SIDE_CTAS) ptx::st_cluster_f32(ptx::cluster_map(ptx::smem_u32(sg + row), lane), g);
+    }
+    ptx::cluster_sync();
+    int lpr = 8;           // lanes per row of the projection
+    while (lpr < 32 && lpr * 8 < dim_p) lpr *= 2;
+    const int sub = lane / lpr, sl = lane % lpr, rpw = 32 / lpr;
+    float ss = 0.f;
+    for (int r0 = warp * rpw; r0 < share; r0 += SIDE_THREADS / 32 * rpw) {   // uniform within a warp
+        const int r = r0 + sub, row = col0 + r;
+        float y = 0.f;
+        if (r < share && row < a.width) {
+            for (int k = sl * 8; k < dim_p; k += lpr * 8) {
+                float w[8], g[8];
+                load_vec<8>(a.proj + weight_at<T>(row, k, dim_p), w);
+                load_vec<8>(sg + k, g);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) y = fmaf(w[e], g[e], y);
+            }
+        }
+        for (int o = lpr / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+        y = to_float<T>(from_float<T>(y));
+        if (sl == 0 && r < share) {
+            ys[r] = y;
+            ss += y * y;
+        }
+    }
+    ss = block_sum2(ss, 0.f, sh).x;
+    if (tid < SIDE_CTAS) ptx::st_cluster_f32(ptx::cluster_map(ptx::smem_u32(s_sum + rank), tid), ss);
+    ptx::cluster_sync();
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < SIDE_CTAS; ++i) sum += s_sum[i];
+    const float rs = rsqrtf(sum / a.width + a.eps);
+    for (int i = tid * 8; i < share; i += SIDE_THREADS * 8) {
+        const int c = col0 + i;
+        float x[8], y[8], w[8];
+        load_vec<8>(xs + c, x);
+        load_vec<8>(ys + i, y);
+        load_vec<8>(a.norm + c, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += y[e] * rs * w[e];
+        store_vec<8>(a.x32 + c, x);
+        if (a.next.w == nullptr) continue;
+        float h[8];
+        tanh_norm8(x, a.next, c, h);
+        store_vec<8>(static_cast<T*>(a.h) + c, h);
+        if (a.shift.mu != nullptr) {
+            float before[8];
+            load_before(a.shift, c, before);
+            store_mixes<T>(a.shift, 0, a.ld, c, h, before);
+            store_vec<8>(a.shift.prev + c, h);
         }
     }
 }
@@ -277,6 +422,21 @@ void launch_side_add(float* x32, const T* y, const bf16* w, const DynTanh& next,
     if (vecs <= 512) launch_kernel(side_add_kernel<T, 1>, dim3(rows), dim3(threads), 0, s, x32, y, w, next, h, shift, width, ld, eps);
     else launch_kernel(side_add_kernel<T, 4>, dim3(rows), dim3(threads), 0, s, x32, y, w, next, h, shift, width, ld, eps);
 }
+
+template <typename T>
+void launch_side_step(const SideStepArgs& a, cudaStream_t s) {
+    ProfileScope prof(KC_ROW, s);
+    CPM_REQUIRE(a.ld % 64 == 0 && a.ld <= 16384 && a.dim >= 1 && a.dim <= 4096, "side_step: unsupported sizes");
+    static bool configured = false;
+    if (!configured) {
+        CUDA_CHECK(cudaFuncSetAttribute(side_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
+        configured = true;
+    }
+    const size_t smem = sizeof(float) * (a.ld + pad64(a.dim) + a.ld / SIDE_CTAS);
+    launch_kernel_cluster(side_step_kernel<T>, dim3(SIDE_CTAS), dim3(SIDE_THREADS), smem, s, SIDE_CTAS, a);
+}
+template void launch_side_step<bf16>(const SideStepArgs&, cudaStream_t);
+template void launch_side_step<float>(const SideStepArgs&, cudaStream_t);
 
 template <typename T>
 void launch_decay(const T* x, int ld_x, const bf16* w2, const bf16* w0, int rank, int channels, float* out, int ld_out, int rows, cudaStream_t s) {

@@ -64,11 +64,26 @@ def test_layered_work_counts_match_the_hand_count():
     import bench_layered as b
     mlp = b._moe(6, 2, 32, 2, (4, 2), 16)
     cfg = b._model(64, 4, 2, 8, 3, 2, mlp)                     # two layers, the second one shares the first one's cache
-    assert b.active_ff(cfg) == 2 * 32 + 16
+    assert b.llama_shape("tipetar", cfg)[2] == 2 * 32 + 16
     V = b.VOCAB
-    by, fl = b.bytes_and_flops(cfg, "tipetar", 2, 10)
+    by, fl = b.bytes_and_flops("tipetar", cfg, "tipetar", 2, 10)
     attn = 2 * (2 * 64 * 32) + 2 * 2 * 8 * 64                  # q and o twice, k and v once
-    assert by == {"linear": 2 * (attn + V * 64), "experts": 2 * 2 * 3 * 64 * 80, "attention": 2 * 2 * 3 * 2 * 8 * 2}
+    assert by == {"linear": 2 * (attn + V * 64), "experts": 2 * 2 * 3 * 64 * 80, "attention": 2 * 2 * 3 * 2 * 8 * 2, "scan": 0}
     assert fl["attention"] == 2 * 4 * (3 + 3) * 32 and fl["experts"] == 2 * 2 * 2 * 3 * 64 * 80
-    by, fl = b.bytes_and_flops(cfg, "llama", 2, 10)
-    assert by["experts"] == 0 and fl["attention"] == 2 * 4 * (9 + 10) * 32
+    wide = b._model(256, 4, 2, 64, 3, 2, mlp)
+    by, fl = b.bytes_and_flops("tipetar", wide, "llama", 2, 10)
+    assert by["experts"] == 0 and fl["attention"] == 2 * 4 * (9 + 10) * 256
+
+
+def test_layered_work_counts_of_recurrent_models():
+    import bench_layered as b
+    cfg = b._fabulix(256, (4, 2, 64), (3, 32), (2, 48), 320, 16, 3)      # lightning, parallel, parallel
+    light = 256 * 5 * 96 + 2 * 256 * 16
+    left, right = 256 * (2 * 256 + 2 * 128), 5 * 256 * 96 + b.DECAY_RANK * (256 + 96)
+    par = left + right + 3 * 256 * 320 + 2 * 256 * 16
+    by, fl = b.bytes_and_flops("fabulix", cfg, "fabulix", 2, 10)
+    assert by["linear"] == 2 * (light + 2 * par + b.VOCAB * 256)
+    assert by["scan"] == 8 * (2 * 48 * 48 + 2 * 3 * 32 * 32) and fl["scan"] == 2 * 5 * (by["scan"] // 8)
+    assert by["attention"] == 2 * 2 * 10 * 2 * 64 * 2 and fl["attention"] == 2 * 4 * (9 + 10) * 256
+    hq, hkv, ff = b.llama_shape("fabulix", cfg)
+    assert (hq, hkv) == (2, 1) and abs(256 * 128 * 6 + 3 * 256 * ff - (light + 2 * par) / 3) <= 3 * 256 * 64
