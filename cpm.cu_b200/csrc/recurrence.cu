@@ -404,32 +404,52 @@ scan_step_kernel(const StepParams p) {
 #pragma unroll
         for (int n = 0; n < STEP_LOADS; ++n) S[n] = make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    auto put = [&](float* dst, const void* src, int col0, int cols, int width) {
-        for (int c = tid; c < width; c += STEP_THREADS) {
-            float v = 0.f;
-            if (c < cols) {
-                v = to_float<T>(static_cast<const T*>(src)[col0 + c]);
-                if (!TIME_MIX) v = silu_f32(v);
-            }
-            dst[c] = v;
-        }
+    // what this thread puts into shared memory, loaded before anything is stored
+    auto get = [&](const void* src, int col0, int c, int cols) {
+        if (c >= cols) return 0.f;
+        const float v = to_float<T>(static_cast<const T*>(src)[col0 + c]);
+        return TIME_MIX ? v : silu_f32(v);
     };
-    put(sr, a.r, h * a.dim, a.dim, p.kp);
-    put(sk, a.k, h * a.dim, a.dim, p.kp);
-    put(sv, a.v, h * a.vdim + v0, vcols, p.cols);
+    static_assert(STEP_THREADS >= 256, "one key channel per thread");
+    const float r_t = get(a.r, h * a.dim, tid, a.dim), k_t = get(a.k, h * a.dim, tid, a.dim), v_t = get(a.v, h * a.vdim + v0, tid, vcols);
+    const float x_t = TIME_MIX && tid < p.a.rank ? to_float<T>(static_cast<const T*>(p.a.inner)[tid]) : 0.f;
+    const float z_t = TIME_MIX && tid < vcols ? to_float<T>(static_cast<const T*>(p.a.gate)[h * a.vdim + tid]) : 0.f;
+    if (tid < p.kp) {
+        sr[tid] = r_t;
+        sk[tid] = k_t;
+    }
+    if (tid < p.cols) sv[tid] = v_t;
+    for (int c = tid + STEP_THREADS; c < p.cols; c += STEP_THREADS) sv[c] = get(a.v, h * a.vdim + v0, c, vcols);
     if (TIME_MIX) {
         float* inner = red;               // [rank], before red is needed
-        for (int k = tid; k < p.a.rank; k += STEP_THREADS) inner[k] = tanhf(to_float<T>(static_cast<const T*>(p.a.inner)[k]));
+        if (tid < p.a.rank) inner[tid] = tanhf(x_t);
+        for (int k = tid + STEP_THREADS; k < p.a.rank; k += STEP_THREADS) inner[k] = tanhf(to_float<T>(static_cast<const T*>(p.a.inner)[k]));
         __syncthreads();
-        for (int c = warp; c < p.kp; c += STEP_THREADS / 32) {
-            float z = 0.f;
-            if (c < a.dim) {
-                const bf16* w = p.a.w2 + (static_cast<size_t>(h) * a.dim + c) * p.a.rank;
-                for (int k = lane; k < p.a.rank; k += 32) z = fmaf(__bfloat162float(w[k]), inner[k], z);
-                z = warp_sum(z) + __bfloat162float(p.a.w0[h * a.dim + c]);
+        constexpr int WARPS = STEP_THREADS / 32;
+        for (int c0 = warp; c0 < a.dim; c0 += WARPS * 8) {   // eight channels of a warp at once
+            float z[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const int c = c0 + e * WARPS;
+                z[e] = lane == 0 && c < a.dim ? __bfloat162float(__ldg(p.a.w0 + h * a.dim + c)) : 0.f;
             }
-            if (lane == 0) sw[c] = c < a.dim ? expf(-expf(z)) : 0.f;
+            const bf16* w = p.a.w2 + (static_cast<size_t>(h) * a.dim + c0) * p.a.rank;
+            for (int k = lane; k < p.a.rank; k += 32) {
+                const float in = inner[k];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    if (c0 + e * WARPS < a.dim) z[e] = fmaf(__bfloat162float(__ldg(w + static_cast<size_t>(e) * WARPS * p.a.rank + k)), in, z[e]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) z[e] = warp_sum(z[e]);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const int c = c0 + e * WARPS;
+                if (lane == e && c < a.dim) sw[c] = expf(-expf(z[e]));
+            }
         }
+        if (tid >= a.dim && tid < p.kp) sw[tid] = 0.f;
         if (warp == 0) {
             float b = 0.f;
             for (int c = lane; c < a.dim; c += 32) b += sr[c] * __bfloat162float(a.bonus[h * a.dim + c]) * sk[c];
@@ -463,9 +483,9 @@ scan_step_kernel(const StepParams p) {
     __syncthreads();
     const T* gate = static_cast<const T*>(p.a.gate);
     T* out = static_cast<T*>(p.a.out);
-    auto gated = [&](float v, int at, float rs) {
-        const float z = to_float<T>(gate[at]), s = 1.f / (1.f + expf(-z));
-        out[at] = from_float<T>(v * rs * __bfloat162float(p.a.norm[at]) * (TIME_MIX ? z * s : s) * p.a.scale);
+    auto gated = [&](float v, float z, float w, float rs) {
+        const float s = 1.f / (1.f + expf(-z));
+        return v * rs * w * (TIME_MIX ? z * s : s) * p.a.scale;
     };
     if (TIME_MIX) {
         float ss = 0.f;
@@ -476,7 +496,10 @@ scan_step_kernel(const StepParams p) {
             ss += v * v;
         }
         const float rs = rsqrtf(block_sum2(ss, 0.f, sh).x / a.vdim + p.a.eps);
-        for (int c = tid; c < vcols; c += STEP_THREADS) gated(sv[c], h * a.vdim + c, rs);
+        for (int c = tid; c < vcols; c += STEP_THREADS) {
+            const int at = h * a.vdim + c;
+            out[at] = from_float<T>(gated(sv[c], c == tid ? z_t : to_float<T>(gate[at]), __bfloat162float(__ldg(p.a.norm + at)), rs));
+        }
     } else {
         for (int c = tid; c < vcols; c += STEP_THREADS) {
             float v = 0.f;
@@ -496,12 +519,39 @@ scan_step_kernel(const StepParams p) {
         __threadfence();
         const int nv = a.heads * a.vdim;
         float ss = 0.f;
+        if (nv % 8 == 0 && nv <= STEP_THREADS * 16 && reinterpret_cast<uintptr_t>(gate) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0) {
+            float f[2][8], z[2][8], w[2][8];
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const int c = (tid + n * STEP_THREADS) * 8;
+                if (c >= nv) continue;
+                const float4 x = __ldcg(reinterpret_cast<const float4*>(a.out + c)), y = __ldcg(reinterpret_cast<const float4*>(a.out + c + 4));
+                f[n][0] = x.x; f[n][1] = x.y; f[n][2] = x.z; f[n][3] = x.w;
+                f[n][4] = y.x; f[n][5] = y.y; f[n][6] = y.z; f[n][7] = y.w;
+                load_vec<8>(gate + c, z[n]);
+                load_vec<8>(p.a.norm + c, w[n]);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss += f[n][e] * f[n][e];
+            }
+            const float rs = rsqrtf(block_sum2(ss, 0.f, sh).x / nv + p.a.eps);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const int c = (tid + n * STEP_THREADS) * 8;
+                if (c >= nv) continue;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) f[n][e] = gated(f[n][e], z[n][e], w[n][e], rs);
+                store_vec<8>(out + c, f[n]);
+            }
+            return;
+        }
         for (int c = tid; c < nv; c += STEP_THREADS) {
             const float v = __ldcg(a.out + c);
             ss += v * v;
         }
         const float rs = rsqrtf(block_sum2(ss, 0.f, sh).x / nv + p.a.eps);
-        for (int c = tid; c < nv; c += STEP_THREADS) gated(__ldcg(a.out + c), c, rs);
+        for (int c = tid; c < nv; c += STEP_THREADS) {
+            out[c] = from_float<T>(gated(__ldcg(a.out + c), to_float<T>(gate[c]), __bfloat162float(p.a.norm[c]), rs));
+        }
     }
 }
 

@@ -170,7 +170,7 @@ side_add_kernel(float* __restrict__ x32, const T* __restrict__ y, const bf16* __
 }
 
 // ---------------------------------------------------------------- one row through the token side input
-constexpr int SIDE_CTAS = 8, SIDE_THREADS = 512;
+constexpr int SIDE_CTAS = 16, SIDE_THREADS = 512;   // at most; a cluster of 16 is above the portable size
 
 // element (row, k) of a matrix with K columns: tile-major (linear_weight_elems) or row-major
 template <typename T>
@@ -193,11 +193,12 @@ side_step_kernel(const SideStepArgs a) {
     const int dim_p = (a.dim + 63) / 64 * 64;
     float* xs = sm;                // [ld] the stream
     float* sg = xs + a.ld;         // [dim_p] gated side input
-    float* ys = sg + dim_p;        // [ld / SIDE_CTAS] this CTA's columns of the projection
+    float* ys = sg + dim_p;        // this CTA's columns of the projection
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int rank = static_cast<int>(ptx::cluster_ctarank());
-    const int share = a.ld / SIDE_CTAS, col0 = rank * share;
-    const int per = (a.dim + SIDE_CTAS - 1) / SIDE_CTAS, g0 = rank * per, g1 = min(g0 + per, a.dim);
+    const int ctas = gridDim.x;
+    const int whole = (a.ld / 8 + ctas - 1) / ctas * 8, col0 = min(rank * whole, a.ld), share = min(whole, a.ld - col0);
+    const int per = (a.dim + ctas - 1) / ctas, g0 = rank * per, g1 = min(g0 + per, a.dim);
     grid_dep_trigger();
     {
         const int kb = a.ld / 64, lines = max(g1 - g0, 0) * kb;
@@ -236,7 +237,7 @@ side_step_kernel(const SideStepArgs a) {
     ptx::cluster_sync();   // xs here; sg zeroed in every CTA
     for (int row = g0 + warp; row < g1; row += SIDE_THREADS / 32) {
         float z = 0.f;
-#pragma unroll 4
+#pragma unroll 8
         for (int k = lane * 8; k < a.ld; k += 256) {
             float w[8], x[8];
             load_vec<8>(a.gate + weight_at<T>(row, k, a.ld), w);
@@ -246,38 +247,49 @@ side_step_kernel(const SideStepArgs a) {
         }
         z = to_float<T>(from_float<T>(warp_sum(z)));
         const float g = to_float<T>(from_float<T>(gelu_tanh(z) * __bfloat162float(side[row])));
-        if (lane < SIDE_CTAS) ptx::st_cluster_f32(ptx::cluster_map(ptx::smem_u32(sg + row), lane), g);
+        if (lane < ctas) ptx::st_cluster_f32(ptx::cluster_map(ptx::smem_u32(sg + row), lane), g);
     }
     ptx::cluster_sync();
     int lpr = 8;           // lanes per row of the projection
     while (lpr < 32 && lpr * 8 < dim_p) lpr *= 2;
     const int sub = lane / lpr, sl = lane % lpr, rpw = 32 / lpr;
     float ss = 0.f;
-    for (int r0 = warp * rpw; r0 < share; r0 += SIDE_THREADS / 32 * rpw) {   // uniform within a warp
-        const int r = r0 + sub, row = col0 + r;
-        float y = 0.f;
-        if (r < share && row < a.width) {
-            for (int k = sl * 8; k < dim_p; k += lpr * 8) {
-                float w[8], g[8];
-                load_vec<8>(a.proj + weight_at<T>(row, k, dim_p), w);
-                load_vec<8>(sg + k, g);
+    constexpr int B = 8;   // rows in flight per group of lanes
+    for (int r0 = warp * rpw * B; r0 < share; r0 += SIDE_THREADS / 32 * rpw * B) {   // uniform within a warp
+        float y[B] = {};
+        for (int k = sl * 8; k < dim_p; k += lpr * 8) {
+            float g[8];
+            load_vec<8>(sg + k, g);
+            uint4 w[B];
 #pragma unroll
-                for (int e = 0; e < 8; ++e) y = fmaf(w[e], g[e], y);
+            for (int n = 0; n < B; ++n) {
+                const int r = r0 + n * rpw + sub;
+                w[n] = make_uint4(0, 0, 0, 0);
+                if (r < share && col0 + r < a.width) w[n] = __ldg(reinterpret_cast<const uint4*>(a.proj + weight_at<T>(col0 + r, k, dim_p)));
+            }
+#pragma unroll
+            for (int n = 0; n < B; ++n) {
+                const bf16* e8 = reinterpret_cast<const bf16*>(&w[n]);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) y[n] = fmaf(__bfloat162float(e8[e]), g[e], y[n]);
             }
         }
-        for (int o = lpr / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-        y = to_float<T>(from_float<T>(y));
-        if (sl == 0 && r < share) {
-            ys[r] = y;
-            ss += y * y;
+#pragma unroll
+        for (int n = 0; n < B; ++n) {
+            for (int o = lpr / 2; o > 0; o >>= 1) y[n] += __shfl_xor_sync(0xffffffffu, y[n], o);
+            y[n] = to_float<T>(from_float<T>(y[n]));
+            const int r = r0 + n * rpw + sub;
+            if (sl == 0 && r < share) {
+                ys[r] = y[n];
+                ss += y[n] * y[n];
+            }
         }
     }
     ss = block_sum2(ss, 0.f, sh).x;
-    if (tid < SIDE_CTAS) ptx::st_cluster_f32(ptx::cluster_map(ptx::smem_u32(s_sum + rank), tid), ss);
+    if (tid < ctas) ptx::st_cluster_f32(ptx::cluster_map(ptx::smem_u32(s_sum + rank), tid), ss);
     ptx::cluster_sync();
     float sum = 0.f;
-#pragma unroll
-    for (int i = 0; i < SIDE_CTAS; ++i) sum += s_sum[i];
+    for (int i = 0; i < ctas; ++i) sum += s_sum[i];
     const float rs = rsqrtf(sum / a.width + a.eps);
     for (int i = tid * 8; i < share; i += SIDE_THREADS * 8) {
         const int c = col0 + i;
@@ -427,13 +439,15 @@ template <typename T>
 void launch_side_step(const SideStepArgs& a, cudaStream_t s) {
     ProfileScope prof(KC_ROW, s);
     CPM_REQUIRE(a.ld % 64 == 0 && a.ld <= 16384 && a.dim >= 1 && a.dim <= 4096, "side_step: unsupported sizes");
-    static bool configured = false;
-    if (!configured) {
-        CUDA_CHECK(cudaFuncSetAttribute(side_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
-        configured = true;
+    static int ctas = 0;
+    if (ctas == 0) {
+        constexpr int kSmem = 96 * 1024;
+        CUDA_CHECK(cudaFuncSetAttribute(side_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+        CUDA_CHECK(cudaFuncSetAttribute(side_step_kernel<T>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+        ctas = max_active_clusters(side_step_kernel<T>, dim3(SIDE_THREADS), kSmem, SIDE_CTAS) >= 1 ? SIDE_CTAS : 8;
     }
-    const size_t smem = sizeof(float) * (a.ld + pad64(a.dim) + a.ld / SIDE_CTAS);
-    launch_kernel_cluster(side_step_kernel<T>, dim3(SIDE_CTAS), dim3(SIDE_THREADS), smem, s, SIDE_CTAS, a);
+    const size_t smem = sizeof(float) * (a.ld + pad64(a.dim) + a.ld / 8);
+    launch_kernel_cluster(side_step_kernel<T>, dim3(ctas), dim3(SIDE_THREADS), smem, s, ctas, a);
 }
 template void launch_side_step<bf16>(const SideStepArgs&, cudaStream_t);
 template void launch_side_step<float>(const SideStepArgs&, cudaStream_t);
