@@ -16,7 +16,7 @@
 
 namespace {
 
-constexpr int kMinChunk = 64;   // tokens per chunk: 64 or, when that gives enough warps, 128
+constexpr int kMinChunk = 64;   // fewest tokens per chunk
 constexpr int TT = 8;           // tokens in shared memory
 
 template <int KG>
@@ -50,28 +50,6 @@ struct ScanParams {
     int vec_k, vec_v;        // rows of r, k, w / of v can be copied 16 bytes at a time
 };
 
-// ---- pairs of fp32
-typedef unsigned long long f32x2;
-__device__ __forceinline__ f32x2 pair(float lo, float hi) {
-    f32x2 r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
-    return r;
-}
-__device__ __forceinline__ float2 unpair(f32x2 p) {
-    float2 f;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(p));
-    return f;
-}
-__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
-    f32x2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
-    f32x2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
 // rows kg * 4 .. + 3 and kg * 4 + 4 KG .. + 3 as four pairs
 template <int KG>
 __device__ __forceinline__ void lds_pairs(const float* p, f32x2* f) {
@@ -106,13 +84,18 @@ __device__ __forceinline__ void copy_rows(E* dst, int width, const void* src, in
 template <typename T>
 __device__ __forceinline__ void convert_rows(float* dst, const T* raw, int width, int cols, int n, bool silu) {
     for (int i = threadIdx.x * 8; i < n * width; i += blockDim.x * 8) {
-        const int c = i % width;
         float f[8];
         load_vec<8>(raw + i, f);
+        if (silu) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-            if (silu) f[e] = silu_f32(f[e]);
-            if (c + e >= cols) f[e] = 0.f;
+            for (int e = 0; e < 8; ++e) f[e] = silu_of<T>(f[e]);
+        }
+        if (cols != width) {
+            const int c = i % width;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                if (c + e >= cols) f[e] = 0.f;
+            }
         }
         store_vec<8>(dst + i, f);
     }
@@ -138,16 +121,16 @@ __device__ __forceinline__ void fold(float* o, int lane) {
 template <typename T, int KG, bool CONST_DECAY>
 struct ScanSmem {
     static constexpr int KP = Shape<KG>::KP;
-    // floats: r, k, v of the tokens being walked over, decays of two batches; then the raw rows of two batches
+    // floats: r, k, v of the tokens being walked over, a batch's decay, decays of two batches; then the raw rows of two batches
     static size_t bytes(int vb, bool out) {
         const int keys = out ? 2 : 1;
-        return sizeof(float) * TT * (keys * KP + vb + (CONST_DECAY ? 0 : 2 * KP)) + sizeof(T) * 2 * TT * (keys * KP + vb);
+        return sizeof(float) * (TT * (keys * KP + vb + (CONST_DECAY ? 0 : 2 * KP)) + KP) + sizeof(T) * 2 * TT * (keys * KP + vb);
     }
 };
 
 // OUT: outputs from the state a chunk (or the sequence) begins with; otherwise what a chunk alone leaves behind.
 template <typename T, int KG, bool CONST_DECAY, bool OUT>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 4)
 scan_kernel(const ScanParams p) {
     using S_ = Shape<KG>;
     constexpr int KP = S_::KP;
@@ -157,7 +140,8 @@ scan_kernel(const ScanParams p) {
     float* sr = sm;
     float* sk = sr + (OUT ? TT * KP : 0);
     float* sv = sk + TT * KP;
-    float* sw = sv + TT * VB;                          // two batches
+    float* sd = sv + TT * VB;                          // [KP] decay over a batch
+    float* sw = sd + KP;                               // two batches
     T* raw = reinterpret_cast<T*>(sw + (CONST_DECAY ? 0 : 2 * TT * KP));
     const int raw_batch = TT * ((OUT ? 2 : 1) * KP + VB);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -219,11 +203,21 @@ scan_kernel(const ScanParams p) {
             bonus[i] = pair(u[0], u[1]);
         }
     }
+    const float lam = CONST_DECAY ? a.decay[h] : 0.f;
     f32x2 w[4];
     if (CONST_DECAY) {
-        const float d = a.decay[h];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) w[i] = pair(d, d);
+        for (int i = 0; i < 4; ++i) w[i] = pair(lam, lam);
+    }
+    float* out = nullptr;   // this lane's columns of a token's output
+    bool out_ok[2] = {false, false};
+    if constexpr (OUT) {
+        const int j0 = KG == 4 ? (lane & 1) * 4 + ((lane >> 1) & 1) * 2 : (lane & 1) * 4 + ((lane >> 1) & 1) * 2 + ((lane >> 2) & 1);
+        const int c = c_a + (j0 >> 2) * 4 * S_::VG + (j0 & 3);
+        const bool writes = KG <= 8 || (lane & (KG - 1) & ~7) == 0;
+        out = a.out + static_cast<size_t>(begin) * a.ld_out + h * a.vdim + v0 + c;
+        out_ok[0] = writes && c < vcols;
+        out_ok[1] = KG == 4 && writes && c + 1 < vcols;
     }
     int batch = 0;
     for (int row0 = begin; row0 < end; row0 += TT, ++batch) {
@@ -237,20 +231,49 @@ scan_kernel(const ScanParams p) {
         convert_rows<T>(sv, src + (OUT ? 2 : 1) * TT * KP, VB, vcols, n, a.silu);
         __syncthreads();
         const float* swb = sw + (batch & 1) * TT * KP;
+        if constexpr (!OUT) {
+            // keys decayed to the batch's end, so that the state is scaled once per batch
+            for (int c = threadIdx.x; c < KP; c += blockDim.x) {
+                float d = 1.f;
+                for (int t = n - 1; t >= 0; --t) {
+                    sk[t * KP + c] *= d;
+                    d *= CONST_DECAY ? lam : swb[t * KP + c];
+                }
+                sd[c] = d;
+            }
+            __syncthreads();
+            f32x2 d[4];
+            lds_pairs<KG>(sd + kg * 4, d);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                total[i] = mul2(total[i], d[i]);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) S[i][j] = mul2(S[i][j], d[i]);
+            }
+        }
         for (int t = 0; t < n; ++t) {
             f32x2 r[4], k[4];
             float v[8], o[8];
             lds_pairs<KG>(sk + t * KP + kg * 4, k);
             if (OUT) lds_pairs<KG>(sr + t * KP + kg * 4, r);
-            if (!CONST_DECAY) lds_pairs<KG>(swb + t * KP + kg * 4, w);
+            if (OUT && !CONST_DECAY) lds_pairs<KG>(swb + t * KP + kg * 4, w);
             {
                 const float4 x = *reinterpret_cast<const float4*>(sv + t * VB + c_a),
                              y = *reinterpret_cast<const float4*>(sv + t * VB + c_a + 4 * S_::VG);
                 v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
                 v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
             }
+            if constexpr (!OUT) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const f32x2 vv = pair(v[j], v[j]);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) S[i][j] = fma2(k[i], vv, S[i][j]);
+                }
+                continue;
+            }
             float own = 0.f;   // this lane's share of r . (u k)
-            if (OUT && !CONST_DECAY) {
+            if (!CONST_DECAY) {
                 f32x2 b = mul2(mul2(r[0], bonus[0]), k[0]);
 #pragma unroll
                 for (int i = 1; i < 4; ++i) b = fma2(mul2(r[i], bonus[i]), k[i], b);
@@ -260,38 +283,26 @@ scan_kernel(const ScanParams p) {
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
                 const f32x2 vv = pair(v[j], v[j]);
-                f32x2 acc = 0;
-                if (OUT && !CONST_DECAY) {
+                f32x2 acc;
+                if (!CONST_DECAY) {
                     acc = mul2(r[0], S[0][j]);
 #pragma unroll
                     for (int i = 1; i < 4; ++i) acc = fma2(r[i], S[i][j], acc);
                 }
 #pragma unroll
                 for (int i = 0; i < 4; ++i) S[i][j] = fma2(w[i], S[i][j], mul2(k[i], vv));
-                if (OUT && CONST_DECAY) {
+                if (CONST_DECAY) {
                     acc = mul2(r[0], S[0][j]);
 #pragma unroll
                     for (int i = 1; i < 4; ++i) acc = fma2(r[i], S[i][j], acc);
                 }
-                if (OUT) {
-                    const float2 f = unpair(acc);
-                    o[j] = CONST_DECAY ? f.x + f.y : fmaf(own, v[j], f.x + f.y);
-                }
+                const float2 f = unpair(acc);
+                o[j] = CONST_DECAY ? f.x + f.y : fmaf(own, v[j], f.x + f.y);
             }
-            if constexpr (OUT) {
-                fold<KG>(o, lane);
-                if (KG <= 8 || (lane & (KG - 1) & ~7) == 0) {
-                    const int j0 = KG == 4 ? (lane & 1) * 4 + ((lane >> 1) & 1) * 2 : (lane & 1) * 4 + ((lane >> 1) & 1) * 2 + ((lane >> 2) & 1);
-#pragma unroll
-                    for (int e = 0; e < (KG == 4 ? 2 : 1); ++e) {
-                        const int j = j0 + e, c = c_a + (j >> 2) * 4 * S_::VG + (j & 3);
-                        if (c < vcols) a.out[static_cast<size_t>(row0 + t) * a.ld_out + h * a.vdim + v0 + c] = o[e];
-                    }
-                }
-            } else {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) total[i] = mul2(total[i], w[i]);
-            }
+            fold<KG>(o, lane);
+            if (out_ok[0]) out[0] = o[0];
+            if (out_ok[1]) out[1] = o[1];
+            out += a.ld_out;
         }
     }
     if (!OUT || !chunked) {
@@ -408,7 +419,7 @@ scan_step_kernel(const StepParams p) {
     auto get = [&](const void* src, int col0, int c, int cols) {
         if (c >= cols) return 0.f;
         const float v = to_float<T>(static_cast<const T*>(src)[col0 + c]);
-        return TIME_MIX ? v : silu_f32(v);
+        return TIME_MIX ? v : silu_of<T>(v);
     };
     static_assert(STEP_THREADS >= 256, "one key channel per thread");
     const float r_t = get(a.r, h * a.dim, tid, a.dim), k_t = get(a.k, h * a.dim, tid, a.dim), v_t = get(a.v, h * a.vdim + v0, tid, vcols);
@@ -569,8 +580,10 @@ void run_scan(const ScanParams& base, const Geometry& g, cudaStream_t s) {
     }
     const dim3 block(g.warps * 32);
     if (a.rows > kMinChunk) {
-        const long long warps = static_cast<long long>(a.heads) * g.vblocks * g.warps * ceil_div(a.rows, 2 * kMinChunk);
-        p.chunk = warps >= 8LL * runtime().num_sms ? 2 * kMinChunk : kMinChunk;
+        // the shortest chunks whose CTAs all run at once (128 registers: 16 warps per SM), up to four times the shortest
+        const long long slots = static_cast<long long>(runtime().num_sms) * (16 / g.warps);
+        p.chunk = kMinChunk;
+        while (p.chunk < 4 * kMinChunk && static_cast<long long>(a.heads) * g.vblocks * ceil_div(a.rows, p.chunk) > slots) p.chunk *= 2;
         p.chunks = ceil_div(a.rows, p.chunk);
         launch_kernel(scan_kernel<T, KG, CONST_DECAY, false>, dim3(a.heads, g.vblocks, p.chunks), block, M::bytes(vb, false), s, p);
         const size_t n4 = static_cast<size_t>(a.heads) * g.kp * g.vp / 4;

@@ -70,5 +70,32 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* sh) {
 __device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 __device__ __forceinline__ float silu_f32(float v) { return v / (1.f + expf(-v)); }
+// of a value that is known to bf16 precision only: the approximate exponential and division are far finer than that
+__device__ __forceinline__ float silu_fast(float v) { return __fdividef(v, 1.f + __expf(-v)); }
+template <typename T>
+__device__ __forceinline__ float silu_of(float v) { return sizeof(T) == 2 ? silu_fast(v) : silu_f32(v); }
+
+// ---- pairs of fp32 for the packed instructions
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pair(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 unpair(f32x2 p) {
+    float2 f;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(p));
+    return f;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 
 }  // namespace

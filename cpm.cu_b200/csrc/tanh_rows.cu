@@ -205,22 +205,34 @@ side_step_kernel(const SideStepArgs a) {
         for (int i = tid; i < lines; i += SIDE_THREADS) prefetch_l2(a.gate + weight_at<T>(g0 + i / kb, (i % kb) * 64, a.ld));
         const int pb = dim_p / 64, plines = max(min(share, a.width - col0), 0) * pb;
         for (int i = tid; i < plines; i += SIDE_THREADS) prefetch_l2(a.proj + weight_at<T>(col0 + i / pb, (i % pb) * 64, dim_p));
-        for (int c = col0 + tid * 64; c < col0 + share; c += SIDE_THREADS * 64) {
-            prefetch_l2(a.norm + c);
-            if (a.next.w != nullptr) {
-                prefetch_l2(a.next.w + c);
-                prefetch_l2(a.next.b + c);
-            }
-            if (a.shift.mu != nullptr) {
-                for (int m = 0; m < kMixes; ++m) prefetch_l2(a.shift.mu + static_cast<size_t>(m) * a.ld + c);
-            }
-        }
         for (int c = tid * 64; c < a.ld; c += SIDE_THREADS * 64) {
             prefetch_l2(a.post.w + c);
             prefetch_l2(a.post.b + c);
         }
     }
     for (int k = tid; k < dim_p; k += SIDE_THREADS) sg[k] = 0.f;
+    // what this thread's columns need at the end (all weights, and the mixer input of the step before, which the host has waited for)
+    const int mine = col0 + tid * 8;
+    const bool has = tid * 8 < share;
+    uint4 w_norm, w_next, b_next, w_mu[kMixes];
+    float prev[8];
+    w_norm = w_next = b_next = make_uint4(0, 0, 0, 0);
+#pragma unroll
+    for (int m = 0; m < kMixes; ++m) w_mu[m] = make_uint4(0, 0, 0, 0);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) prev[e] = 0.f;
+    if (has) {
+        w_norm = *reinterpret_cast<const uint4*>(a.norm + mine);
+        if (a.next.w != nullptr) {
+            w_next = *reinterpret_cast<const uint4*>(a.next.w + mine);
+            b_next = *reinterpret_cast<const uint4*>(a.next.b + mine);
+        }
+        if (a.shift.mu != nullptr) {
+#pragma unroll
+            for (int m = 0; m < kMixes; ++m) w_mu[m] = *reinterpret_cast<const uint4*>(a.shift.mu + static_cast<size_t>(m) * a.ld + mine);
+            load_vec<8>(a.shift.prev + mine, prev);
+        }
+    }
     grid_dep_wait();
     for (int c = tid * 8; c < a.ld; c += SIDE_THREADS * 8) {
         float x[8], d[8], y[8];
@@ -291,65 +303,89 @@ side_step_kernel(const SideStepArgs a) {
     float sum = 0.f;
     for (int i = 0; i < ctas; ++i) sum += s_sum[i];
     const float rs = rsqrtf(sum / a.width + a.eps);
-    for (int i = tid * 8; i < share; i += SIDE_THREADS * 8) {
-        const int c = col0 + i;
-        float x[8], y[8], w[8];
-        load_vec<8>(xs + c, x);
-        load_vec<8>(ys + i, y);
-        load_vec<8>(a.norm + c, w);
+    if (!has) return;   // share <= 8 * SIDE_THREADS
+    auto bf8 = [](const uint4& u, int e) { return __bfloat162float(reinterpret_cast<const bf16*>(&u)[e]); };
+    float x[8], y[8], h[8];
+    load_vec<8>(xs + mine, x);
+    load_vec<8>(ys + tid * 8, y);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] += y[e] * rs * w[e];
-        store_vec<8>(a.x32 + c, x);
-        if (a.next.w == nullptr) continue;
-        float h[8];
-        tanh_norm8(x, a.next, c, h);
-        store_vec<8>(static_cast<T*>(a.h) + c, h);
-        if (a.shift.mu != nullptr) {
-            float before[8];
-            load_before(a.shift, c, before);
-            store_mixes<T>(a.shift, 0, a.ld, c, h, before);
-            store_vec<8>(a.shift.prev + c, h);
-        }
+    for (int e = 0; e < 8; ++e) x[e] += y[e] * rs * bf8(w_norm, e);
+    store_vec<8>(a.x32 + mine, x);
+    if (a.next.w == nullptr) return;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) h[e] = tanh_norm(x[e], a.next.alpha, bf8(w_next, e), bf8(b_next, e));
+    store_vec<8>(static_cast<T*>(a.h) + mine, h);
+    if (a.shift.mu == nullptr) return;
+    const bool first = *a.shift.kv_len + a.shift.kv_off == 0;
+#pragma unroll
+    for (int m = 0; m < kMixes; ++m) {
+        float f[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = h[e] + ((first ? 0.f : prev[e]) - h[e]) * bf8(w_mu[m], e);
+        store_vec<8>(static_cast<T*>(a.shift.out) + m * a.shift.stride + mine, f);
     }
+    store_vec<8>(a.shift.prev + mine, h);
 }
 
-// kDecayRows tokens x 256 channels per CTA, one channel per thread.
-constexpr int kDecayRows = 8;
+// ROWS tokens x 256 channels per CTA, two channels per thread.
+constexpr int DECAY_THREADS = 128;
 
-template <typename T>
-__global__ void decay_kernel(const T* __restrict__ x, int ld_x, const bf16* __restrict__ w2, const bf16* __restrict__ w0, int rank, int channels,
-                             float* __restrict__ out, int ld_out, int rows) {
-    extern __shared__ float inner[];   // [rank][kDecayRows]
-    const int row0 = blockIdx.y * kDecayRows, n = min(kDecayRows, rows - row0);
+template <typename T, int ROWS>
+__global__ void __launch_bounds__(DECAY_THREADS)
+decay_kernel(const T* __restrict__ x, int ld_x, const bf16* __restrict__ w2, const bf16* __restrict__ w0, int rank, int channels,
+             float* __restrict__ out, int ld_out, int rows) {
+    extern __shared__ __align__(16) float inner[];   // [rank][ROWS]
+    const int row0 = blockIdx.y * ROWS, n = min(ROWS, rows - row0);
     grid_dependency_sync();
-    for (int i = threadIdx.x; i < kDecayRows * rank; i += blockDim.x) {
+    for (int i = threadIdx.x; i < ROWS * rank; i += DECAY_THREADS) {
         const int t = i / rank, k = i - t * rank;
-        inner[k * kDecayRows + t] = t < n ? tanhf(to_float<T>(x[static_cast<size_t>(row0 + t) * ld_x + k])) : 0.f;
+        inner[k * ROWS + t] = t < n ? tanhf(to_float<T>(x[static_cast<size_t>(row0 + t) * ld_x + k])) : 0.f;
     }
     __syncthreads();
-    const int c = blockIdx.x * blockDim.x + threadIdx.x;
-    if (c >= channels) return;
-    const float b = __bfloat162float(w0[c]);
-    float z[kDecayRows];
+    int c[2];
+    const bf16* w[2];
+    f32x2 z[2][ROWS / 2];
 #pragma unroll
-    for (int t = 0; t < kDecayRows; ++t) z[t] = b;
-    const bf16* w = w2 + static_cast<size_t>(c) * rank;
-    auto add = [&](float wk, int k) {
-        const float4 p = *reinterpret_cast<const float4*>(inner + k * kDecayRows), q = *reinterpret_cast<const float4*>(inner + k * kDecayRows + 4);
-        z[0] = fmaf(wk, p.x, z[0]); z[1] = fmaf(wk, p.y, z[1]); z[2] = fmaf(wk, p.z, z[2]); z[3] = fmaf(wk, p.w, z[3]);
-        z[4] = fmaf(wk, q.x, z[4]); z[5] = fmaf(wk, q.y, z[5]); z[6] = fmaf(wk, q.z, z[6]); z[7] = fmaf(wk, q.w, z[7]);
+    for (int m = 0; m < 2; ++m) {
+        c[m] = blockIdx.x * 2 * DECAY_THREADS + m * DECAY_THREADS + threadIdx.x;
+        const int at = min(c[m], channels - 1);
+        w[m] = w2 + static_cast<size_t>(at) * rank;
+        const float b = __bfloat162float(w0[at]);
+#pragma unroll
+        for (int t = 0; t < ROWS / 2; ++t) z[m][t] = pair(b, b);
+    }
+    auto add = [&](float a, float b, int k) {
+        const f32x2 wa = pair(a, a), wb = pair(b, b);
+#pragma unroll
+        for (int t = 0; t < ROWS / 2; t += 2) {
+            const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(inner + k * ROWS + 2 * t);
+            z[0][t] = fma2(wa, v.x, z[0][t]);
+            z[0][t + 1] = fma2(wa, v.y, z[0][t + 1]);
+            z[1][t] = fma2(wb, v.x, z[1][t]);
+            z[1][t + 1] = fma2(wb, v.y, z[1][t + 1]);
+        }
     };
     if (rank % 8 == 0) {
         for (int k = 0; k < rank; k += 8) {
-            float f[8];
-            load_vec<8>(w + k, f);
+            float f[2][8];
+            load_vec<8>(w[0] + k, f[0]);
+            load_vec<8>(w[1] + k, f[1]);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) add(f[e], k + e);
+            for (int e = 0; e < 8; ++e) add(f[0][e], f[1][e], k + e);
         }
     } else {
-        for (int k = 0; k < rank; ++k) add(__bfloat162float(w[k]), k);
+        for (int k = 0; k < rank; ++k) add(__bfloat162float(w[0][k]), __bfloat162float(w[1][k]), k);
     }
-    for (int t = 0; t < n; ++t) out[static_cast<size_t>(row0 + t) * ld_out + c] = expf(-expf(z[t]));
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+        if (c[m] >= channels) continue;
+#pragma unroll
+        for (int t = 0; t < ROWS / 2; ++t) {
+            const float2 f = unpair(z[m][t]);
+            if (2 * t < n) out[static_cast<size_t>(row0 + 2 * t) * ld_out + c[m]] = expf(-expf(f.x));
+            if (2 * t + 1 < n) out[static_cast<size_t>(row0 + 2 * t + 1) * ld_out + c[m]] = expf(-expf(f.y));
+        }
+    }
 }
 
 // One CTA per row; one warp per group, or the whole CTA for a single group.
@@ -378,6 +414,46 @@ __global__ void norm_gate_kernel(const float* __restrict__ o, int ld_o, int grou
             const float rs = rsqrtf(warp_sum(ss) / group + eps);
             for (int c = g * group + lane; c < (g + 1) * group; c += 32) finish(c, rs);
         }
+    }
+}
+
+// The same with 8 columns per thread: `lanes` neighbouring threads hold a group (a power of two, at most a warp), or the CTA holds
+// the single group, at most 8 * VPT columns per thread.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(256)
+norm_gate8_kernel(const float* __restrict__ o, int ld_o, int lanes, int cols, int group, const bf16* __restrict__ w, const T* __restrict__ gate,
+                  int ld_gate, int silu, float eps, float scale, T* __restrict__ out, int ld_out) {
+    grid_dependency_sync();
+    __shared__ float sh[64];
+    o += static_cast<size_t>(blockIdx.x) * ld_o;
+    gate += static_cast<size_t>(blockIdx.x) * ld_gate;
+    out += static_cast<size_t>(blockIdx.x) * ld_out;
+    float v[VPT][8], g[VPT][8], wv[VPT][8], ss[VPT], sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int c = (threadIdx.x + j * blockDim.x) * 8;
+        ss[j] = 0.f;
+        if (c >= cols) continue;
+        load_vec<8>(o + c, v[j]);
+        load_vec<8>(gate + c, g[j]);
+        load_vec<8>(w + c, wv[j]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss[j] += v[j][e] * v[j][e];
+        sum += ss[j];
+    }
+    if (lanes == 0) sum = block_sum2(sum, 0.f, sh).x;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        for (int m = lanes / 2; m > 0; m >>= 1) ss[j] += __shfl_xor_sync(0xffffffffu, ss[j], m);
+        const int c = (threadIdx.x + j * blockDim.x) * 8;
+        if (c >= cols) continue;
+        const float rs = rsqrtf((lanes == 0 ? sum : ss[j]) / group + eps) * scale;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            const float s = sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-g[j][e])) : 1.f / (1.f + expf(-g[j][e]));
+            v[j][e] = v[j][e] * rs * wv[j][e] * (silu ? g[j][e] * s : s);
+        }
+        store_vec<8>(out + c, v[j]);
     }
 }
 
@@ -456,14 +532,31 @@ template <typename T>
 void launch_decay(const T* x, int ld_x, const bf16* w2, const bf16* w0, int rank, int channels, float* out, int ld_out, int rows, cudaStream_t s) {
     ProfileScope prof(KC_ROW, s);
     CPM_REQUIRE(rank >= 1 && rank <= 1024, "time mix: inner width of the decay must be in [1, 1024]");
-    launch_kernel(decay_kernel<T>, dim3(ceil_div(channels, 256), ceil_div(rows, kDecayRows)), dim3(256), rank * kDecayRows * sizeof(float), s, x, ld_x,
-                  w2, w0, rank, channels, out, ld_out, rows);
+    const int blocks = ceil_div(channels, 2 * DECAY_THREADS);
+    auto run = [&](auto kernel, int n) {
+        launch_kernel(kernel, dim3(blocks, ceil_div(rows, n)), dim3(DECAY_THREADS), rank * n * sizeof(float), s, x, ld_x, w2, w0, rank, channels, out,
+                      ld_out, rows);
+    };
+    if (rows >= 256 && rank <= 512) run(decay_kernel<T, 16>, 16);
+    else run(decay_kernel<T, 4>, 4);
 }
 
 template <typename T>
 void launch_norm_gate(const float* o, int ld_o, int groups, int group, const bf16* w, const T* gate, int ld_gate, bool silu, float eps,
                       float scale, T* out, int ld_out, int rows, cudaStream_t s) {
     ProfileScope prof(KC_ROW, s);
+    const int lanes = groups == 1 ? 0 : group / 8, cols = groups * group;
+    const bool wide = group % 8 == 0 && (lanes & (lanes - 1)) == 0 && lanes <= 32 && ld_o % 4 == 0 && ld_gate % 8 == 0 && ld_out % 8 == 0 &&
+                      reinterpret_cast<uintptr_t>(gate) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0 && cols <= 4 * 256 * 8;
+    if (wide) {
+        auto run = [&](auto kernel) {
+            launch_kernel(kernel, dim3(rows), dim3(256), 0, s, o, ld_o, lanes, cols, group, w, gate, ld_gate, silu ? 1 : 0, eps, scale, out, ld_out);
+        };
+        if (cols <= 256 * 8) run(norm_gate8_kernel<T, 1>);
+        else if (cols <= 2 * 256 * 8) run(norm_gate8_kernel<T, 2>);
+        else run(norm_gate8_kernel<T, 4>);
+        return;
+    }
     launch_kernel(norm_gate_kernel<T>, dim3(rows), dim3(256), 0, s, o, ld_o, groups, group, w, gate, ld_gate, silu ? 1 : 0, eps, scale, out,
                   ld_out);
 }
