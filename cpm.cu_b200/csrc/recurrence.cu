@@ -1,9 +1,9 @@
 // Recurrences with an outer-product state (layered.cuh: ScanArgs) on the fp32 pipes.
 //
-// A warp holds 8 * KG rows (key channels) x 8 * (32 / KG) columns (value channels) of a head's state in registers, 8 x 8 per
+// A warp holds 16 * KG rows (key channels) x 4 * (32 / KG) columns (value channels) of a head's state in registers, 16 x 4 per
 // lane as pairs of rows for the packed fp32 instructions, and walks over the tokens; r, k, w, v of a few tokens at a time lie
 // in shared memory, the next ones on their way.  The output of a token is a sum over the KG lanes of a column, folded so that
-// every lane ends up with one column.
+// a lane ends up with one column (two for KG = 2).
 //
 // Long portions are cut into chunks: a first walk over every chunk alone, from a zero state and without outputs, leaves what
 // the chunk adds to the state and its decay, scan_link_kernel runs over the chunks and replaces that by the state each chunk
@@ -21,9 +21,9 @@ constexpr int TT = 8;           // tokens in shared memory
 
 template <int KG>
 struct Shape {
-    static constexpr int KP = 8 * KG;           // key channels, padded
+    static constexpr int KP = 16 * KG;          // key channels, padded
     static constexpr int VG = 32 / KG;
-    static constexpr int CW = 8 * VG;           // value columns per warp
+    static constexpr int CW = 4 * VG;           // value columns per warp
 };
 
 struct Geometry {
@@ -31,11 +31,11 @@ struct Geometry {
 };
 Geometry geometry(int dim, int vdim) {
     Geometry g;
-    g.kg = dim <= 32 ? 4 : dim <= 64 ? 8 : dim <= 128 ? 16 : 32;
-    const int cw = 8 * (32 / g.kg);
+    g.kg = dim <= 32 ? 2 : dim <= 64 ? 4 : dim <= 128 ? 8 : 16;
+    const int cw = 4 * (32 / g.kg);
     g.warps = std::min(4, ceil_div(vdim, cw));
     g.vblocks = ceil_div(vdim, g.warps * cw);
-    g.kp = 8 * g.kg;
+    g.kp = 16 * g.kg;
     g.vp = g.vblocks * g.warps * cw;
     return g;
 }
@@ -49,13 +49,6 @@ struct ScanParams {
     int chunks;
     int vec_k, vec_v;        // rows of r, k, w / of v can be copied 16 bytes at a time
 };
-
-// rows kg * 4 .. + 3 and kg * 4 + 4 KG .. + 3 as four pairs
-template <int KG>
-__device__ __forceinline__ void lds_pairs(const float* p, f32x2* f) {
-    const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(p), b = *reinterpret_cast<const ulonglong2*>(p + 4 * KG);
-    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
-}
 
 __device__ __forceinline__ void copy16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src) : "memory");
@@ -101,11 +94,34 @@ __device__ __forceinline__ void convert_rows(float* dst, const T* raw, int width
     }
 }
 
-// Sum over the KG lanes of a column group.  Afterwards the lane holds the sums of columns fold_column() (+ 1 for KG = 4).
+// r and k of a batch at once, and own[t] = r . (u k)
+template <typename T, int KP>
+__device__ __forceinline__ void convert_keys(float* sr, float* sk, const T* raw_r, const T* raw_k, const float* su, float* own, int cols) {
+    // whole warps stay together: TT * KP / 8 is a multiple of 32
+    for (int i = threadIdx.x * 8; i < TT * KP; i += blockDim.x * 8) {
+        const int c = i % KP;
+        float r[8], k[8], u[8], b = 0.f;
+        load_vec<8>(raw_r + i, r);
+        load_vec<8>(raw_k + i, k);
+        load_vec<8>(su + c, u);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            if (cols != KP && c + e >= cols) r[e] = k[e] = 0.f;
+            b = fmaf(r[e] * u[e], k[e], b);
+        }
+        store_vec<8>(sr + i, r);
+        store_vec<8>(sk + i, k);
+#pragma unroll
+        for (int o = KP / 16; o > 0; o >>= 1) b += __shfl_xor_sync(0xffffffffu, b, o);
+        if (c == 0) own[i / KP] = b;
+    }
+}
+
+// Sum over the KG lanes of a column group: afterwards the lane holds column fold_column() (and the next one for KG = 2).
 template <int KG>
 __device__ __forceinline__ void fold(float* o, int lane) {
 #pragma unroll
-    for (int b = 0, n = 4; b < 3; ++b, n /= 2) {
+    for (int b = 0, n = 2; b < 2; ++b, n /= 2) {
         if ((1 << b) >= KG) break;
         const bool up = (lane >> b) & 1;
 #pragma unroll
@@ -115,16 +131,21 @@ __device__ __forceinline__ void fold(float* o, int lane) {
         }
     }
 #pragma unroll
-    for (int b = 8; b < KG; b *= 2) o[0] += __shfl_xor_sync(0xffffffffu, o[0], b);
+    for (int b = 4; b < KG; b *= 2) o[0] += __shfl_xor_sync(0xffffffffu, o[0], b);
+}
+template <int KG>
+__device__ __forceinline__ int fold_column(int lane) {
+    return KG == 2 ? (lane & 1) * 2 : (lane & 1) * 2 + ((lane >> 1) & 1);
 }
 
 template <typename T, int KG, bool CONST_DECAY>
 struct ScanSmem {
     static constexpr int KP = Shape<KG>::KP;
-    // floats: r, k, v of the tokens being walked over, a batch's decay, decays of two batches; then the raw rows of two batches
+    // floats: r, k, v of the tokens being walked over, two rows of key channels, a number per token, decays of two batches; then
+    // the raw rows of two batches
     static size_t bytes(int vb, bool out) {
         const int keys = out ? 2 : 1;
-        return sizeof(float) * (TT * (keys * KP + vb + (CONST_DECAY ? 0 : 2 * KP)) + KP) + sizeof(T) * 2 * TT * (keys * KP + vb);
+        return sizeof(float) * (TT * (keys * KP + vb + (CONST_DECAY ? 0 : 2 * KP)) + 2 * KP + TT) + sizeof(T) * 2 * TT * (keys * KP + vb);
     }
 };
 
@@ -140,15 +161,17 @@ scan_kernel(const ScanParams p) {
     float* sr = sm;
     float* sk = sr + (OUT ? TT * KP : 0);
     float* sv = sk + TT * KP;
-    float* sd = sv + TT * VB;                          // [KP] decay over a batch
-    float* sw = sd + KP;                               // two batches
+    float* sd = sv + TT * VB;                          // [KP] decay over a batch, or the bonus
+    float* stot = sd + KP;                             // [KP] decay over the chunk so far
+    float* own = stot + KP;                            // [TT] r . (u k)
+    float* sw = own + TT;                              // two batches
     T* raw = reinterpret_cast<T*>(sw + (CONST_DECAY ? 0 : 2 * TT * KP));
     const int raw_batch = TT * ((OUT ? 2 : 1) * KP + VB);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int kg = lane % KG, vg = lane / KG;
     const int h = blockIdx.x, v0 = blockIdx.y * VB;
     const int begin = blockIdx.z * p.chunk, end = min(begin + p.chunk, a.rows);
-    const int c_a = warp * S_::CW + vg * 4;            // this lane's columns: c_a .. + 3 and c_a + 4 VG .. + 3
+    const int c_a = warp * S_::CW + vg * 4;            // this lane's columns: c_a .. + 3
     const int vcols = min(VB, a.vdim - v0);
     // columns of the raw rows that nothing is copied to: any finite value
     for (int i = threadIdx.x; i < 2 * raw_batch; i += blockDim.x) raw[i] = from_float<T>(0.f);
@@ -169,56 +192,34 @@ scan_kernel(const ScanParams p) {
     };
     fetch(0, begin);
 
-    // S[i][j]: rows 2 i, 2 i + 1 of this lane's eight, column j
-    f32x2 S[4][8], total[4], bonus[4];
+    if (OUT && !CONST_DECAY) {
+        for (int c = threadIdx.x; c < KP; c += blockDim.x) sd[c] = c < a.dim ? __bfloat162float(a.bonus[h * a.dim + c]) : 0.f;
+    }
+    if (!OUT) {
+        for (int c = threadIdx.x; c < KP; c += blockDim.x) stot[c] = 1.f;
+    }
+    // S[i][j]: rows k_of(i), k_of(i) + 1, column j
+    f32x2 S[8][4];
     const bool chunked = p.chunk_state != nullptr;
     float* state = (chunked ? p.chunk_state + static_cast<size_t>(blockIdx.z) * a.heads * KP * p.vp : a.state) +
                    static_cast<size_t>(h) * KP * p.vp + v0 + c_a;
-    auto k_of = [&](int i) { return (i >> 2) * 4 * KG + kg * 4 + (i & 3); };
+    auto k_of = [&](int i) { return (i >> 1) * 4 * KG + kg * 4 + (i & 1) * 2; };
     const bool zero = !OUT || (!chunked && *a.kv_len + a.kv_off == 0);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        float f[2][8];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const float* q = state + static_cast<size_t>(k_of(2 * i + e)) * p.vp;
-            float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
-            if (!zero) {
-                x = *reinterpret_cast<const float4*>(q);
-                y = *reinterpret_cast<const float4*>(q + 4 * S_::VG);
-            }
-            f[e][0] = x.x; f[e][1] = x.y; f[e][2] = x.z; f[e][3] = x.w;
-            f[e][4] = y.x; f[e][5] = y.y; f[e][6] = y.z; f[e][7] = y.w;
+    for (int i = 0; i < 8; ++i) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+        if (!zero) {
+            const float* q = state + static_cast<size_t>(k_of(i)) * p.vp;
+            x = *reinterpret_cast<const float4*>(q);
+            y = *reinterpret_cast<const float4*>(q + p.vp);
         }
-#pragma unroll
-        for (int j = 0; j < 8; ++j) S[i][j] = pair(f[0][j], f[1][j]);
-        total[i] = pair(1.f, 1.f);
-        if (OUT && !CONST_DECAY) {
-            float u[2];
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int c = k_of(2 * i + e);
-                u[e] = c < a.dim ? __bfloat162float(a.bonus[h * a.dim + c]) : 0.f;
-            }
-            bonus[i] = pair(u[0], u[1]);
-        }
+        S[i][0] = pair(x.x, y.x); S[i][1] = pair(x.y, y.y); S[i][2] = pair(x.z, y.z); S[i][3] = pair(x.w, y.w);
     }
     const float lam = CONST_DECAY ? a.decay[h] : 0.f;
-    f32x2 w[4];
-    if (CONST_DECAY) {
-#pragma unroll
-        for (int i = 0; i < 4; ++i) w[i] = pair(lam, lam);
-    }
-    float* out = nullptr;   // this lane's columns of a token's output
-    bool out_ok[2] = {false, false};
-    if constexpr (OUT) {
-        const int j0 = KG == 4 ? (lane & 1) * 4 + ((lane >> 1) & 1) * 2 : (lane & 1) * 4 + ((lane >> 1) & 1) * 2 + ((lane >> 2) & 1);
-        const int c = c_a + (j0 >> 2) * 4 * S_::VG + (j0 & 3);
-        const bool writes = KG <= 8 || (lane & (KG - 1) & ~7) == 0;
-        out = a.out + static_cast<size_t>(begin) * a.ld_out + h * a.vdim + v0 + c;
-        out_ok[0] = writes && c < vcols;
-        out_ok[1] = KG == 4 && writes && c + 1 < vcols;
-    }
+    const f32x2 lam2 = pair(lam, lam);
+    const int col = c_a + fold_column<KG>(lane);   // what this lane stores of a token's output
+    const bool ok = OUT && (KG <= 4 || (kg & ~3) == 0) && col < vcols, ok2 = KG == 2 && ok && col + 1 < vcols;
+    float* out = OUT ? a.out + static_cast<size_t>(begin) * a.ld_out + h * a.vdim + v0 + col : nullptr;
     int batch = 0;
     for (int row0 = begin; row0 < end; row0 += TT, ++batch) {
         const int n = min(TT, end - row0);
@@ -226,8 +227,12 @@ scan_kernel(const ScanParams p) {
         __syncthreads();   // this batch's raw rows are here, the last batch has been walked over
         if (row0 + TT < end) fetch(batch + 1, row0 + TT);
         const T* src = raw + (batch & 1) * raw_batch;
-        if (OUT) convert_rows<T>(sr, src, KP, a.dim, n, a.silu);
-        convert_rows<T>(sk, src + (OUT ? TT * KP : 0), KP, a.dim, n, a.silu);
+        if (OUT && !CONST_DECAY) {
+            convert_keys<T, KP>(sr, sk, src, src + TT * KP, sd, own, a.dim);
+        } else {
+            if (OUT) convert_rows<T>(sr, src, KP, a.dim, n, a.silu);
+            convert_rows<T>(sk, src + (OUT ? TT * KP : 0), KP, a.dim, n, a.silu);
+        }
         convert_rows<T>(sv, src + (OUT ? 2 : 1) * TT * KP, VB, vcols, n, a.silu);
         __syncthreads();
         const float* swb = sw + (batch & 1) * TT * KP;
@@ -240,93 +245,82 @@ scan_kernel(const ScanParams p) {
                     d *= CONST_DECAY ? lam : swb[t * KP + c];
                 }
                 sd[c] = d;
+                stot[c] *= d;
             }
             __syncthreads();
-            f32x2 d[4];
-            lds_pairs<KG>(sd + kg * 4, d);
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                total[i] = mul2(total[i], d[i]);
+            for (int i = 0; i < 8; i += 2) {
+                const ulonglong2 d = *reinterpret_cast<const ulonglong2*>(sd + k_of(i));
 #pragma unroll
-                for (int j = 0; j < 8; ++j) S[i][j] = mul2(S[i][j], d[i]);
+                for (int j = 0; j < 4; ++j) {
+                    S[i][j] = mul2(S[i][j], d.x);
+                    S[i + 1][j] = mul2(S[i + 1][j], d.y);
+                }
             }
         }
         for (int t = 0; t < n; ++t) {
-            f32x2 r[4], k[4];
-            float v[8], o[8];
-            lds_pairs<KG>(sk + t * KP + kg * 4, k);
-            if (OUT) lds_pairs<KG>(sr + t * KP + kg * 4, r);
-            if (OUT && !CONST_DECAY) lds_pairs<KG>(swb + t * KP + kg * 4, w);
-            {
-                const float4 x = *reinterpret_cast<const float4*>(sv + t * VB + c_a),
-                             y = *reinterpret_cast<const float4*>(sv + t * VB + c_a + 4 * S_::VG);
-                v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
-                v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
-            }
-            if constexpr (!OUT) {
+            const float4 v = *reinterpret_cast<const float4*>(sv + t * VB + c_a);
+            const f32x2 vv[4] = {pair(v.x, v.x), pair(v.y, v.y), pair(v.z, v.z), pair(v.w, v.w)};
+            f32x2 o[4] = {0, 0, 0, 0};
 #pragma unroll
-                for (int j = 0; j < 8; ++j) {
-                    const f32x2 vv = pair(v[j], v[j]);
+            for (int i = 0; i < 8; i += 2) {
+                const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(sk + t * KP + k_of(i));
+                if constexpr (!OUT) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) S[i][j] = fma2(k[i], vv, S[i][j]);
+                    for (int j = 0; j < 4; ++j) {
+                        S[i][j] = fma2(k.x, vv[j], S[i][j]);
+                        S[i + 1][j] = fma2(k.y, vv[j], S[i + 1][j]);
+                    }
+                } else {
+                    const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(sr + t * KP + k_of(i));
+                    ulonglong2 w = make_ulonglong2(lam2, lam2);
+                    if (!CONST_DECAY) w = *reinterpret_cast<const ulonglong2*>(swb + t * KP + k_of(i));
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        if (!CONST_DECAY) {
+                            o[j] = fma2(r.x, S[i][j], o[j]);
+                            o[j] = fma2(r.y, S[i + 1][j], o[j]);
+                        }
+                        S[i][j] = fma2(w.x, S[i][j], mul2(k.x, vv[j]));
+                        S[i + 1][j] = fma2(w.y, S[i + 1][j], mul2(k.y, vv[j]));
+                        if (CONST_DECAY) {
+                            o[j] = fma2(r.x, S[i][j], o[j]);
+                            o[j] = fma2(r.y, S[i + 1][j], o[j]);
+                        }
+                    }
                 }
-                continue;
             }
-            float own = 0.f;   // this lane's share of r . (u k)
-            if (!CONST_DECAY) {
-                f32x2 b = mul2(mul2(r[0], bonus[0]), k[0]);
+            if constexpr (OUT) {
+                float f[4];
 #pragma unroll
-                for (int i = 1; i < 4; ++i) b = fma2(mul2(r[i], bonus[i]), k[i], b);
-                const float2 f = unpair(b);
-                own = f.x + f.y;
-            }
-#pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                const f32x2 vv = pair(v[j], v[j]);
-                f32x2 acc;
+                for (int j = 0; j < 4; ++j) {
+                    const float2 q = unpair(o[j]);
+                    f[j] = q.x + q.y;
+                }
+                fold<KG>(f, lane);
                 if (!CONST_DECAY) {
-                    acc = mul2(r[0], S[0][j]);
-#pragma unroll
-                    for (int i = 1; i < 4; ++i) acc = fma2(r[i], S[i][j], acc);
+                    const float b = own[t];
+                    f[0] = fmaf(b, sv[t * VB + col], f[0]);
+                    if (KG == 2) f[1] = fmaf(b, sv[t * VB + col + 1], f[1]);
                 }
-#pragma unroll
-                for (int i = 0; i < 4; ++i) S[i][j] = fma2(w[i], S[i][j], mul2(k[i], vv));
-                if (CONST_DECAY) {
-                    acc = mul2(r[0], S[0][j]);
-#pragma unroll
-                    for (int i = 1; i < 4; ++i) acc = fma2(r[i], S[i][j], acc);
-                }
-                const float2 f = unpair(acc);
-                o[j] = CONST_DECAY ? f.x + f.y : fmaf(own, v[j], f.x + f.y);
+                if (ok) out[0] = f[0];
+                if (ok2) out[1] = f[1];
+                out += a.ld_out;
             }
-            fold<KG>(o, lane);
-            if (out_ok[0]) out[0] = o[0];
-            if (out_ok[1]) out[1] = o[1];
-            out += a.ld_out;
         }
     }
     if (!OUT || !chunked) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            float2 f[8];
-#pragma unroll
-            for (int j = 0; j < 8; ++j) f[j] = unpair(S[i][j]);
-            float* q = state + static_cast<size_t>(k_of(2 * i)) * p.vp;
+        for (int i = 0; i < 8; ++i) {
+            const float2 f[4] = {unpair(S[i][0]), unpair(S[i][1]), unpair(S[i][2]), unpair(S[i][3])};
+            float* q = state + static_cast<size_t>(k_of(i)) * p.vp;
             *reinterpret_cast<float4*>(q) = make_float4(f[0].x, f[1].x, f[2].x, f[3].x);
-            *reinterpret_cast<float4*>(q + 4 * S_::VG) = make_float4(f[4].x, f[5].x, f[6].x, f[7].x);
-            q += p.vp;   // the next row
-            *reinterpret_cast<float4*>(q) = make_float4(f[0].y, f[1].y, f[2].y, f[3].y);
-            *reinterpret_cast<float4*>(q + 4 * S_::VG) = make_float4(f[4].y, f[5].y, f[6].y, f[7].y);
+            *reinterpret_cast<float4*>(q + p.vp) = make_float4(f[0].y, f[1].y, f[2].y, f[3].y);
         }
     }
-    if (!OUT && blockIdx.y == 0 && warp == 0 && vg == 0) {
+    if (!OUT && blockIdx.y == 0) {   // every thread wrote the channels it reads here
         float* d = p.chunk_decay + (static_cast<size_t>(blockIdx.z) * a.heads + h) * KP;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const float2 f = unpair(total[i]);
-            d[k_of(2 * i)] = f.x;
-            d[k_of(2 * i + 1)] = f.y;
-        }
+        for (int c = threadIdx.x; c < KP; c += blockDim.x) d[c] = stot[c];
     }
 }
 
@@ -633,10 +627,10 @@ void launch_scan(const ScanArgs& a, cudaStream_t s) {
         else run_scan<T, KG, false>(p, g, s);
     };
     switch (g.kg) {
+        case 2: run(std::integral_constant<int, 2>()); break;
         case 4: run(std::integral_constant<int, 4>()); break;
         case 8: run(std::integral_constant<int, 8>()); break;
-        case 16: run(std::integral_constant<int, 16>()); break;
-        default: run(std::integral_constant<int, 32>()); break;
+        default: run(std::integral_constant<int, 16>()); break;
     }
 }
 bool scan_step_fits(int dim, int vdim, bool time_mix) {
