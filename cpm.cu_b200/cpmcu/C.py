@@ -70,6 +70,13 @@ _SIGNATURES = {
     "cpmcu_layer_attention": (_c_int, [_c_void_p] * 4 + [_c_int] * 5 + [_c_void_p]),
     "cpmcu_layer_qkv_norm_append": (_c_int, [_c_void_p] * 4 + [_c_float, _c_void_p] + [_c_int] * 4 + [_c_void_p] * 3),
     "cpmcu_layer_scan": (_c_int, [_c_void_p] * 8 + [_c_int] * 3 + [_c_void_p]),
+    "cpmcu_layer_scan_step": (_c_int, [_c_void_p] * 12 + [_c_float] + [_c_int] * 2 + [_c_void_p]),
+    "cpmcu_layer_decay": (_c_int, [_c_void_p] * 3 + [_c_int] * 4 + [_c_void_p]),
+    "cpmcu_layer_norm_gate": (_c_int, [_c_void_p] * 3 + [_c_int] * 3 + [_c_float] * 2 + [_c_int] * 2 + [_c_void_p]),
+    "cpmcu_layer_tanh_norm": (_c_int, [_c_void_p] * 3 + [_c_float] + [_c_void_p] * 2 + [_c_int] * 4 + [_c_void_p] * 2),
+    "cpmcu_layer_clamped_gate": (_c_int, [_c_void_p] + [_c_int] * 2 + [_c_float] * 2 + [_c_int, _c_void_p]),
+    "cpmcu_layer_side_step": (_c_int, [_c_void_p] * 4 + [_c_float] + [_c_void_p] * 5 + [_c_int] * 6 + [_c_float, _c_int]),
+    "cpmcu_grouped_linear": (_c_int, [_c_void_p] * 2 + [_c_int] * 6 + [_c_void_p]),
     "cpmcu_layer_scan_state_floats": (ctypes.c_long, [_c_void_p]),
     "cpmcu_layer_out_norm": (_c_int, [_c_void_p] * 3 + [_c_float, _c_void_p] + [_c_int] * 3 + [_c_float, _c_int]),
     "cpmcu_moe_route": (_c_int, [_c_void_p] * 4 + [_c_int] * 2 + [_c_void_p] * 2),

@@ -829,6 +829,131 @@ int cpmcu_layer_scan(const cpmcu_layer_spec* spec, const void* r, const void* k,
     });
 }
 
+int cpmcu_layer_scan_step(const cpmcu_layer_spec* spec, const void* r, const void* k, const void* v, const void* inner, const void* w2,
+                          const void* w0, const float* decay, const void* bonus, float* state, const void* norm, const void* gate, float eps,
+                          int position, int fp32, void* out) {
+    return guarded([&] {
+        const LayerSpec sp = to_spec(*spec);
+        CPM_REQUIRE(sp.rec != REC_NONE && scan_step_fits(sp.rec_dim, sp.rec_vdim, sp.rec == REC_TIME_MIX), "layer_scan_step: bad sizes");
+        cudaStream_t s = runtime().stream;
+        DeviceBuf len(4), o(static_cast<size_t>(sp.rec_heads) * sp.rec_vdim * 4), ticket(4);
+        CUDA_CHECK(cudaMemcpyAsync(len.p, &position, 4, cudaMemcpyHostToDevice, s));
+        CUDA_CHECK(cudaMemsetAsync(ticket.p, 0, 4, s));
+        ScanStepArgs a;
+        a.scan.r = r; a.scan.k = k; a.scan.v = v;
+        a.scan.heads = sp.rec_heads; a.scan.dim = sp.rec_dim; a.scan.vdim = sp.rec_vdim; a.scan.rows = 1;
+        a.scan.silu = sp.rec == REC_LIGHTNING;
+        a.scan.decay = decay; a.scan.bonus = static_cast<const bf16*>(bonus);
+        a.scan.state = state; a.scan.out = static_cast<float*>(o.p);
+        a.scan.kv_len = static_cast<const int32_t*>(len.p);
+        a.inner = inner; a.w2 = static_cast<const bf16*>(w2); a.w0 = static_cast<const bf16*>(w0); a.rank = sp.rec_rank;
+        a.norm = static_cast<const bf16*>(norm); a.gate = gate; a.eps = eps; a.scale = sp.rec_scale;
+        a.out = out; a.ticket = static_cast<int32_t*>(ticket.p);
+        if (fp32) launch_scan_step<float>(a, s);
+        else launch_scan_step<bf16>(a, s);
+        sync_and_check("layer_scan_step");
+        return 0;
+    });
+}
+
+int cpmcu_layer_decay(const void* x, const void* w2, const void* w0, int rank, int channels, int rows, int fp32, float* out) {
+    return guarded([&] {
+        cudaStream_t s = runtime().stream;
+        const bf16 *a = static_cast<const bf16*>(w2), *b = static_cast<const bf16*>(w0);
+        if (fp32) launch_decay<float>(static_cast<const float*>(x), rank, a, b, rank, channels, out, channels, rows, s);
+        else launch_decay<bf16>(static_cast<const bf16*>(x), rank, a, b, rank, channels, out, channels, rows, s);
+        sync_and_check("layer_decay");
+        return 0;
+    });
+}
+
+int cpmcu_layer_norm_gate(const float* o, const void* w, const void* gate, int groups, int group, int silu, float eps, float scale, int rows,
+                          int fp32, void* out) {
+    return guarded([&] {
+        cudaStream_t s = runtime().stream;
+        const int n = groups * group;
+        const bf16* wb = static_cast<const bf16*>(w);
+        if (fp32) launch_norm_gate<float>(o, n, groups, group, wb, static_cast<const float*>(gate), n, silu != 0, eps, scale, static_cast<float*>(out), n, rows, s);
+        else launch_norm_gate<bf16>(o, n, groups, group, wb, static_cast<const bf16*>(gate), n, silu != 0, eps, scale, static_cast<bf16*>(out), n, rows, s);
+        sync_and_check("layer_norm_gate");
+        return 0;
+    });
+}
+
+int cpmcu_layer_tanh_norm(const float* x32, const void* w, const void* b, float alpha, const void* mu, float* prev, int rows, int ld, int position,
+                          int fp32, void* h, void* mixes) {
+    return guarded([&] {
+        cudaStream_t s = runtime().stream;
+        DeviceBuf len(4);
+        CUDA_CHECK(cudaMemcpyAsync(len.p, &position, 4, cudaMemcpyHostToDevice, s));
+        DynTanh n;
+        n.w = static_cast<const bf16*>(w); n.b = static_cast<const bf16*>(b); n.alpha = alpha;
+        TokenShift t;
+        if (mu != nullptr) {
+            t.mu = static_cast<const bf16*>(mu); t.out = mixes; t.stride = static_cast<size_t>(rows) * ld; t.prev = prev;
+            t.kv_len = static_cast<const int32_t*>(len.p);
+        }
+        if (fp32) launch_tanh_norm<float>(x32, nullptr, n, static_cast<float*>(h), t, rows, ld, s);
+        else launch_tanh_norm<bf16>(x32, nullptr, n, static_cast<bf16*>(h), t, rows, ld, s);
+        sync_and_check("layer_tanh_norm");
+        return 0;
+    });
+}
+
+int cpmcu_layer_clamped_gate(const void* gu, int rows, int ff, float limit, float alpha, int fp32, void* act) {
+    return guarded([&] {
+        cudaStream_t s = runtime().stream;
+        if (fp32) launch_clamped_gate<float>(static_cast<const float*>(gu), 2 * ff, static_cast<float*>(act), ff, rows, ff, limit, alpha, false, s);
+        else launch_clamped_gate<bf16>(static_cast<const bf16*>(gu), 2 * ff, static_cast<bf16*>(act), ff, rows, ff, limit, alpha, false, s);
+        sync_and_check("layer_clamped_gate");
+        return 0;
+    });
+}
+
+int cpmcu_layer_side_step(float* x32, const void* delta, const void* w, const void* b, float alpha, const void* gate, const void* proj,
+                          const void* norm, const int32_t* id, const void* table, int layers, int layer, int dim, int vocab, int width, int ld,
+                          float eps, int fp32) {
+    return guarded([&] {
+        cudaStream_t s = runtime().stream;
+        const int dp = pad64(dim);
+        DeviceBuf g(linear_weight_elems(dim, ld) * 2), p(linear_weight_elems(width, dp) * 2);
+        CUDA_CHECK(cudaMemsetAsync(g.p, 0, linear_weight_elems(dim, ld) * 2, s));
+        CUDA_CHECK(cudaMemsetAsync(p.p, 0, linear_weight_elems(width, dp) * 2, s));
+        if (fp32) {
+            CUDA_CHECK(cudaMemcpy2DAsync(g.p, static_cast<size_t>(ld) * 2, gate, static_cast<size_t>(width) * 2, static_cast<size_t>(width) * 2, dim, cudaMemcpyDefault, s));
+            CUDA_CHECK(cudaMemcpy2DAsync(p.p, static_cast<size_t>(dp) * 2, proj, static_cast<size_t>(dim) * 2, static_cast<size_t>(dim) * 2, width, cudaMemcpyDefault, s));
+        } else {
+            retile_weight_rows(gate, dim, width, static_cast<bf16*>(g.p), ld, 0, 0, 0, s);
+            retile_weight_rows(proj, width, dim, static_cast<bf16*>(p.p), dp, 0, 0, 0, s);
+        }
+        SideStepArgs a;
+        a.x32 = x32; a.delta = delta;
+        a.post.w = static_cast<const bf16*>(w); a.post.b = static_cast<const bf16*>(b); a.post.alpha = alpha;
+        a.gate = static_cast<const bf16*>(g.p); a.proj = static_cast<const bf16*>(p.p); a.norm = static_cast<const bf16*>(norm);
+        a.ids = id; a.table = static_cast<const bf16*>(table); a.table_ld = layers * dim; a.col0 = layer * dim; a.dim = dim; a.vocab = vocab;
+        a.width = width; a.ld = ld; a.eps = eps;
+        if (fp32) launch_side_step<float>(a, s);
+        else launch_side_step<bf16>(a, s);
+        sync_and_check("layer_side_step");
+        return 0;
+    });
+}
+
+int cpmcu_grouped_linear(const void* x, const void* w, int n, int N, int N_s, int K, int rows, int ldy, void* y) {
+    return guarded([&] {
+        cudaStream_t s = runtime().stream;
+        const size_t one = linear_weight_elems(N, K), all = n * one + (N_s > 0 ? linear_weight_elems(N_s, K) : 0);
+        DeviceBuf t(all * 2);
+        CUDA_CHECK(cudaMemsetAsync(t.p, 0, all * 2, s));
+        const bf16* src = static_cast<const bf16*>(w);
+        for (int i = 0; i < n; ++i) retile_weight_rows(src + static_cast<size_t>(i) * N * K, N, K, static_cast<bf16*>(t.p) + i * one, K, 0, 0, 0, s);
+        if (N_s > 0) retile_weight_rows(src + static_cast<size_t>(n) * N * K, N_s, K, static_cast<bf16*>(t.p) + n * one, K, 0, 0, 0, s);
+        launch_moe_gemm(make_grouped_plan(static_cast<const bf16*>(t.p), n, N, N_s, K, static_cast<const bf16*>(x), static_cast<bf16*>(y), ldy, rows), s);
+        sync_and_check("grouped_linear");
+        return 0;
+    });
+}
+
 long cpmcu_layer_scan_state_floats(const cpmcu_layer_spec* spec) {
     const LayerSpec sp = to_spec(*spec);
     return static_cast<long>(scan_state_floats(sp.rec_heads, sp.rec_dim, sp.rec_vdim));

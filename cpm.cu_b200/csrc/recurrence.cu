@@ -574,10 +574,10 @@ void run_scan(const ScanParams& base, const Geometry& g, cudaStream_t s) {
     }
     const dim3 block(g.warps * 32);
     if (a.rows > kMinChunk) {
-        // the shortest chunks whose CTAs all run at once (128 registers: 16 warps per SM), up to four times the shortest
+        // the shortest chunks whose CTAs all run at once (128 registers: 16 warps per SM)
         const long long slots = static_cast<long long>(runtime().num_sms) * (16 / g.warps);
         p.chunk = kMinChunk;
-        while (p.chunk < 4 * kMinChunk && static_cast<long long>(a.heads) * g.vblocks * ceil_div(a.rows, p.chunk) > slots) p.chunk *= 2;
+        while (p.chunk < 8 * kMinChunk && static_cast<long long>(a.heads) * g.vblocks * ceil_div(a.rows, p.chunk) > slots) p.chunk += TT;
         p.chunks = ceil_div(a.rows, p.chunk);
         launch_kernel(scan_kernel<T, KG, CONST_DECAY, false>, dim3(a.heads, g.vblocks, p.chunks), block, M::bytes(vb, false), s, p);
         const size_t n4 = static_cast<size_t>(a.heads) * g.kp * g.vp / 4;

@@ -333,6 +333,29 @@ int cpmcu_layer_qkv_norm_append(const cpmcu_layer_spec* spec, const void* qkv, c
 int cpmcu_layer_scan(const cpmcu_layer_spec* spec, const void* r, const void* k, const void* v, const float* w, const float* decay,
                      const void* bonus, float* state, int rows, int position, int fp32, float* out);
 long cpmcu_layer_scan_state_floats(const cpmcu_layer_spec* spec);
+/* One token's recurrence with what is around it: time mix: decays from inner [rec_rank] as cpmcu_layer_decay; then the norm and
+ * gate of cpmcu_layer_norm_gate (time mix: per head, silu; lightning: over all heads, sigmoid), factor rec_scale.  out [heads * vdim]. */
+int cpmcu_layer_scan_step(const cpmcu_layer_spec* spec, const void* r, const void* k, const void* v, const void* inner, const void* w2,
+                          const void* w0, const float* decay, const void* bonus, float* state, const void* norm, const void* gate, float eps,
+                          int position, int fp32, void* out);
+/* out[row][c] = exp(-exp(w2[c] . tanh(x[row]) + w0[c])), fp32; x [rows, rank], w2 [channels, rank]. */
+int cpmcu_layer_decay(const void* x, const void* w2, const void* w0, int rank, int channels, int rows, int fp32, float* out);
+/* out = o / rms(o over each group) * w * (silu(gate) or sigmoid(gate)) * scale; o [rows, groups * group] fp32. */
+int cpmcu_layer_norm_gate(const float* o, const void* w, const void* gate, int groups, int group, int silu, float eps, float scale, int rows,
+                          int fp32, void* out);
+/* h = tanh(alpha * x32) * w + b; with mu [5, ld] also mixes [5, rows, ld]: h + (h of the row before - h) * mu, the row before the
+ * first one being prev [ld] (zero at position 0), which the last row replaces. */
+int cpmcu_layer_tanh_norm(const float* x32, const void* w, const void* b, float alpha, const void* mu, float* prev, int rows, int ld, int position,
+                          int fp32, void* h, void* mixes);
+/* act = g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up cut to [-limit, limit]; gu [rows, gate | up], ff % 64 == 0. */
+int cpmcu_layer_clamped_gate(const void* gu, int rows, int ff, float limit, float alpha, int fp32, void* act);
+/* One row: x32 += tanh(alpha * delta) * w + b, then x32 += rms(proj (gelu_tanh(gate x32) * table[id][layer * dim ..])) * norm.
+ * gate [dim, width], proj [width, dim], table [vocab, layers * dim]. */
+int cpmcu_layer_side_step(float* x32, const void* delta, const void* w, const void* b, float alpha, const void* gate, const void* proj,
+                          const void* norm, const int32_t* id, const void* table, int layers, int layer, int dim, int vocab, int width, int ld,
+                          float eps, int fp32);
+/* n products in one launch: y[i * rows ..] = x[i * rows ..] w_i^T with w [n, N, K], and with N_s > 0 one more of N_s outputs. */
+int cpmcu_grouped_linear(const void* x, const void* w, int n, int N, int N_s, int K, int rows, int ldy, void* y);
 /* x32 += mult * rms(delta) * (1 + w); xh = x32 in the activation dtype. */
 int cpmcu_layer_out_norm(float* x32, void* xh, const void* delta, float mult, const void* w, int rows, int width, int ld,
                          float eps, int fp32);

@@ -193,3 +193,47 @@ def greedy(config, weights, prompt, n):
         out.append(int(forward(config, weights, tokens, seq)[-1].argmax()))
         tokens = out[-1:]
     return out
+
+
+# ---------------------------------------------------------------- models for tests
+def random_weights(config, seed=0, dtype=torch.float64):
+    """Seeded weights of every tensor the configuration needs, rounded to bfloat16 values.  The inner width of a decay differs
+    from layer to layer; decays reach from almost nothing kept to almost everything."""
+    g = torch.Generator().manual_seed(seed)
+    W, V, side, scale = config["width"], config["vocab"], config["token_side"]["dim"], config["embedding"]["scale"]
+
+    def mat(*shape, std=None, mean=0.0):
+        return (torch.randn(*shape, generator=g) * (std if std is not None else shape[-1] ** -0.5) + mean).to(torch.bfloat16)
+
+    w = {"embed": mat(V, W, std=1 / scale), "side.embed": mat(V, len(config["layers"]) * side, std=1.0)}
+
+    def add_norm(name):
+        w[name], w[name + ".b"] = mat(W, std=0.3, mean=1.0), mat(W, std=0.2)
+        w[name + ".alpha"] = mat(1, std=0.1, mean=0.6)[0]
+
+    add_norm("final.norm")
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}", layer["mixer"]
+        for name in ("norm1", "norm1b") + (("norm2", "norm2b") if layer.get("mlp") else ()):
+            add_norm(f"{p}.{name}")
+        if layer["type"] == "lightning":
+            nk, nv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            for name, rows in (("q", nk), ("k", nk), ("v", nv), ("g", nv)):
+                w[f"{p}.mix.{name}"] = mat(rows, W)
+            w[p + ".mix.o"], w[p + ".mix.norm"] = mat(W, nv), mat(nv, std=0.2, mean=1.0)
+        else:
+            a, r, q = m["left"], m["right"], p + ".mix.left"
+            w[q + ".q"], w[q + ".k"] = mat(a["heads"] * a["dim"], W), mat(a["kv_heads"] * a["dim"], W)
+            w[q + ".v"], w[q + ".o"] = mat(a["kv_heads"] * a["vdim"], W), mat(W, a["heads"] * a["vdim"])
+            q, n, rank = p + ".mix.right", r["heads"] * r["dim"], 5 + 3 * i
+            for s in "rkvg":
+                w[f"{q}.{s}"] = mat(n, W)
+            for s in "rkvgw":
+                w[f"{q}.mu.{s}"] = mat(W, std=0.3, mean=0.5)
+            w[q + ".w1"], w[q + ".w2"], w[q + ".w0"] = mat(rank, W), mat(n, rank, std=0.4), mat(n, std=2.0, mean=-2.0)
+            w[q + ".u"], w[q + ".norm"], w[q + ".o"] = mat(r["heads"], r["dim"], std=0.5), mat(n, std=0.2, mean=1.0), mat(W, n)
+        if layer.get("mlp"):
+            ff = layer["mlp"]["ff"]
+            w[p + ".mlp.gate"], w[p + ".mlp.up"], w[p + ".mlp.down"] = mat(ff, W), mat(ff, W), mat(W, ff)
+        w[p + ".side.gate"], w[p + ".side.proj"], w[p + ".side.norm"] = mat(side, W), mat(W, side), mat(W, std=0.2, mean=0.3)
+    return {k: v.to(dtype) for k, v in w.items()}
