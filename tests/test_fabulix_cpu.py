@@ -75,6 +75,25 @@ def test_portions_equal_the_whole(name):
     assert whole.std() > 0.05 and (whole[5] - whole[40]).abs().max() > 0.1
 
 
+def logit_errors(got, ref):
+    d = got - ref
+    return (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / ref.std()
+
+
+def test_side_by_side_scales_and_the_far_past_show():
+    """A wrong factor of either half, a lost state or a lost key changes the logits by far more than the tests let pass."""
+    cfg = case("mixed")
+    w = F.random_weights(cfg, seed=7)
+    toks = tokens_of(cfg, 200, seed=2)
+    ref = F.forward(cfg, w, toks)[-1:]
+    for where, key in ((1, "left_scale"), (1, "right_scale"), (3, "left_scale"), (3, "right_scale")):
+        bad = case("mixed")
+        bad["layers"][where]["mixer"][key] *= 0.8
+        assert logit_errors(F.forward(bad, w, toks)[-1:], ref).max() > 3e-3
+    for changed in (0, 100, 190):
+        assert logit_errors(F.forward(cfg, w, toks[:changed] + [(toks[changed] + 1) % 333] + toks[changed + 1:])[-1:], ref).max() > 1e-3
+
+
 def test_first_token_has_nothing_before_it():
     cfg = case("odd")
     w = F.random_weights(cfg, seed=2)
