@@ -84,7 +84,7 @@ def test_side_by_side_scales_and_the_far_past_show():
     """A wrong factor of either half, a lost state or a lost key changes the logits by far more than the tests let pass."""
     cfg = case("mixed")
     w = F.random_weights(cfg, seed=7)
-    toks = tokens_of(cfg, 200, seed=2)
+    toks = torch.randint(0, cfg["vocab"], (200,), generator=torch.Generator().manual_seed(2)).tolist()
     ref = F.forward(cfg, w, toks)[-1:]
     for where, key in ((1, "left_scale"), (1, "right_scale"), (3, "left_scale"), (3, "right_scale")):
         bad = case("mixed")
