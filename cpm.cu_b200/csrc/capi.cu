@@ -836,7 +836,9 @@ int cpmcu_layer_scan_step(const cpmcu_layer_spec* spec, const void* r, const voi
         const LayerSpec sp = to_spec(*spec);
         CPM_REQUIRE(sp.rec != REC_NONE && scan_step_fits(sp.rec_dim, sp.rec_vdim, sp.rec == REC_TIME_MIX), "layer_scan_step: bad sizes");
         cudaStream_t s = runtime().stream;
-        DeviceBuf len(4), o(static_cast<size_t>(sp.rec_heads) * sp.rec_vdim * 4), ticket(4);
+        const int channels = sp.rec_heads * sp.rec_dim;
+        DeviceBuf len(4), o(static_cast<size_t>(sp.rec_heads) * sp.rec_vdim * 4), ticket(4), w2t(static_cast<size_t>(channels) * sp.rec_rank * 2);
+        if (sp.rec == REC_TIME_MIX) upload_transposed(w2, channels, sp.rec_rank, static_cast<bf16*>(w2t.p), s);
         CUDA_CHECK(cudaMemcpyAsync(len.p, &position, 4, cudaMemcpyHostToDevice, s));
         CUDA_CHECK(cudaMemsetAsync(ticket.p, 0, 4, s));
         ScanStepArgs a;
@@ -846,7 +848,7 @@ int cpmcu_layer_scan_step(const cpmcu_layer_spec* spec, const void* r, const voi
         a.scan.decay = decay; a.scan.bonus = static_cast<const bf16*>(bonus);
         a.scan.state = state; a.scan.out = static_cast<float*>(o.p);
         a.scan.kv_len = static_cast<const int32_t*>(len.p);
-        a.inner = inner; a.w2 = static_cast<const bf16*>(w2); a.w0 = static_cast<const bf16*>(w0); a.rank = sp.rec_rank;
+        a.inner = inner; a.w2 = static_cast<const bf16*>(w2t.p); a.w0 = static_cast<const bf16*>(w0); a.rank = sp.rec_rank;
         a.norm = static_cast<const bf16*>(norm); a.gate = gate; a.eps = eps; a.scale = sp.rec_scale;
         a.out = out; a.ticket = static_cast<int32_t*>(ticket.p);
         if (fp32) launch_scan_step<float>(a, s);
@@ -859,7 +861,9 @@ int cpmcu_layer_scan_step(const cpmcu_layer_spec* spec, const void* r, const voi
 int cpmcu_layer_decay(const void* x, const void* w2, const void* w0, int rank, int channels, int rows, int fp32, float* out) {
     return guarded([&] {
         cudaStream_t s = runtime().stream;
-        const bf16 *a = static_cast<const bf16*>(w2), *b = static_cast<const bf16*>(w0);
+        DeviceBuf w2t(static_cast<size_t>(channels) * rank * 2);
+        upload_transposed(w2, channels, rank, static_cast<bf16*>(w2t.p), s);
+        const bf16 *a = static_cast<const bf16*>(w2t.p), *b = static_cast<const bf16*>(w0);
         if (fp32) launch_decay<float>(static_cast<const float*>(x), rank, a, b, rank, channels, out, channels, rows, s);
         else launch_decay<bf16>(static_cast<const bf16*>(x), rank, a, b, rank, channels, out, channels, rows, s);
         sync_and_check("layer_decay");

@@ -80,7 +80,7 @@ struct LayeredWeights {
     // matrix with rows q | k | v | g
     bf16* rec_proj = nullptr;
     size_t rec_part = 0;
-    bf16* w2 = nullptr;                         // [rec_heads * rec_dim][rec_rank], row-major
+    bf16* w2 = nullptr;                         // [rec_rank][rec_heads * rec_dim]
     bf16 *w0 = nullptr, *bonus = nullptr, *rec_norm = nullptr;
     bf16* mu = nullptr;                         // [kMixes][ld]
     float* decay = nullptr;                     // [rec_heads]

@@ -370,7 +370,7 @@ void Engine::load_layered(const std::string& name, const void* src) {
                 else throw std::invalid_argument("Unsupported name " + name);
             } else if (m == "w0") plain(w.w0, 1, ck, ck);
             else if (m == "w1") matrix(w.rec_proj + 4 * w.rec_part, s.rec_rank, W, L, 0, 0, 0);
-            else if (m == "w2") plain(w.w2, ck, s.rec_rank, s.rec_rank);
+            else if (m == "w2") upload_transposed(src, ck, s.rec_rank, w.w2, st);
             else if (m == "u") plain(w.bonus, 1, ck, ck);
             else {
                 const bool mu = m.rfind("mu.", 0) == 0;

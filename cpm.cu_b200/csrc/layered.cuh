@@ -154,8 +154,10 @@ struct SideStepArgs {
 };
 template <typename T>
 void launch_side_step(const SideStepArgs& a, cudaStream_t s);
-// Decays of a time-mix layer: out[r][c] = exp(-exp(w2[c] . tanh(x[r]) + w0[c])), c < channels; x: `rank` columns of T, w2
-// [channels][rank]
+// dst [cols][rows] = src [rows][cols], host or device memory
+void upload_transposed(const void* src, int rows, int cols, bf16* dst, cudaStream_t s);
+// Decays of a time-mix layer: out[r][c] = exp(-exp(sum_k w2[k][c] tanh(x[r][k]) + w0[c])), c < channels; x: `rank` columns of
+// T, w2 [rank][channels] (upload_transposed)
 template <typename T>
 void launch_decay(const T* x, int ld_x, const bf16* w2, const bf16* w0, int rank, int channels, float* out, int ld_out, int rows, cudaStream_t s);
 // out[r][c] = rms over each group of `group` columns of o[r] * w[c] * gate(g[r][c]) * scale; gate: silu, or sigmoid

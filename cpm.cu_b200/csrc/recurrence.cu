@@ -11,6 +11,7 @@
 //
 // A single token takes scan_step_kernel, which streams the state and does what surrounds the recurrence as well.
 #include <algorithm>
+#include <vector>
 
 #include "row_ops.cuh"
 
@@ -396,8 +397,10 @@ scan_step_kernel(const StepParams p) {
         if (g < groups && i < p.kp) S[n] = *reinterpret_cast<const float4*>(state + static_cast<size_t>(i) * p.vp);
     }
     if (TIME_MIX) {
-        const bf16* w = p.a.w2 + static_cast<size_t>(h) * a.dim * p.a.rank;
-        for (int i = tid * 64; i < a.dim * p.a.rank; i += STEP_THREADS * 64) prefetch_l2(w + i);
+        const int per = (a.dim + 63) / 64;
+        for (int i = tid; i < p.a.rank * per; i += STEP_THREADS) {
+            prefetch_l2(p.a.w2 + static_cast<size_t>(i / per) * a.heads * a.dim + h * a.dim + i % per * 64);
+        }
         if (tid * 64 < a.dim) {
             prefetch_l2(p.a.w0 + h * a.dim + tid * 64);
             prefetch_l2(a.bonus + h * a.dim + tid * 64);
@@ -430,29 +433,21 @@ scan_step_kernel(const StepParams p) {
         if (tid < p.a.rank) inner[tid] = tanhf(x_t);
         for (int k = tid + STEP_THREADS; k < p.a.rank; k += STEP_THREADS) inner[k] = tanhf(to_float<T>(static_cast<const T*>(p.a.inner)[k]));
         __syncthreads();
-        constexpr int WARPS = STEP_THREADS / 32;
-        for (int c0 = warp; c0 < a.dim; c0 += WARPS * 8) {   // eight channels of a warp at once
-            float z[8];
-#pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                const int c = c0 + e * WARPS;
-                z[e] = lane == 0 && c < a.dim ? __bfloat162float(__ldg(p.a.w0 + h * a.dim + c)) : 0.f;
-            }
-            const bf16* w = p.a.w2 + (static_cast<size_t>(h) * a.dim + c0) * p.a.rank;
-            for (int k = lane; k < p.a.rank; k += 32) {
-                const float in = inner[k];
-#pragma unroll
-                for (int e = 0; e < 8; ++e) {
-                    if (c0 + e * WARPS < a.dim) z[e] = fmaf(__bfloat162float(__ldg(w + static_cast<size_t>(e) * WARPS * p.a.rank + k)), in, z[e]);
-                }
-            }
-#pragma unroll
-            for (int e = 0; e < 8; ++e) z[e] = warp_sum(z[e]);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                const int c = c0 + e * WARPS;
-                if (lane == e && c < a.dim) sw[c] = expf(-expf(z[e]));
-            }
+        // kp divides the threads: each channel's sum over the rank in parts
+        float* part = red + p.a.rank;     // [STEP_THREADS]
+        const int c = tid % p.kp, parts = STEP_THREADS / p.kp, channels = a.heads * a.dim;
+        float z = 0.f;
+        if (c < a.dim) {
+            const bf16* w = p.a.w2 + h * a.dim + c;
+#pragma unroll 16
+            for (int k = tid / p.kp; k < p.a.rank; k += parts) z = fmaf(__bfloat162float(__ldg(w + static_cast<size_t>(k) * channels)), inner[k], z);
+        }
+        part[tid] = z;
+        __syncthreads();
+        if (tid < a.dim) {
+            z = __bfloat162float(__ldg(p.a.w0 + h * a.dim + tid));
+            for (int n = 0; n < parts; ++n) z += part[n * p.kp + tid];
+            sw[tid] = expf(-expf(z));
         }
         if (tid >= a.dim && tid < p.kp) sw[tid] = 0.f;
         if (warp == 0) {
@@ -633,6 +628,18 @@ void launch_scan(const ScanArgs& a, cudaStream_t s) {
         default: run(std::integral_constant<int, 16>()); break;
     }
 }
+void upload_transposed(const void* src, int rows, int cols, bf16* dst, cudaStream_t s) {
+    const size_t n = static_cast<size_t>(rows) * cols;
+    std::vector<bf16> a(n), b(n);
+    CUDA_CHECK(cudaMemcpyAsync(a.data(), src, n * sizeof(bf16), cudaMemcpyDefault, s));
+    CUDA_CHECK(cudaStreamSynchronize(s));
+    for (int r = 0; r < rows; ++r) {
+        for (int c = 0; c < cols; ++c) b[static_cast<size_t>(c) * rows + r] = a[static_cast<size_t>(r) * cols + c];
+    }
+    CUDA_CHECK(cudaMemcpyAsync(dst, b.data(), n * sizeof(bf16), cudaMemcpyHostToDevice, s));
+    CUDA_CHECK(cudaStreamSynchronize(s));
+}
+
 bool scan_step_fits(int dim, int vdim, bool time_mix) {
     const Geometry g = geometry(dim, vdim);
     return !time_mix || static_cast<long long>(g.kp) * g.vp <= 4LL * STEP_LOADS * STEP_THREADS;
@@ -659,7 +666,7 @@ void launch_scan_step(const ScanStepArgs& a, cudaStream_t s) {
     const dim3 grid(sc.heads, ceil_div(sc.vdim, p.cols));
     const int groups = STEP_THREADS / (p.cols / 4);
     CPM_REQUIRE(groups >= 1 && groups * STEP_LOADS >= p.kp, "recurrence step: unsupported sizes");
-    const size_t smem = sizeof(float) * (3 * p.kp + p.cols + std::max(groups * p.cols, a.rank));
+    const size_t smem = sizeof(float) * (3 * p.kp + p.cols + std::max(groups * p.cols, a.rank + STEP_THREADS));
     if (time_mix) launch_kernel(scan_step_kernel<T, true>, grid, dim3(STEP_THREADS), smem, s, p);
     else launch_kernel(scan_step_kernel<T, false>, grid, dim3(STEP_THREADS), smem, s, p);
 }

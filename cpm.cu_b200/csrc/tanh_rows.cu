@@ -327,7 +327,7 @@ side_step_kernel(const SideStepArgs a) {
     store_vec<8>(a.shift.prev + mine, h);
 }
 
-// ROWS tokens x 256 channels per CTA, two channels per thread.
+// ROWS tokens x 256 channels per CTA, two neighbouring channels per thread.
 constexpr int DECAY_THREADS = 128;
 
 template <typename T, int ROWS>
@@ -336,23 +336,21 @@ decay_kernel(const T* __restrict__ x, int ld_x, const bf16* __restrict__ w2, con
              float* __restrict__ out, int ld_out, int rows) {
     extern __shared__ __align__(16) float inner[];   // [rank][ROWS]
     const int row0 = blockIdx.y * ROWS, n = min(ROWS, rows - row0);
+    const int c = (blockIdx.x * DECAY_THREADS + threadIdx.x) * 2;
+    const bool one = c < channels, two = c + 1 < channels;
+    const float b0 = one ? __bfloat162float(w0[c]) : 0.f, b1 = two ? __bfloat162float(w0[c + 1]) : 0.f;
     grid_dependency_sync();
     for (int i = threadIdx.x; i < ROWS * rank; i += DECAY_THREADS) {
         const int t = i / rank, k = i - t * rank;
         inner[k * ROWS + t] = t < n ? tanhf(to_float<T>(x[static_cast<size_t>(row0 + t) * ld_x + k])) : 0.f;
     }
     __syncthreads();
-    int c[2];
-    const bf16* w[2];
+    if (!one) return;
     f32x2 z[2][ROWS / 2];
 #pragma unroll
-    for (int m = 0; m < 2; ++m) {
-        c[m] = blockIdx.x * 2 * DECAY_THREADS + m * DECAY_THREADS + threadIdx.x;
-        const int at = min(c[m], channels - 1);
-        w[m] = w2 + static_cast<size_t>(at) * rank;
-        const float b = __bfloat162float(w0[at]);
-#pragma unroll
-        for (int t = 0; t < ROWS / 2; ++t) z[m][t] = pair(b, b);
+    for (int t = 0; t < ROWS / 2; ++t) {
+        z[0][t] = pair(b0, b0);
+        z[1][t] = pair(b1, b1);
     }
     auto add = [&](float a, float b, int k) {
         const f32x2 wa = pair(a, a), wb = pair(b, b);
@@ -365,25 +363,37 @@ decay_kernel(const T* __restrict__ x, int ld_x, const bf16* __restrict__ w2, con
             z[1][t + 1] = fma2(wb, v.y, z[1][t + 1]);
         }
     };
-    if (rank % 8 == 0) {
-        for (int k = 0; k < rank; k += 8) {
-            float f[2][8];
-            load_vec<8>(w[0] + k, f[0]);
-            load_vec<8>(w[1] + k, f[1]);
+    const bf16* w = w2 + c;
+    if (channels % 2 == 0) {
+        int k = 0;
+        for (; k + 8 <= rank; k += 8) {
+            __nv_bfloat162 f[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) add(f[0][e], f[1][e], k + e);
+            for (int e = 0; e < 8; ++e) f[e] = *reinterpret_cast<const __nv_bfloat162*>(w + static_cast<size_t>(k + e) * channels);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) add(__low2float(f[e]), __high2float(f[e]), k + e);
+        }
+        for (; k < rank; ++k) {
+            const __nv_bfloat162 f = *reinterpret_cast<const __nv_bfloat162*>(w + static_cast<size_t>(k) * channels);
+            add(__low2float(f), __high2float(f), k);
         }
     } else {
-        for (int k = 0; k < rank; ++k) add(__bfloat162float(w[0][k]), __bfloat162float(w[1][k]), k);
+        for (int k = 0; k < rank; ++k) {
+            const bf16* q = w + static_cast<size_t>(k) * channels;
+            add(__bfloat162float(q[0]), two ? __bfloat162float(q[1]) : 0.f, k);
+        }
     }
 #pragma unroll
-    for (int m = 0; m < 2; ++m) {
-        if (c[m] >= channels) continue;
-#pragma unroll
-        for (int t = 0; t < ROWS / 2; ++t) {
-            const float2 f = unpair(z[m][t]);
-            if (2 * t < n) out[static_cast<size_t>(row0 + 2 * t) * ld_out + c[m]] = expf(-expf(f.x));
-            if (2 * t + 1 < n) out[static_cast<size_t>(row0 + 2 * t + 1) * ld_out + c[m]] = expf(-expf(f.y));
+    for (int t = 0; t < ROWS / 2; ++t) {
+        const float2 f = unpair(z[0][t]), g = unpair(z[1][t]);
+        float* o = out + static_cast<size_t>(row0 + 2 * t) * ld_out + c;
+        if (2 * t < n) {
+            o[0] = expf(-expf(f.x));
+            if (two) o[1] = expf(-expf(g.x));
+        }
+        if (2 * t + 1 < n) {
+            o[ld_out] = expf(-expf(f.y));
+            if (two) o[ld_out + 1] = expf(-expf(g.y));
         }
     }
 }
