@@ -1,6 +1,6 @@
 // Layered models: decoders whose configuration lists every layer with its own sizes and mechanisms (LayerSpec), on a
 // 32-bit residual stream.  This header holds the layer description and the launch prototypes of the kernels such a
-// layer is made of (layered_ops.cu, moe.cu; the bf16 matrix products and attention are gemm_umma.cu and tree_attn.cu).
+// layer is made of (layered_ops.cu, tanh_rows.cu, recurrence.cu, moe.cu; the bf16 matrix products and attention are gemm_umma.cu and tree_attn.cu).
 //
 // Every kernel that handles activations exists for bf16 and for fp32 (T): bf16 is what a model is served in, fp32 runs
 // everything in true 32-bit through plain SIMT matrix products.  Weights are bf16 in both.
